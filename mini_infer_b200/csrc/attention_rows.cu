@@ -4,11 +4,14 @@
 // own rows, a sink score per head in the softmax's denominator, and a distance bias with a slope per
 // head.  Prompt portions and single decoded tokens alike.
 //
+// With `window` > 0 a query at position p sees the keys j > p - window only; chunks wholly before the
+// tile's first window are not walked.
+//
 // A block takes R = 16 MT query rows that share one key/value head (MT = 1: four warps, for steps of
 // single tokens; MT = 2 or 4: eight or sixteen warps, for prompt portions, with two buffers for the
 // chunk's rows where shared memory allows, so that the next chunk is copied while this one is multiplied): with G = nq / nkv query heads per
-// key/value head, the rows are (token, head in group) pairs, R / G tokens by G heads when G divides
-// R, or R of the G heads of one token when R divides G.  It walks the request's keys in chunks of 64
+// key/value head, the rows are (token, head in group) pairs: R / G (rounded down) tokens by G heads when G is
+// below R, else up to R of the G heads of one token; rows left over stand for nothing.  It walks the request's keys in chunks of 64
 // (cut at absolute multiples of 64): the chunk's rows are gathered from their pages into shared
 // memory (un-permuted); each group of four warps owns 16 of the rows, and in it warp w computes the
 // scores of keys 16 w .. 16 w + 15 (S = Q K^T), the four exchange row maxima and sums and the bf16
@@ -100,11 +103,15 @@ __device__ __forceinline__ void gather_rows_async(bf16* __restrict__ dst, int pi
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::: "memory"); }
 
-// Which token (within the tile) and which head a row of a tile of R rows stands for.
+// Which token (within the tile) and which head a row of a tile of R rows stands for.  A row that stands for
+// nothing has a token beyond every tile (and some head of the group).
 struct RowMap {
   int G, R, kvh, hs;
-  __device__ __forceinline__ int token(int r) const { return G >= R ? 0 : r / G; }
-  __device__ __forceinline__ int head(int r) const { return G >= R ? kvh * G + hs * R + r : kvh * G + r % G; }
+  __device__ __forceinline__ int token(int r) const {
+    if (G >= R) return hs * R + r < G ? 0 : 0x3fffffff;
+    return r / G;                       // rows behind the last whole token: R / G, one past the tile's tokens
+  }
+  __device__ __forceinline__ int head(int r) const { return kvh * G + (G >= R ? min(hs * R + r, G - 1) : r % G); }
 };
 
 // DVW: value columns per warp that the accumulators have room for (dv <= 4 * DVW).  DB: two buffers for
@@ -118,7 +125,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
                       const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                       const int* __restrict__ tile_tok0, int tile_tokens, int nq, int nkv, int d, int dv, float scale,
                       const float* __restrict__ sinks, const float* __restrict__ slopes, int v_prefix,
-                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml) {
+                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window) {
   mi_pdl_enter();
   constexpr int R = ROWS * MT, NW = QUARTERS * MT, NT = NW * 32;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -137,7 +144,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   const int warp = (tid >> 5) % QUARTERS, mt = (tid >> 5) / QUARTERS;   // the quarter, and which 16 rows
   const int g = lane >> 2, t4 = lane & 3;                      // the fragment's row (and row + 8) and column pair
   const int G = nq / nkv;
-  const int head_tiles = G >= R ? G / R : 1;
+  const int head_tiles = G >= R ? (G + R - 1) / R : 1;
   int bid = blockIdx.x;
   const int split = bid % n_splits;
   bid /= n_splits;
@@ -156,8 +163,10 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   auto row_token = [&](int r) { return rows.token(r); };
   auto row_head = [&](int r) { return rows.head(r); };
   // this block's run of keys: whole chunks, the same cut for every row of the tile
-  const int chunks_all = (j_end + CHUNK - 1) / CHUNK, chunks_mine = (chunks_all + n_splits - 1) / n_splits;
-  const int j_begin = split * chunks_mine * CHUNK, j_stop = min(j_end, (split + 1) * chunks_mine * CHUNK);
+  const int j_lo = window > 0 ? max(0, p0 - window + 1) : 0;    // the first key that any row sees
+  const int chunk0 = j_lo / CHUNK;
+  const int chunks_all = (j_end + CHUNK - 1) / CHUNK - chunk0, chunks_mine = (chunks_all + n_splits - 1) / n_splits;
+  const int j_begin = (chunk0 + split * chunks_mine) * CHUNK, j_stop = min(j_end, (chunk0 + (split + 1) * chunks_mine) * CHUNK);
 
   // ---- the queries: 16-byte pieces, zero for rows without a token
   const int pieces = d >> 3;
@@ -173,6 +182,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   const int r_lo = mt * ROWS + g, r_hi = r_lo + 8;
   const bool ok_lo = row_token(r_lo) < nt, ok_hi = row_token(r_hi) < nt;
   const int pos_lo = p0 + row_token(r_lo), pos_hi = p0 + row_token(r_hi);
+  const unsigned span = window > 0 ? window : 0x7fffffff;          // a key up to span - 1 positions back is seen
   const float slope_lo = slopes ? slopes[row_head(r_lo)] : 0.f, slope_hi = slopes ? slopes[row_head(r_hi)] : 0.f;
   constexpr float LOG2E = 1.4426950408889634f;
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;     // running maximum (in units of log2) and sum
@@ -188,7 +198,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
     if (tid < CHUNK) {
       const int j = j0 + tid;
       int base = -1;
-      if (j < j_stop) {
+      if (j >= j_lo && j < j_stop) {
         const int page = block_table[(size_t)trow * bt_stride + j / page_size];
         base = (page * nkv + kvh) * page_size + j % page_size;
       }
@@ -256,7 +266,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
         const int j = j0 + warp * 16 + n * 8 + 2 * t4 + (e & 1);
         const bool hi = e >= 2;
         const int pos = hi ? pos_hi : pos_lo;
-        const bool ok = (hi ? ok_hi : ok_lo) && j <= pos;
+        const bool ok = (hi ? ok_hi : ok_lo) && (unsigned)(pos - j) < span;      // not behind the query, not before its window
         const float v = ok ? (s[n][e] * scale - (hi ? slope_hi : slope_lo) * (float)(pos - j)) * LOG2E : -INFINITY;
         s[n][e] = v;
         if (hi) mx_hi = fmaxf(mx_hi, v); else mx_lo = fmaxf(mx_lo, v);
@@ -398,7 +408,7 @@ attention_rows_merge_kernel(const float* __restrict__ part_o, const float* __res
   int bid = blockIdx.x / R;
   const int unit = bid;
   const int G = nq / nkv;
-  const int head_tiles = G >= R ? G / R : 1;
+  const int head_tiles = G >= R ? (G + R - 1) / R : 1;
   const int hs = bid % head_tiles;
   bid /= head_tiles;
   const int kvh = bid % nkv;
@@ -459,12 +469,10 @@ attention_rows_merge_kernel(const float* __restrict__ part_o, const float* __res
   }
 }
 
-// Tokens per tile of `rows` rows for a group of G query heads per key/value head, or 0 when the
-// kernel does not take the group size.
+// Tokens per tile of `rows` rows for a group of G query heads per key/value head (0: no such rows or group).
 extern "C" int mi_attention_rows_tile_tokens(int G, int rows) {
   if (G <= 0 || (rows != ROWS && rows != 2 * ROWS && rows != 4 * ROWS)) return 0;
-  if (G >= rows) return G % rows == 0 ? 1 : 0;
-  return rows % G == 0 ? rows / G : 0;
+  return G >= rows ? 1 : rows / G;
 }
 
 extern "C" int mi_attention_rows_supported(int nq, int nkv, int d, int dv, int v_prefix) {
@@ -479,7 +487,7 @@ extern "C" int mi_attention_rows_supported(int nq, int nkv, int d, int dv, int v
 extern "C" int mi_attention_rows_scratch(int n_tiles, int rows, int nq, int nkv, int dv, int n_splits,
                                          long long* o_floats, long long* ml_floats) {
   const int G = nq / nkv;
-  const long long units = (long long)n_tiles * nkv * (G >= rows ? G / rows : 1);
+  const long long units = (long long)n_tiles * nkv * (G >= rows ? (G + rows - 1) / rows : 1);
   *o_floats = n_splits > 1 ? units * n_splits * rows * dv : 0;
   *ml_floats = n_splits > 1 ? units * n_splits * rows * 2 : 0;
   return 0;
@@ -491,7 +499,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
                                  const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens, int rows,
                                  int nq, int nkv, int d, int dv, float scale, const float* sinks, const float* slopes,
                                  int v_prefix, int n_splits, float* part_o, float* part_ml, int stages,
-                                 cudaStream_t stream) {
+                                 int window, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (stages != 1 && stages != 2) MI_REFUSE("attention_rows: one or two buffers for a chunk, not %d", stages);
   if ((rows == 2 * ROWS && stages != 2) || (rows == ROWS && stages != 1))
@@ -501,14 +509,14 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
   const int G = nq / nkv;
   if (!mi_attention_rows_tile_tokens(G, rows) || tile_tokens != mi_attention_rows_tile_tokens(G, rows))
     MI_REFUSE("attention_rows: tiles of %d tokens and %d rows do not fit a group of %d heads", tile_tokens, rows, G);
-  if (page_size <= 0) MI_REFUSE("attention_rows: bad page size %d", page_size);
+  if (page_size <= 0 || window < 0) MI_REFUSE("attention_rows: bad page size %d or window %d", page_size, window);
   if (!v_prefix && !vcache) MI_REFUSE("attention_rows: no value cache");
   if (n_splits < 1 || n_splits > MERGE_MAX_SPLITS || (n_splits > 1 && (!part_o || !part_ml)))
     MI_REFUSE("attention_rows: 1 to %d runs of keys, and scratch for more than one", MERGE_MAX_SPLITS);
   if (!mi_aligned(q, 16) || !mi_aligned(kcache, 16) || !mi_aligned(vcache, 16) || !mi_aligned(out, 4) ||
       !mi_aligned(part_o, 16) || q_stride % 8 || out_stride % 2 || (n_splits > 1 && (!mi_aligned(out, 8) || out_stride % 4)))
     MI_REFUSE("attention_rows: q and the caches must be 16-byte aligned with rows of whole 16-byte pieces");
-  const long long units = (long long)n_tiles * nkv * (G >= rows ? G / rows : 1);
+  const long long units = (long long)n_tiles * nkv * (G >= rows ? (G + rows - 1) / rows : 1);
   const long long blocks = units * n_splits;
   if (blocks > 0x7fffffffLL || units * rows > 0x7fffffffLL) MI_REFUSE("attention_rows: too many blocks for one launch");
   const size_t smem = ((size_t)rows * (d + PAD) +
@@ -526,7 +534,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
     MI_LAUNCH(kern, (unsigned)blocks, QUARTERS * MT * 32, smem, stream, (const bf16*)q, q_stride, (bf16*)out,    \
               out_stride, (const bf16*)kcache, (const bf16*)vcache, block_table, bt_stride, table_rows, page_size, \
               q_start, q_len, kv_len, tile_req, tile_tok0, tile_tokens, nq, nkv, d, dv, scale, sinks, slopes,    \
-              v_prefix, n_splits, part_o, part_ml);                                                             \
+              v_prefix, n_splits, part_o, part_ml, window);                                                     \
   } while (0)
   if (rows == ROWS) {
     if (dv <= 128) MI_GO(32, 1, false);

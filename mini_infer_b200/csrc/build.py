@@ -45,6 +45,7 @@ LIBRARIES: dict[str, tuple[list[str], list[str], list[str]]] = {
     "stream": (["stream.cu"], ["common.cuh"], []),
     "qk_prepare": (["qk_prepare.cu"], ["common.cuh"], []),
     "attention_rows": (["attention_rows.cu"], ["common.cuh"], []),
+    "depth": (["depth.cu"], ["common.cuh"], []),
 }
 
 

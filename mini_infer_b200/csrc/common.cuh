@@ -194,4 +194,9 @@ __device__ __forceinline__ void mi_rotate(float x1, float x2, float s, float c, 
   y2 = __fadd_rn(__fmul_rn(x2, c), __fmul_rn(x1, s));
 }
 
+// An activation of one value: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0.
+__device__ __forceinline__ float mi_xielu(float z, float a, float b) {
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
+
 static inline bool mi_aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) % a) == 0; }

@@ -219,8 +219,11 @@ struct EpilogueFusion {
   float* residual;
   const float* gain;
   float* stats_out;
+  float act_a, act_b;      // the numbers of an activation of single values (ACT_XIELU)
 };
 #define FUSED_MAX_TOKENS 16
+// `swiglu` beyond the gated forms: an activation of every value of the product by itself
+#define ACT_XIELU 3
 
 template <typename OutT, bool kFused>
 __global__ void __launch_bounds__(GT_THREADS, 1)
@@ -418,6 +421,12 @@ gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
           fus.stats_out[tile * FUSED_MAX_TOKENS + etid] =
               (square_sums[0][etid] + square_sums[1][etid]) + (square_sums[2][etid] + square_sums[3][etid]);
         asm volatile("bar.sync 1, 128;\n" ::: "memory");   // the sums are read before the next tile writes them
+      } else if (swiglu == ACT_XIELU) {
+        if (n < N) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(mi_xielu(v[j], fus.act_a, fus.act_b));
+        }
       } else if (swiglu) {
         // rows alternate gate, up: the even lane of a pair has the gate, its neighbour the up
 #pragma unroll
@@ -619,7 +628,8 @@ extern "C" int mi_gemm_tma_workspace(int M, int N, int blocks, long long* partia
 
 // x [M, K] bf16 (row stride ldx), w [N, K] bf16 contiguous, y [M, N] (row stride ldy) bf16 or
 // fp32.  With `swiglu` (1: SiLU, 2: the tanh form of GELU) the rows of w alternate gate, up and y is [M, N / 2]:
-// y[m, i] = act(x w[2i]) * (x w[2i+1]), computed on the fp32 accumulators.  `blocks` is the number of persistent blocks (the number of SMs); `partials` and
+// y[m, i] = act(x w[2i]) * (x w[2i+1]), computed on the fp32 accumulators; with `swiglu` 3 y is [M, N] and every value
+// passes mi_xielu with act_a and act_b.  `blocks` is the number of persistent blocks (the number of SMs); `partials` and
 // `counters` (zero before the first call; the kernel leaves them zero) as mi_gemm_tma_workspace
 // says.
 //
@@ -631,8 +641,8 @@ extern "C" int mi_gemm_tma_workspace(int M, int N, int blocks, long long* partia
 extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N,
                                  int K, int out_dtype, int swiglu, int blocks, float* partials, int* counters,
                                  const float* stats_in, int stat_tiles, int width, float eps, float* residual,
-                                 const float* gain, float* stats_out, cudaStream_t stream) {
-  EpilogueFusion fus = {stats_in, stat_tiles, width > 0 ? 1.f / (float)width : 0.f, eps, residual, gain, stats_out};
+                                 const float* gain, float* stats_out, float act_a, float act_b, cudaStream_t stream) {
+  EpilogueFusion fus = {stats_in, stat_tiles, width > 0 ? 1.f / (float)width : 0.f, eps, residual, gain, stats_out, act_a, act_b};
   if (stats_in || residual) {
     if (M > FUSED_MAX_TOKENS)
       MI_REFUSE("gemm_tma: the fused epilogues take at most %d rows of x, got %d", FUSED_MAX_TOKENS, M);
@@ -642,8 +652,8 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
       MI_REFUSE("gemm_tma: the residual epilogue needs a gain and room for its statistics, and no gate/up pairs");
     if (residual && !mi_aligned(residual, 4)) MI_REFUSE("gemm_tma: misaligned residual stream");
   }
-  if (swiglu < 0 || swiglu > 2) MI_REFUSE("gemm_tma: unknown gate activation %d", swiglu);
-  if (swiglu && (N % 2)) MI_REFUSE("gemm_tma: the gate/up epilogue needs an even number of rows of W, got %d", N);
+  if (swiglu < 0 || swiglu > ACT_XIELU) MI_REFUSE("gemm_tma: unknown activation %d", swiglu);
+  if (swiglu && swiglu != ACT_XIELU && (N % 2)) MI_REFUSE("gemm_tma: the gate/up epilogue needs an even number of rows of W, got %d", N);
   if (M <= 0 || N <= 0) return 0;
   if (M > MAX_TOKENS) MI_REFUSE("gemm_tma: %d rows of x; this kernel takes at most %d", M, MAX_TOKENS);
   if (K <= 0 || K % 8 != 0 || ldx % 8 != 0)
@@ -709,5 +719,5 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
 extern "C" int mi_gemm_tma(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
                            int out_dtype, int swiglu, int blocks, float* partials, int* counters, cudaStream_t stream) {
   return mi_gemm_tma_fused(x, ldx, w, y, ldy, M, N, K, out_dtype, swiglu, blocks, partials, counters, nullptr, 0, 0,
-                           0.f, nullptr, nullptr, nullptr, stream);
+                           0.f, nullptr, nullptr, nullptr, 0.f, 0.f, stream);
 }

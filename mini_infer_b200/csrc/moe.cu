@@ -52,7 +52,9 @@ __device__ __forceinline__ float mi_clamped_glu_value(float g, float u, float li
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 moe_select_kernel(const float* __restrict__ logits, int stride, int* __restrict__ ids,
                   float* __restrict__ weights, int M, int E, int top, int mode, int n_groups,
-                  int keep, float scale, const float* __restrict__ correction, int group_top2) {
+                  int keep, float scale, const float* __restrict__ correction, int group_top2,
+                  const float* __restrict__ bias) {
+  // bias [E]: added to the logits before anything else; correction [E] (mode 2): to the choice scores alone
   mi_pdl_enter();
   __shared__ float choice_sh[ROUTE_WARPS][32 * ROUTE_MAX_PER_LANE];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -64,7 +66,7 @@ moe_select_kernel(const float* __restrict__ logits, int stride, int* __restrict_
 #pragma unroll
   for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
-    lg[i] = e < E ? z[e] : -INFINITY;
+    lg[i] = e < E ? z[e] + (bias ? bias[e] : 0.f) : -INFINITY;
     sc[i] = 0.f;
     if (mode == 2 && e < E) {
       sc[i] = 1.f / (1.f + expf(-lg[i]));
@@ -185,7 +187,7 @@ moe_select_kernel(const float* __restrict__ logits, int stride, int* __restrict_
 
 extern "C" int mi_moe_select(const float* logits, int stride, int* ids, float* weights, int M, int E, int top,
                              int mode, int n_groups, int keep, float scale, const float* correction,
-                             int group_top2, cudaStream_t stream) {
+                             int group_top2, const float* bias, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (E <= 0 || E > 32 * ROUTE_MAX_PER_LANE) MI_REFUSE("moe: %d experts (1 to %d are taken)", E, 32 * ROUTE_MAX_PER_LANE);
   if (top <= 0 || top > E || top > 32) MI_REFUSE("moe: %d of %d experts per token", top, E);
@@ -196,7 +198,7 @@ extern "C" int mi_moe_select(const float* logits, int stride, int* ids, float* w
     if (keep * (E / n_groups) < top) MI_REFUSE("moe: %d groups of %d experts cannot give %d experts", keep, E / n_groups, top);
   }
   MI_LAUNCH((moe_select_kernel), (M + ROUTE_WARPS - 1) / ROUTE_WARPS, 32 * ROUTE_WARPS, 0, stream, logits, stride, ids,
-            weights, M, E, top, mode, n_groups, keep, scale, correction, group_top2);
+            weights, M, E, top, mode, n_groups, keep, scale, correction, group_top2, bias);
   MI_RETURN_LAUNCH_STATUS();
 }
 

@@ -196,7 +196,7 @@ def _sig_gemm_tma(lib: ctypes.CDLL) -> None:
                                 c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]
     lib.mi_gemm_tma_fused.argtypes = [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int,
                                       c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
-                                      c_void_p, c_void_p, c_void_p, c_void_p]
+                                      c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p]
     lib.mi_gemm_tma_workspace.argtypes = [c_int, c_int, c_int, ctypes.POINTER(ctypes.c_longlong),
                                           ctypes.POINTER(c_int)]
     lib.mi_gemm_tma_status.argtypes = [c_int]
@@ -266,7 +266,7 @@ def _sig_recurrent(lib: ctypes.CDLL) -> None:
 def _sig_moe(lib: ctypes.CDLL) -> None:
     ll = ctypes.c_longlong
     lib.mi_moe_select.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_float, c_void_p, c_int, c_void_p]
+                                  c_float, c_void_p, c_int, c_void_p, c_void_p]
     lib.mi_moe_plan.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
     lib.mi_moe_tile_rows.argtypes = [c_int]
     lib.mi_moe_tile_rows.restype = c_int
@@ -295,6 +295,16 @@ def _sig_stream(lib: ctypes.CDLL) -> None:
     lib.mi_token_gate.argtypes = [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int,
                                   c_int, c_int, c_void_p]
     lib.mi_scale_f32.argtypes = [c_void_p, ll, c_float, c_void_p]
+    lib.mi_xielu_map.argtypes = [c_void_p, c_void_p, ll, c_float, c_float, c_int, c_void_p]
+
+
+def _sig_depth(lib: ctypes.CDLL) -> None:
+    ll = ctypes.c_longlong
+    lib.mi_branch_depth.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, ll, c_void_p,
+                                    c_void_p, c_int, c_int, c_int, c_void_p]
+    lib.mi_input_conv.argtypes = [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, ll, c_void_p, c_void_p, c_void_p,
+                                  c_void_p, c_int, c_int, c_int, c_int, c_void_p]
 
 
 def _sig_qk_prepare(lib: ctypes.CDLL) -> None:
@@ -303,7 +313,7 @@ def _sig_qk_prepare(lib: ctypes.CDLL) -> None:
                                           c_void_p, c_int, c_int, c_int, c_void_p]
     lib.mi_latent_prepare.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                       c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p,
-                                      c_void_p, c_int, c_int, c_int, c_void_p]
+                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
 
 
     lib.mi_qk_norm_rope_store.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -316,13 +326,14 @@ def _sig_attention_rows(lib: ctypes.CDLL) -> None:
     lib.mi_attention_rows.argtypes = [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
+        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p]
     lib.mi_attention_rows_tile_tokens.argtypes = [c_int, c_int]
     lib.mi_attention_rows_supported.argtypes = [c_int, c_int, c_int, c_int, c_int]
 
 
 _SIGNATURES = {
     "attention_rows": _sig_attention_rows,
+    "depth": _sig_depth,
     "stream": _sig_stream,
     "qk_prepare": _sig_qk_prepare,
     "layernorm": _sig_layernorm,
@@ -1007,12 +1018,13 @@ class RowStats:
 def gemm_tma(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
              swiglu: bool | int = False, row_stats: RowStats | None = None,
              residual: torch.Tensor | None = None, gain: torch.Tensor | None = None,
-             eps: float = 0.0):
+             eps: float = 0.0, act: tuple[str, tuple[float, float]] | None = None):
     """``x [M <= 128, K] @ w [N, K]^T`` for bfloat16 operands on the tcgen05 tensor cores,
     streaming ``w`` once through TMA (gemm_tma.cu); the result is bfloat16 or float32.  With
     ``swiglu`` (True or 1: SiLU; 2: the tanh form of GELU) the rows of ``w`` alternate gate, up and
     the result is ``[M, N / 2]``: ``act(gate) * up`` computed on the fp32 accumulators in the
-    product's epilogue.
+    product's epilogue.  ``act``: an activation of every single value of the product (a key of ``UNARY_ACT``
+    and its numbers), likewise on the accumulators.
 
     Two fused forms for at most 16 rows.  ``row_stats``: every row of the product is first
     scaled by ``rsqrt(sum of its squares / width + eps)`` (the input was multiplied by a norm's
@@ -1033,6 +1045,8 @@ def gemm_tma(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
     partial, count = _tma_workspace(x.device, int(floats.value), int(counters.value))
     if swiglu and N % 2:
         raise KernelError("gemm_tma: the gate/up epilogue needs an even number of rows")
+    if act is not None and (swiglu or residual is not None):
+        raise KernelError("gemm_tma: an activation of single values goes with the plain product")
     n_out = N // 2 if swiglu else N
     out = torch.empty((M, n_out), dtype=out_dtype, device=x.device)
     sums_in = tiles_in = width = None
@@ -1051,9 +1065,10 @@ def gemm_tma(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
         stats_out = torch.empty((-(-N // TMA_GEMM_TILE_ROWS), TMA_GEMM_STAT_TOKENS), dtype=torch.float32,
                                 device=x.device)
     rc = lib.mi_gemm_tma_fused(_ptr(x), x.stride(0) if M > 1 else K, _ptr(w), _ptr(out), n_out, M, N, K,
-                               _code(out_dtype), int(swiglu), blocks, _ptr(partial), _ptr(count),
-                               _ptr(sums_in), tiles_in or 0, width or 0, row_stats.eps if row_stats else 0.0,
-                               _ptr(residual), _ptr(gain), _ptr(stats_out), _stream())
+                               _code(out_dtype), UNARY_ACT[act[0]] if act else int(swiglu), blocks, _ptr(partial),
+                               _ptr(count), _ptr(sums_in), tiles_in or 0, width or 0,
+                               row_stats.eps if row_stats else 0.0, _ptr(residual), _ptr(gain), _ptr(stats_out),
+                               act[1][0] if act else 0.0, act[1][1] if act else 0.0, _stream())
     _finish(lib, rc, "gemm_tma")
     if residual is not None:
         return out, RowStats(stats_out, N, eps)
@@ -1109,6 +1124,25 @@ def linear_swiglu(x: torch.Tensor, w_pairs: torch.Tensor, row_stats: "RowStats |
     if act == "silu":
         return silu_mul(linear(x, w_pairs), pairs=True)
     return glu_mul_pairs(linear(x, w_pairs), act)
+
+
+UNARY_ACT = {"xielu": 3}      # the streaming product's epilogue numbers
+
+
+def linear_activated(x: torch.Tensor, w: torch.Tensor, act: str, numbers: tuple[float, float]) -> torch.Tensor:
+    """``act(x w^T)`` value by value in fp32; ``"xielu"`` with ``numbers = (a, b)``: ``a z^2 + z / 2`` for ``z > 0``,
+    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``.  Decode-sized bfloat16 inputs run the activation in the streaming
+    product's epilogue, everything else runs ``linear`` and the activation in place."""
+    if act not in UNARY_ACT:
+        raise KernelError(f"linear_activated: unknown activation {act!r}")
+    if (x.dtype == torch.bfloat16 and USE_TMA_GEMM and x.shape[0] <= TMA_GEMM_DISPATCH_ROWS
+            and w.dtype == torch.bfloat16 and gemm_tma_ok(x, w)):
+        return gemm_tma(x, w, torch.bfloat16, act=(act, numbers))
+    y = linear(x, w)
+    lib = _lib("stream")
+    rc = lib.mi_xielu_map(_ptr(y), _ptr(y), y.numel(), float(numbers[0]), float(numbers[1]), _code(y.dtype), _stream())
+    _finish(lib, rc, "xielu")
+    return y
 
 
 _MM_OUT_DTYPE: bool | None = None
@@ -1586,7 +1620,7 @@ ROUTE_MODES = {"chosen": 0, "all": 1, "sigmoid": 2}
 def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, all_scores: bool = False, groups: int = 0,
               keep_groups: int = 0, scale: float = 1.0, scores: str | None = None,
               correction: torch.Tensor | None = None, group_top2: bool = False, experts: int | None = None,
-              return_logits: bool = False):
+              return_logits: bool = False, bias: torch.Tensor | None = None):
     """fp32 router logits ``x router^T``; per token the ``top`` experts with the largest logits
     (int32 ``[M, top]``, largest first) and their weights (fp32): the softmax over those logits alone,
     or, with ``all_scores``, their scores under the softmax over all experts divided by the sum of
@@ -1596,8 +1630,9 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, all_scores: bo
     sigmoids; the choice adds ``correction`` (fp32 ``[experts]``) per expert; the weights are the chosen
     scores times ``scale``, with no division by their sum).  ``group_top2``: a group counts as the sum of its two best
     choice scores.  ``experts``: only the router's first ``experts`` rows are experts; the other rows ride
-    along in the product and ``return_logits`` hands all logits back as a third result."""
-    _cuda(x, router, correction)
+    along in the product and ``return_logits`` hands all logits back as a third result.  ``bias`` (fp32
+    ``[experts]``) is added to the logits before anything else."""
+    _cuda(x, router, correction, bias)
     _cols(x, "moe")
     if router.dim() != 2 or router.shape[1] != x.shape[1] or router.dtype != x.dtype or not router.is_contiguous():
         raise KernelError("moe: the router must be a contiguous [experts, H] matrix in x's dtype")
@@ -1607,13 +1642,14 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, top: int, *, all_scores: bo
         raise KernelError(f"moe: {E} experts of a router with {router.shape[0]} rows")
     mode = ROUTE_MODES[scores] if scores is not None else (1 if all_scores else 0)
     _f32vec(correction, E, "moe (correction)")
+    _f32vec(bias, E, "moe (bias)")
     logits = linear(x, router, out_dtype=torch.float32)      # exact products, fp32 sums, for either dtype
     ids = torch.empty((M, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((M, top), dtype=torch.float32, device=x.device)
     lib = _lib("moe")
     rc = lib.mi_moe_select(_ptr(logits), logits.stride(0), _ptr(ids), _ptr(weights), M, E, int(top),
                            mode, int(groups), int(keep_groups), float(scale), _ptr(correction),
-                           1 if group_top2 else 0, _stream())
+                           1 if group_top2 else 0, _ptr(bias), _stream())
     _finish(lib, rc, "moe_select")
     if return_logits:
         return ids, weights, logits
@@ -1888,6 +1924,114 @@ def scale_(x: torch.Tensor, s: float) -> torch.Tensor:
     return x
 
 
+# --------------------------------------------------------------------------------------- behind a branch, along the depth
+
+
+INPUT_CONV_MAX_TAPS = 16
+
+
+def _stream_check(t: torch.Tensor, shape, what: str) -> None:
+    if t.dtype != torch.float32 or tuple(t.shape) != tuple(shape) or not t.is_contiguous():
+        raise KernelError(f"branch_depth: {what} must be contiguous fp32 {tuple(shape)}")
+
+
+def _branch_depth(stream, branch, norm, *, stream_out=None, copy=None, first=None, results=None, n_prev=0, avg=None,
+                  avg_out=None, conv=None, ctx=None, conv_out=None, dtype):
+    if stream.dim() != 2:
+        raise KernelError("branch_depth: the stream must be [M, H]")
+    M, H = stream.shape
+    _stream_check(stream, (M, H), "the stream")
+    w = b = None
+    eps = 0.0
+    if branch is not None:
+        w, b, eps = norm
+        _cols(branch, "branch_depth")
+        if branch.shape != (M, H) or branch.dtype != dtype:
+            raise KernelError("branch_depth: the branch must be [M, H] in the compute dtype")
+        _f32vec(w, H, "branch_depth")
+        _f32vec(b, H, "branch_depth")
+    conv_w = state = slots = None
+    taps, state_stride = 0, 0
+    if conv is not None:
+        conv_w, state = conv
+        taps = _conv_taps(conv_w, H)
+        if M != ctx.n_requests or not ctx.decode_only:
+            raise KernelError("branch_depth: the convolution rides along in steps of single tokens")
+        slots = ctx.state_slot
+        if taps > 1:
+            state_stride = _state_rows(state, "branch_depth")
+    _cuda(stream, branch, first, results, conv_w)
+    lib = _lib("depth")
+    rc = lib.mi_branch_depth(
+        _ptr(stream), _ptr(branch), branch.stride(0) if branch is not None else 0, _ptr(w), _ptr(b), float(eps),
+        _ptr(stream_out), _ptr(copy), _ptr(first), _ptr(results), int(n_prev), _ptr(avg), _ptr(avg_out), _ptr(conv_w),
+        taps, _ptr(state), state_stride, _ptr(slots), _ptr(conv_out), M, H, _code(dtype), _stream())
+    _finish(lib, rc, "branch_depth")
+
+
+def branch_layernorm_add(stream: torch.Tensor, branch: torch.Tensor, gain: torch.Tensor, bias: torch.Tensor, eps: float,
+                         dtype: torch.dtype, keep: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
+    """A branch whose layer norm stands behind it: ``stream + ((y - mean) / sqrt(var + eps) * gain + bias)`` (``stream``
+    fp32 ``[M, H]``, ``y`` the branch's rows in ``dtype``, gain and bias fp32 ``[H]``), in place, or into a new stream
+    with ``keep``.  Returns ``(the updated stream, its copy in dtype)``; for float32 the copy is the stream."""
+    out = torch.empty_like(stream) if keep else stream
+    copy = torch.empty(stream.shape, dtype=dtype, device=stream.device) if dtype != torch.float32 else None
+    _branch_depth(stream, branch, (gain, bias, eps), stream_out=out, copy=copy, dtype=dtype)
+    return out, (out if copy is None else copy)
+
+
+def branch_depth_average(stream: torch.Tensor, branch: torch.Tensor | None, norm, first: torch.Tensor,
+                         results: torch.Tensor, index: int, weights: torch.Tensor, dtype: torch.dtype, ctx,
+                         conv: tuple[torch.Tensor, torch.Tensor | None] | None = None):
+    """What a layer hands on when the results of all layers so far are averaged: with ``X`` the stream with the
+    branch's layer norm added (``norm = (gain, bias, eps)``; no branch: the stream as it is), ``x = sum_j weights[j]
+    X_j`` over ``X_0 = first``, ``X_(j+1) = results[j]`` for ``j < index`` and ``X`` itself, in fp32.  ``X`` is kept in
+    ``results[index]`` where there is such a place.  ``conv = (w [taps, H], state)`` (steps of single tokens): the
+    convolution of ``input_conv`` on ``x`` in the same kernel.  Returns ``(x, the convolved rows or None)``."""
+    M, H = stream.shape
+    _stream_check(first, (M, H), "the first result")
+    _stream_check(weights, (index + 2,), "the weights")
+    if results.dim() != 3 or results.dtype != torch.float32 or tuple(results.shape[1:]) != (M, H) \
+            or not results.is_contiguous() or results.shape[0] < index:
+        raise KernelError("branch_depth: the results must be contiguous fp32 [layers, M, H]")
+    keep = results[index] if index < results.shape[0] else None
+    x = torch.empty_like(stream)
+    conv_out = torch.empty((M, H), dtype=dtype, device=stream.device) if conv is not None else None
+    _branch_depth(stream, branch, norm, stream_out=keep, first=first, results=results if index else None,
+                  n_prev=index + 1, avg=weights, avg_out=x, conv=conv, ctx=ctx, conv_out=conv_out, dtype=dtype)
+    return x, conv_out
+
+
+def _conv_taps(w: torch.Tensor, H: int) -> int:
+    if w.dtype != torch.float32 or w.dim() != 2 or w.shape[1] != H or not w.is_contiguous() \
+            or not 1 <= w.shape[0] <= INPUT_CONV_MAX_TAPS:
+        raise KernelError(f"input_conv: the taps must be contiguous fp32 [1 to {INPUT_CONV_MAX_TAPS}, {H}]")
+    return w.shape[0]
+
+
+def input_conv(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor | None, ctx, dtype: torch.dtype) -> torch.Tensor:
+    """Per channel ``out_t = x_t + sum_j w[j] x_(t - taps + 1 + j)`` over every request's portion, in ``dtype`` (``x``
+    fp32 or in ``dtype``; ``w`` fp32 ``[taps, H]``).  The inputs before a portion are the request's state (fp32
+    ``[slots, taps - 1, H]``, oldest first; zeros at the start of a sequence), which then holds the portion's last
+    inputs."""
+    _cuda(x, w, state)
+    _cols(x, "input_conv")
+    M, H = x.shape
+    taps = _conv_taps(w, H)
+    stride = 0
+    if taps > 1:
+        if state is None:
+            raise KernelError("input_conv: more than one tap needs the per-request state")
+        stride = _state_rows(state, "input_conv")
+    out = torch.empty((M, H), dtype=dtype, device=x.device)
+    lib = _lib("depth")
+    rc = lib.mi_input_conv(_ptr(x), x.stride(0), _code(x.dtype), _ptr(w), taps, _ptr(state), stride, _ptr(ctx.q_start),
+                           _ptr(ctx.q_len), _ptr(ctx.state_slot), _ptr(out), ctx.n_requests, _max_q_len(ctx), H,
+                           _code(dtype), _stream())
+    _finish(lib, rc, "input_conv")
+    return out
+
+
 # --------------------------------------------------------------------------------------- between projection and attention
 
 
@@ -2000,20 +2144,26 @@ def qk_norm_rope_store(packed: torch.Tensor, q_off: int, k_off: int, v_off: int 
 
 
 def latent_prepare(packed: torch.Tensor, q_off: int, nq: int, q_head: int, q_rot_off: int, c_off: int, rank: int,
-                   rot_dim: int, rot: int, *, positions: torch.Tensor, freq: torch.Tensor, c_gain: torch.Tensor,
-                   eps: float, qfull: torch.Tensor, slots: torch.Tensor | None = None,
-                   kcache: torch.Tensor | None = None) -> None:
+                   rot_dim: int, rot: int, *, positions: torch.Tensor, freq: torch.Tensor, c_gain: torch.Tensor | None,
+                   eps: float, qfull: torch.Tensor | None, slots: torch.Tensor | None = None,
+                   kcache: torch.Tensor | None = None, interleaved: bool = False, cq_off: int = 0,
+                   cq_gain: torch.Tensor | None = None, cq_out: torch.Tensor | None = None) -> None:
     """From the packed projection ``[M, stride]`` of a latent attention: the latent (``rank`` columns
     at ``c_off``) gets an RMS norm with ``c_gain``; the key part behind it (``rot_dim`` columns) and
     every query head's part at ``q_rot_off`` within its ``q_head`` columns are rotated by the
     position (half layout over the first ``rot`` dimensions, ``freq`` float64 ``[rot / 2]``).  The
     cache row ``[latent, rotated key part]`` is stored at ``slots`` of ``kcache``
     ``[pages, 1, page_size, rank + rot_dim]``; the rotated query parts go behind the first ``rank``
-    columns of every head of ``qfull [M, nq, rank + rot_dim]``."""
-    _cuda(packed, positions, freq, c_gain, qfull, slots, kcache)
+    columns of every head of ``qfull [M, nq, rank + rot_dim]``.  ``interleaved``: dimension ``2i`` is paired
+    with ``2i + 1`` instead of the half layout.
+
+    The two halves may run apart: without ``c_gain`` (and caches) only the queries are rotated, with ``nq`` 0
+    only the cache row is made.  With ``cq_gain`` (fp32 ``[q rank]``) the columns at ``cq_off`` are the queries' own
+    latent: its RMS norm with that gain goes to ``cq_out [M, q rank]``."""
+    _cuda(packed, positions, freq, c_gain, qfull, slots, kcache, cq_gain, cq_out)
     _cols(packed, "latent_prepare")
     M, width = packed.shape
-    if q_off + nq * q_head > width or c_off + rank + rot_dim > width:
+    if q_off + nq * q_head > width or (c_gain is not None and c_off + rank + rot_dim > width):
         raise KernelError("latent_prepare: a column range lies outside the packed projection")
     if positions.dtype != torch.int32 or positions.shape != (M,):
         raise KernelError("latent_prepare: positions must be int32 [M]")
@@ -2021,7 +2171,16 @@ def latent_prepare(packed: torch.Tensor, q_off: int, nq: int, q_head: int, q_rot
         raise KernelError("latent_prepare: freq must be float64 [rot / 2]")
     _opt_f32(c_gain, rank, "latent_prepare (gain)")
     dk = rank + rot_dim
-    if qfull.shape != (M, nq, dk) or qfull.dtype != packed.dtype or not qfull.is_contiguous():
+    cq_rank = 0
+    if cq_gain is not None:
+        cq_rank = cq_gain.numel()
+        _opt_f32(cq_gain, cq_rank, "latent_prepare (query gain)")
+        if (cq_out is None or cq_out.shape != (M, cq_rank) or cq_out.dtype != packed.dtype
+                or not cq_out.is_contiguous() or cq_off + cq_rank > width):
+            raise KernelError(f"latent_prepare: the queries' latent needs {cq_rank} packed columns and a contiguous output")
+    if kcache is not None and c_gain is None:
+        raise KernelError("latent_prepare: a cache row needs the latent's gain")
+    if nq and (qfull is None or qfull.shape != (M, nq, dk) or qfull.dtype != packed.dtype or not qfull.is_contiguous()):
         raise KernelError(f"latent_prepare: qfull must be contiguous [{M}, {nq}, {dk}] in the packed dtype")
     writes = kcache is not None
     page_size = 0
@@ -2036,6 +2195,7 @@ def latent_prepare(packed: torch.Tensor, q_off: int, nq: int, q_head: int, q_rot
     rc = lib.mi_latent_prepare(_ptr(packed), packed.stride(0), q_off, M, nq, q_head, q_rot_off, c_off, rank, rot_dim,
                                int(rot), _ptr(positions), _ptr(freq), _ptr(c_gain), float(eps), _ptr(qfull),
                                nq * dk, dk, _ptr(slots), _ptr(kcache), page_size, 1 if writes else 0,
+                               1 if interleaved else 0, int(cq_off), cq_rank, _ptr(cq_gain), _ptr(cq_out),
                                _code(packed.dtype), _stream())
     _finish(lib, rc, "latent_prepare")
 
@@ -2046,13 +2206,12 @@ ROWS_ATTENTION_ROWS = (16, 32, 64)   # query rows per block of attention_rows.cu
 
 def rows_attention_tile_tokens(group: int, rows: int = 16) -> int:
     """Tokens per tile of the tensor-core kernel of ``attention_ext`` for ``group`` query heads per
-    key/value head and blocks of ``rows`` rows of (token, head in group), or 0 where it does not take
-    the group size.  The same rule as the library's ``mi_attention_rows_tile_tokens``."""
+    key/value head and blocks of ``rows`` rows of (token, head in group); rows behind the last whole token,
+    or behind a group's last head, stand for nothing.  The same rule as the library's
+    ``mi_attention_rows_tile_tokens`` (0: no such rows or group)."""
     if group <= 0 or rows not in ROWS_ATTENTION_ROWS:
         return 0
-    if group >= rows:
-        return 1 if group % rows == 0 else 0
-    return rows // group if rows % group == 0 else 0
+    return 1 if group >= rows else rows // group
 
 
 def rows_attention_tile_sizes(nq: int, nkv: int, d: int, dv: int, values_in_keys: bool) -> frozenset[int]:
@@ -2066,7 +2225,7 @@ def rows_attention_tile_sizes(nq: int, nkv: int, d: int, dv: int, values_in_keys
 def rows_attention_supported(nq: int, nkv: int, d: int, dv: int, values_in_keys: bool) -> bool:
     """Whether attention_rows.cu takes these sizes (the library's ``mi_attention_rows_supported``, made
     here so that a model it does not take never compiles it): keys a multiple of 16 up to 1024,
-    values a multiple of 32 up to 512, a group size that divides 16 or is a multiple of it."""
+    values a multiple of 32 up to 512."""
     if not USE_ROWS_ATTENTION or nq <= 0 or nkv <= 0 or nq % nkv or not rows_attention_tile_tokens(nq // nkv, 16):
         return False
     if d < 16 or d % 16 or d > 1024 or dv < 32 or dv % 32 or dv > 512:
@@ -2081,7 +2240,8 @@ def _rows_attention_smem(rows: int, d: int, dv: int, values_in_keys: bool, stage
     return (rows * (d + 8) + stages * chunk + rows * 72) * 2 + 32 * rows + stages * 512
 
 
-def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys: bool, device) -> tuple[int, int, int, int]:
+def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys: bool, device,
+                         window: int = 0) -> tuple[int, int, int, int]:
     """``(rows per block, tokens per tile, runs of keys per tile, buffers per chunk)`` for this step:
     steps of single tokens take 16 rows and cut every request's keys into runs, so that the blocks
     fill the GPU; prompt portions take 64 rows with two buffers for the chunk's rows (the next chunk
@@ -2097,8 +2257,10 @@ def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys
                 return rows, tt, 1, stages
         return 16, rows_attention_tile_tokens(group, 16), 1, 1
     tt = rows_attention_tile_tokens(group, 16)
-    units = ctx.tiles[tt][2] * nkv * max(1, group // 16)
+    units = ctx.tiles[tt][2] * nkv * max(1, -(-group // 16))
     chunks = max(1, -(-int(getattr(ctx, "max_kv_len", 0) or 64) // 64))
+    if window:                       # the keys of one window touch at most this many chunks
+        chunks = min(chunks, -(-(window - 1) // 64) + 1)
     splits = max(1, min(-(-4 * _sms(device) // units), chunks, 64))
     return 16, tt, splits, 1
 
@@ -2143,15 +2305,15 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
                              tile_req, tile_tok0, n_tiles, tt, nq, nkv, d, scale, int(window),
                              table_rows=group.table_rows, sinks=sinks, slopes=slopes)
         return
-    if (q.dtype == torch.bfloat16 and not window and not chunk
+    if (q.dtype == torch.bfloat16 and not chunk
             and rows_attention_supported(nq, nkv, d, dv, values_in_keys)
             and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0 and out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0
             and rows_attention_tile_tokens(nq // nkv, 16) in ctx.tiles):
-        rows, tt, splits, stages = _rows_attention_plan(ctx, nq, nkv, d, dv, values_in_keys, q.device)
+        rows, tt, splits, stages = _rows_attention_plan(ctx, nq, nkv, d, dv, values_in_keys, q.device, int(window))
         tile_req, tile_tok0, n_tiles = ctx.q_tiles(tt)
         part_o = part_ml = None
         if splits > 1:
-            units = n_tiles * nkv * max(1, (nq // nkv) // rows)
+            units = n_tiles * nkv * max(1, -(-(nq // nkv) // rows))
             part_o = torch.empty(units * splits * rows * dv, dtype=torch.float32, device=q.device)
             part_ml = torch.empty(units * splits * rows * 2, dtype=torch.float32, device=q.device)
         lib = _lib("attention_rows")
@@ -2159,7 +2321,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), _ptr(vc), _ptr(bt), bt.stride(0),
             _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len),
             _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), tt, rows, nq, nkv, d, dv, float(scale), _ptr(sinks),
-            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, _stream())
+            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, int(window), _stream())
         _finish(lib, rc, "attention")
         if splits > 1:
             launch_count += 1        # the merge of the runs

@@ -141,7 +141,8 @@ latent_prepare_kernel(const T* __restrict__ packed, int stride, int q_off, int n
                       int rank, int rot_dim, int rot, const int* __restrict__ positions,
                       const double* __restrict__ freq, const float* __restrict__ c_gain, float eps,
                       T* __restrict__ qfull, int qfull_stride, int qfull_head, const int* __restrict__ slots,
-                      T* __restrict__ kcache, int page_size, int writes) {
+                      T* __restrict__ kcache, int page_size, int writes, int interleaved, int cq_off, int cq_rank,
+                      const float* __restrict__ cq_gain, T* __restrict__ cq_out) {
   mi_pdl_enter();
   __shared__ float sn[LATENT_MAX_ROT / 2], cs[LATENT_MAX_ROT / 2];
   __shared__ float red[32];
@@ -158,13 +159,37 @@ latent_prepare_kernel(const T* __restrict__ packed, int stride, int q_off, int n
     sn[i] = s;
     cs[i] = c;
   }
-  // the latent's sum of squares (fixed order: by thread, then by warp)
-  float ss = 0.f;
-  for (int k = tid; k < rank; k += blockDim.x) {
-    const float v = mi_to_float(row[c_off + k]);
-    ss += v * v;
+  if (cq_rank > 0) {                   // the queries' own latent: an RMS norm, the next product's input
+    float sq = 0.f;
+    for (int k = tid; k < cq_rank; k += blockDim.x) {
+      const float v = mi_to_float(row[cq_off + k]);
+      sq += v * v;
+    }
+    const float m = 1.f / sqrtf(mi_block_sum(sq, red) / (float)cq_rank + eps);
+    for (int k = tid; k < cq_rank; k += blockDim.x)
+      cq_out[(size_t)t * cq_rank + k] = mi_from_float<T>(mi_to_float(row[cq_off + k]) * m * cq_gain[k]);
   }
-  const float mult = 1.f / sqrtf(mi_block_sum(ss, red) / (float)rank + eps);   // its barriers also publish sn, cs
+  // element k of a rotated part: half layout (k with k + half) or interleaved pairs (2i with 2i + 1)
+  auto rotated = [&](const T* src, int k) {
+    if (k >= rot) return mi_to_float(src[k]);
+    const int i = interleaved ? k >> 1 : (k < half ? k : k - half);
+    const bool upper = interleaved ? (k & 1) : k >= half;
+    const float u = mi_to_float(src[interleaved ? 2 * i : i]), v = mi_to_float(src[interleaved ? 2 * i + 1 : i + half]);
+    float y1, y2;
+    mi_rotate(u, v, sn[i], cs[i], y1, y2);
+    return upper ? y2 : y1;
+  };
+  // the latent's sum of squares (fixed order: by thread, then by warp)
+  float mult = 0.f;
+  if (c_gain) {
+    float ss = 0.f;
+    for (int k = tid; k < rank; k += blockDim.x) {
+      const float v = mi_to_float(row[c_off + k]);
+      ss += v * v;
+    }
+    mult = 1.f / sqrtf(mi_block_sum(ss, red) / (float)rank + eps);
+  }
+  __syncthreads();                     // sn and cs are there
   constexpr int EPC = 16 / (int)sizeof(T);
   const int dk = rank + rot_dim;
   if (writes) {
@@ -175,53 +200,39 @@ latent_prepare_kernel(const T* __restrict__ packed, int stride, int q_off, int n
     for (int k = tid; k < rank; k += blockDim.x)
       kdst[mi_swizzled(k, offset, mk, EPC)] = mi_from_float<T>(mi_to_float(row[c_off + k]) * mult * c_gain[k]);
     const T* kr = row + c_off + rank;
-    for (int k = tid; k < rot_dim; k += blockDim.x) {
-      float y = mi_to_float(kr[k]);
-      if (k < rot) {
-        const int i = k < half ? k : k - half;
-        const float u = mi_to_float(kr[i]), v = mi_to_float(kr[i + half]);
-        float y1, y2;
-        mi_rotate(u, v, sn[i], cs[i], y1, y2);
-        y = k < half ? y1 : y2;
-      }
-      kdst[mi_swizzled(rank + k, offset, mk, EPC)] = mi_from_float<T>(y);
-    }
+    for (int k = tid; k < rot_dim; k += blockDim.x)
+      kdst[mi_swizzled(rank + k, offset, mk, EPC)] = mi_from_float<T>(rotated(kr, k));
   }
   for (int idx = tid; idx < nq * rot_dim; idx += blockDim.x) {
     const int h = idx / rot_dim, k = idx - h * rot_dim;
     const T* qr = row + q_off + h * q_head + q_rot_off;
-    float y = mi_to_float(qr[k]);
-    if (k < rot) {
-      const int i = k < half ? k : k - half;
-      const float u = mi_to_float(qr[i]), v = mi_to_float(qr[i + half]);
-      float y1, y2;
-      mi_rotate(u, v, sn[i], cs[i], y1, y2);
-      y = k < half ? y1 : y2;
-    }
-    qfull[(size_t)t * qfull_stride + h * qfull_head + rank + k] = mi_from_float<T>(y);
+    qfull[(size_t)t * qfull_stride + h * qfull_head + rank + k] = mi_from_float<T>(rotated(qr, k));
   }
 }
 
 extern "C" int mi_latent_prepare(const void* packed, int stride, int q_off, int M, int nq, int q_head, int q_rot_off,
                                  int c_off, int rank, int rot_dim, int rot, const int* positions, const double* freq,
                                  const float* c_gain, float eps, void* qfull, int qfull_stride, int qfull_head,
-                                 const int* slots, void* kcache, int page_size, int writes, int dtype,
+                                 const int* slots, void* kcache, int page_size, int writes, int interleaved,
+                                 int cq_off, int cq_rank, const float* cq_gain, void* cq_out, int dtype,
                                  cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (rank <= 0 || rot_dim < 0 || nq <= 0) MI_REFUSE("latent_prepare: bad sizes rank=%d rot_dim=%d heads=%d", rank, rot_dim, nq);
+  if (cq_rank < 0 || (cq_rank > 0 && (!cq_gain || !cq_out))) MI_REFUSE("latent_prepare: a query latent of %d needs its gain and an output", cq_rank);
+  if (rank <= 0 || rot_dim < 0 || nq < 0) MI_REFUSE("latent_prepare: bad sizes rank=%d rot_dim=%d heads=%d", rank, rot_dim, nq);
   if (rot < 0 || rot > rot_dim || (rot & 1) || rot > LATENT_MAX_ROT)
     MI_REFUSE("latent_prepare: %d rotated dimensions of %d (an even number up to %d)", rot, rot_dim, LATENT_MAX_ROT);
-  if (q_rot_off + rot_dim > q_head || qfull_head < rank + rot_dim) MI_REFUSE("latent_prepare: a head's rotated part lies outside the head");
-  if (!positions || (rot > 0 && !freq) || !c_gain || !qfull) MI_REFUSE("latent_prepare: positions, frequencies, gain and qfull are needed");
+  if (nq > 0 && (q_rot_off + rot_dim > q_head || qfull_head < rank + rot_dim)) MI_REFUSE("latent_prepare: a head's rotated part lies outside the head");
+  if (!positions || (rot > 0 && !freq) || (nq > 0 && !qfull) || (writes && !c_gain))
+    MI_REFUSE("latent_prepare: positions, frequencies, gain and qfull are needed");
   if (writes && (!slots || !kcache || page_size <= 0)) MI_REFUSE("latent_prepare: a cache write needs slots and pages");
   if (dtype == MI_DTYPE_F32)
     MI_LAUNCH((latent_prepare_kernel<float>), M, 128, 0, stream, (const float*)packed, stride, q_off, nq, q_head, q_rot_off,
               c_off, rank, rot_dim, rot, positions, freq, c_gain, eps, (float*)qfull, qfull_stride, qfull_head, slots,
-              (float*)kcache, page_size, writes);
+              (float*)kcache, page_size, writes, interleaved, cq_off, cq_rank, cq_gain, (float*)cq_out);
   else if (dtype == MI_DTYPE_BF16)
     MI_LAUNCH((latent_prepare_kernel<bf16>), M, 128, 0, stream, (const bf16*)packed, stride, q_off, nq, q_head, q_rot_off,
               c_off, rank, rot_dim, rot, positions, freq, c_gain, eps, (bf16*)qfull, qfull_stride, qfull_head, slots,
-              (bf16*)kcache, page_size, writes);
+              (bf16*)kcache, page_size, writes, interleaved, cq_off, cq_rank, cq_gain, (bf16*)cq_out);
   else
     MI_REFUSE("latent_prepare: unknown dtype %d", dtype);
   MI_RETURN_LAUNCH_STATUS();

@@ -381,6 +381,43 @@ extern "C" int mi_token_gate(const void* z, int z_stride, int z_dtype, const voi
   MI_RETURN_LAUNCH_STATUS();
 }
 
+template <typename T, int V>
+__global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n, float a, float b) {
+  mi_pdl_enter();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
+    if (V == 8) {                    // bfloat16, eight values per access
+      uint4 v = reinterpret_cast<const uint4*>(x)[idx];
+      uint32_t* w = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
+        const __nv_bfloat162 o = __floats2bfloat162_rn(mi_xielu(f.x, a, b), mi_xielu(f.y, a, b));
+        w[j] = *reinterpret_cast<const uint32_t*>(&o);
+      }
+      reinterpret_cast<uint4*>(out)[idx] = v;
+    } else {
+      out[idx] = mi_from_float<T>(mi_xielu(mi_to_float(x[idx]), a, b));
+    }
+  }
+}
+
+// out = xielu(x) value by value (mi_xielu); out may be x
+extern "C" int mi_xielu_map(const void* x, void* out, long long n, float a, float b, int dtype, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const bool eight = dtype == MI_DTYPE_BF16 && n % 8 == 0 && mi_aligned(x, 16) && mi_aligned(out, 16);
+  const size_t items = eight ? (size_t)n / 8 : (size_t)n;
+  const int blocks = (int)((items + 255) / 256 < 8192 ? (items + 255) / 256 : 8192);
+  if (dtype == MI_DTYPE_F32)
+    MI_LAUNCH((xielu_kernel<float, 1>), blocks, 256, 0, stream, (const float*)x, (float*)out, items, a, b);
+  else if (dtype == MI_DTYPE_BF16 && eight)
+    MI_LAUNCH((xielu_kernel<bf16, 8>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
+  else if (dtype == MI_DTYPE_BF16)
+    MI_LAUNCH((xielu_kernel<bf16, 1>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
+  else
+    MI_REFUSE("xielu: unknown dtype %d", dtype);
+  MI_RETURN_LAUNCH_STATUS();
+}
+
 __global__ void scale_f32_kernel(float* __restrict__ x, size_t n, float s) {
   mi_pdl_enter();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x)

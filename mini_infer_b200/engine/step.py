@@ -282,8 +282,11 @@ class StepRunner:
                              for gi in range(len(self.cache.groups))]
         if self._layer_caches is None:     # the views never change: build them once
             caches: list[LayerCache] = []
-            for entry in self.model.schedule:
+            input_index = getattr(self.model, "input_state_index", None)
+            for i, entry in enumerate(self.model.schedule):
                 lc = LayerCache(writes=entry.writes_cache)
+                if input_index is not None:
+                    lc.input_state = self.cache.layer_state(input_index(i))
                 if entry.cache in self.cache.layer_place:
                     lc.group, lc.k, lc.v = self.cache.layer_kv(entry.cache)
                 lc.state = self.cache.layer_state(entry.cache)

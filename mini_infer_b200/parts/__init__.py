@@ -5,6 +5,7 @@ from .base import (  # noqa: F401
     DeferredNorm,
     FeedForward,
     GroupView,
+    InputPart,
     KVNeed,
     LayerCache,
     Mixer,
@@ -15,6 +16,7 @@ from .base import (  # noqa: F401
     Position,
     StateNeed,
     StepContext,
+    StreamPart,
     StreamSink,
     build_part,
     lookup,
@@ -22,9 +24,11 @@ from .base import (  # noqa: F401
     register_embedding,
     register_feed_forward,
     register_head,
+    register_input_part,
     register_mixer,
     register_norm,
     register_position,
+    register_stream_part,
 )
 from .model import DecoderModel  # noqa: F401
 from .spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry  # noqa: F401

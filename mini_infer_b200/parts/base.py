@@ -105,6 +105,7 @@ class LayerCache:
     k: torch.Tensor | None = None      # [pages, kv_heads, page_size, head_dim]
     v: torch.Tensor | None = None
     state: torch.Tensor | None = None  # [request slots, *StateNeed.shape]
+    input_state: torch.Tensor | None = None   # the same for the layer's input part
     writes: bool = True
 
 
@@ -288,12 +289,33 @@ class StreamCopy(BranchSum):
     To a part that only knows ``BranchSum`` it is an empty sum."""
 
     rounded: torch.Tensor | None = None
+    # what the next layer's mixer reads, where whoever finished the stream has already run that layer's
+    # input part (``StreamPart.prepares_input``); ``rounded`` may then be missing
+    prepared: torch.Tensor | None = None
 
     @classmethod
-    def of(cls, rounded: torch.Tensor) -> "StreamCopy":
+    def of(cls, rounded: torch.Tensor | None, prepared: torch.Tensor | None = None) -> "StreamCopy":
         c = cls(())
-        c.rounded = rounded
+        c.rounded, c.prepared = rounded, prepared
         return c
+
+
+class PendingBranch(BranchSum):
+    """What a layer hands on when its last branch has run but not what stands behind it: ``norm`` (a norm
+    with ``add_branch``) is still to take the branch's output ``branch`` and add it to the stream.  Handed
+    only to a stream part that asks for it (``StreamPart.finishes_branch``)."""
+
+    norm: "Norm | None" = None
+    branch: torch.Tensor | None = None
+
+    @classmethod
+    def of(cls, norm: "Norm", branch: torch.Tensor) -> "PendingBranch":
+        c = cls(())
+        c.norm, c.branch = norm, branch
+        return c
+
+    def total(self):
+        raise RuntimeError("a branch whose norm has not run cannot be summed")
 
 
 class Norm(Part):
@@ -355,15 +377,36 @@ class FeedForward(Part):
         return False
 
 
+class InputPart(Part):
+    """Something that works on what a mixer reads, right before it (``LayerSpec.mixer_input``), and may keep
+    a per-request state of its own (``state_need``; handed in as ``LayerCache.input_state``).
+
+    ``forward(h, ctx, cache) -> h'``: ``h`` as the arrangement has it (the fp32 stream, or a tensor of the
+    compute dtype), ``h'`` in the compute dtype."""
+
+    def state_need(self) -> StateNeed | None:
+        return None
+
+    def forward(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        raise NotImplementedError
+
+
 class StreamPart(Part):
     """Something a model does to the residual stream between two layers (``ScheduleEntry.before``).
 
     ``forward(x, residual, ctx, embedded) -> (x, residual)`` with ``(x, residual)`` as layers hand them
     on (``x``: what is not yet added to the fp32 stream ``residual``; ``residual`` None before the first
     layer, when ``x`` is the embedding's output) and ``embedded`` the embedding's output of this step,
-    which must not be changed.  ``needs_embedding`` tells the model to keep it."""
+    which must not be changed.  ``needs_embedding`` tells the model to keep it.
+
+    Two things a part behind a layer (``ScheduleEntry.after``) may say.  ``finishes_branch``: it takes a
+    ``PendingBranch`` in ``x``'s place, so that the norm and the sum behind the layer's last branch run in its
+    own kernel.  ``prepares_input``: it is also given ``following=(input part, cache)`` of the layer that comes
+    next, or None, and may run that input part on its result (``StreamCopy.prepared``)."""
 
     needs_embedding: ClassVar[bool] = False
+    finishes_branch: ClassVar[bool] = False
+    prepares_input: ClassVar[bool] = False
 
     def forward(self, x, residual, ctx: StepContext, embedded: torch.Tensor | None):
         raise NotImplementedError
@@ -378,6 +421,12 @@ class Arrangement:
     """
 
     kind: ClassVar[str] = ""
+    # whether the layer can leave its last branch's norm and sum to the part behind it (then called with
+    # ``leave_branch=True``, it hands on a ``PendingBranch``)
+    leaves_branch: ClassVar[bool] = False
+    # whether the arrangement runs an input part in front of its mixer (``mixer_input``)
+    takes_mixer_input: ClassVar[bool] = False
+    mixer_input: "InputPart | None" = None
 
     def __init__(self, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm,
                  feed_forward_norm: Norm, position: Position | None) -> None:
@@ -389,6 +438,8 @@ class Arrangement:
 
     def parts(self) -> list[Part]:
         ps: list[Part] = [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
+        if self.mixer_input is not None:
+            ps.append(self.mixer_input)
         if self.position is not None:
             ps.append(self.position)
         return ps
@@ -415,6 +466,7 @@ _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {
     "embedding": {},
     "head": {},
     "stream": {},
+    "input": {},
 }
 
 
@@ -457,8 +509,12 @@ def register_stream_part(kind: str, cls, *, replace: bool = False) -> None:
     _register("stream", kind, cls, replace)
 
 
+def register_input_part(kind: str, cls, *, replace: bool = False) -> None:
+    _register("input", kind, cls, replace)
+
+
 def lookup(family: str, kind: str):
-    from . import builtin, experts, latent, mixers  # noqa: F401  (register the parts that ship with the package)
+    from . import builtin, depth, experts, latent, mixers  # noqa: F401  (register the parts that ship with the package)
 
     try:
         return _REGISTRIES[family][kind]

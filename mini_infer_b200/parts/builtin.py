@@ -23,6 +23,7 @@ from .base import (
     Norm,
     ParamDecl,
     Part,
+    PendingBranch,
     PlanNeeds,
     Position,
     StepContext,
@@ -204,12 +205,50 @@ class BranchRMSNorm(Norm):
         self.mult = float(self.spec.params.get("mult", 1.0))
         self.dtype = dtype
 
-    def add_branch(self, stream: torch.Tensor, y: torch.Tensor) -> torch.Tensor:
-        """Adds the normed branch to the fp32 ``stream`` in place; returns the stream's copy in the
-        compute dtype (the stream itself for float32)."""
+    def add_branch(self, stream: torch.Tensor, y: torch.Tensor, keep: bool = False):
+        """Adds the normed branch to the fp32 ``stream``, in place unless it is to be kept (``keep``).  Returns
+        ``(stream, its copy in the compute dtype)``; for float32 the copy is the stream itself."""
         if isinstance(y, BranchSum):
             y = y.total()
-        return ops.scaled_norm_add(stream, y, self.weight, self.eps, self.mult, self.dtype)
+        if keep:
+            stream = stream.clone()
+        return stream, ops.scaled_norm_add(stream, y, self.weight, self.eps, self.mult, self.dtype)
+
+    def forward(self, x, residual, rows=None):
+        raise RuntimeError("this norm stands behind a branch; the arrangement calls add_branch")
+
+
+class BranchLayerNorm(Norm):
+    """A layer norm that stands behind a branch: the stream takes ``s * ((y - mean) / sqrt(var + eps) * w + b)``
+    of the branch's output ``y`` (``add_branch``), ``var`` the mean of the squared deviations and ``s``, with
+    ``layer_scale``, one number per channel.  Everything from the statistics to the sum is fp32; ``s`` is
+    multiplied into ``w`` and ``b`` once.
+
+    params: ``hidden_size``, ``eps``, optional ``layer_scale`` (default False).
+    tensors: ``weight``, ``bias`` and, as asked, ``scale``, each ``[hidden_size]``.
+    """
+
+    def param_decls(self):
+        H = int(self.param("hidden_size"))
+        decls = {"weight": ParamDecl((H,), "gain"), "bias": ParamDecl((H,), "table")}
+        if self.spec.params.get("layer_scale", False):
+            decls["scale"] = ParamDecl((H,), "gain")
+        return decls
+
+    def bind(self, tensors, dtype, device):
+        self.weight = tensors["weight"].to(torch.float32).contiguous()
+        self.bias = tensors["bias"].to(torch.float32).contiguous()
+        if self.spec.params.get("layer_scale", False):
+            scale = tensors["scale"].to(torch.float32)
+            self.weight, self.bias = self.weight * scale, self.bias * scale
+        self.eps = float(self.param("eps"))
+        self.dtype = dtype
+
+    def add_branch(self, stream: torch.Tensor, y: torch.Tensor, keep: bool = False):
+        """As ``BranchRMSNorm.add_branch``."""
+        if isinstance(y, BranchSum):
+            y = y.total()
+        return ops.branch_layernorm_add(stream, y, self.weight, self.bias, self.eps, self.dtype, keep=keep)
 
     def forward(self, x, residual, rows=None):
         raise RuntimeError("this norm stands behind a branch; the arrangement calls add_branch")
@@ -230,6 +269,17 @@ def stream_and_copy(x, residual, dtype: torch.dtype):
     if x is not None:
         residual = residual + x.to(torch.float32)
     return residual, ops.scaled_norm_add(residual, None, None, 0.0, 1.0, dtype)
+
+
+def fp32_stream(x, residual) -> torch.Tensor:
+    """The fp32 stream alone, from what a layer is handed (``stream_and_copy`` without the copy)."""
+    if isinstance(x, StreamCopy) and residual is not None:
+        return residual
+    if isinstance(x, BranchSum):
+        x = x.total() if len(x) or x.stream_add is not None or x.row_add is not None else None
+    if residual is None:
+        return x if x.dtype == torch.float32 else x.to(torch.float32)
+    return residual if x is None else residual + x.to(torch.float32)
 
 
 class NoNorm(Norm):
@@ -527,6 +577,35 @@ class ClampedGLU(FeedForward):
         return self.down(ops.clamped_glu(self.gate_up(x), self.limit, self.alpha, self.up_offset))
 
 
+class ActivatedMLP(FeedForward):
+    """``down(act(up(x)))`` without gate and biases.  ``activation`` ``"xielu"``: with ``a = softplus(p)`` and ``b =
+    1/2 + softplus(q)`` of the two numbers in the tensor ``act``, ``act(z) = a z^2 + z / 2`` for ``z > 0`` and
+    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``, in fp32.
+
+    params: ``hidden_size``, ``intermediate_size``, ``activation``.  tensors: ``up``, ``down`` and, for
+    ``"xielu"``, ``act [2]``.
+    """
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.activation = str(self.param("activation"))
+        if self.activation not in ops.UNARY_ACT:
+            raise ValueError(f"unknown activation {self.activation!r}; known: {sorted(ops.UNARY_ACT)}")
+
+    def param_decls(self):
+        H, I = int(self.param("hidden_size")), int(self.param("intermediate_size"))
+        return {"up": ParamDecl((I, H)), "down": ParamDecl((H, I)), "act": ParamDecl((2,), "table")}
+
+    def bind(self, tensors, dtype, device):
+        self.up = _as_compute(tensors["up"], dtype).contiguous()
+        self.down = Linear(_as_compute(tensors["down"], dtype).contiguous())
+        p, q = (float(v) for v in torch.nn.functional.softplus(tensors["act"].to(torch.float64).cpu()))
+        self.act_params = (p, 0.5 + q)
+
+    def forward(self, x, ctx):
+        return self.down(ops.linear_activated(x, self.up, self.activation, self.act_params))
+
+
 # ----------------------------------------------------------------------------- embedding / head
 
 
@@ -675,15 +754,35 @@ class ParallelBlock(Arrangement):
 
 class BranchNormBlock(Arrangement):
     """``h += norm1(mixer(h)); h += norm2(ffn(h))``: both branches read the stream itself (its copy in
-    the compute dtype) and each norm, a ``BranchRMSNorm`` with the residual factor in it, stands behind
-    its branch.  The fp32 stream is updated in place; the block hands on a ``StreamCopy``.  A layer
-    without a feed-forward (``no_feed_forward``) is the mixer's half alone."""
+    the compute dtype) and each norm, a ``BranchRMSNorm`` or ``BranchLayerNorm`` with the residual factor or
+    the layer scale in it, stands behind its branch.  With a ``mixer_input`` the mixer reads that part's
+    output instead.  The fp32 stream is updated in place (an embedding's output that the model keeps stays as it is); the
+    block hands on a ``StreamCopy``, or, where the part behind it finishes branches, a ``PendingBranch``.
+    A layer without a feed-forward (``no_feed_forward``) is the mixer's half alone."""
 
-    def forward(self, x, residual, ctx, cache):
-        stream, h = stream_and_copy(x, residual, ctx.dtype)
-        h = self.mixer_norm.add_branch(stream, self.mixer.forward(h, ctx, cache, self.position))
-        if not isinstance(self.feed_forward, NoFeedForward):
-            h = self.feed_forward_norm.add_branch(stream, self.feed_forward.forward(h, ctx))
+    leaves_branch = True
+    takes_mixer_input = True
+
+    def forward(self, x, residual, ctx, cache, leave_branch=False):
+        if self.mixer_input is None:
+            stream, h = stream_and_copy(x, residual, ctx.dtype)
+        else:
+            stream = fp32_stream(x, residual)
+            h = x.prepared if isinstance(x, StreamCopy) else None
+            if h is None:
+                h = self.mixer_input.forward(stream, ctx, cache)
+        y = self.mixer.forward(h, ctx, cache, self.position)
+        keep = stream is ctx.scratch.get("embedded")
+        if isinstance(self.feed_forward, NoFeedForward):
+            if leave_branch:
+                return PendingBranch.of(self.mixer_norm, y), stream
+            stream, h = self.mixer_norm.add_branch(stream, y, keep=keep)
+            return StreamCopy.of(h), stream
+        stream, h = self.mixer_norm.add_branch(stream, y, keep=keep)
+        y = self.feed_forward.forward(h, ctx)
+        if leave_branch:
+            return PendingBranch.of(self.feed_forward_norm, y), stream
+        stream, h = self.feed_forward_norm.add_branch(stream, y)
         return StreamCopy.of(h), stream
 
 
@@ -739,6 +838,8 @@ register_norm("rmsnorm", RMSNorm, replace=True)
 register_norm("layernorm", LayerNorm, replace=True)
 register_norm("no_norm", NoNorm, replace=True)
 register_norm("branch_rmsnorm", BranchRMSNorm, replace=True)
+register_norm("branch_layernorm", BranchLayerNorm, replace=True)
+register_feed_forward("activated_mlp", ActivatedMLP, replace=True)
 register_arrangement("branch_norm", BranchNormBlock, replace=True)
 register_stream_part("token_side_input", TokenSideInput, replace=True)
 register_norm("same_norm", SameNorm, replace=True)

@@ -30,8 +30,9 @@ class RoutedExperts(FeedForward):
     params: ``hidden_size``, ``experts``, ``top``, ``expert_ff``, ``limit`` (with the clamped activation),
     optional ``alpha`` (default 1.702), ``shared_ff`` (0 or absent: no shared expert), ``shared_limit``,
     ``activation``, ``scores``, ``route_scale`` (default 1), ``groups``, ``keep_groups``, ``group_score``,
-    ``correction`` (default False) and ``shared_gate``.
-    tensors: ``router``, ``e{i}.gate``, ``e{i}.up``, ``e{i}.down``, with a correction ``correction`` and, with a
+    ``correction`` (default False), ``router_bias`` (default False: a bias per expert on the logits, fp32) and
+    ``shared_gate``.
+    tensors: ``router``, with its bias ``router.b``, ``e{i}.gate``, ``e{i}.up``, ``e{i}.down``, with a correction ``correction`` and, with a
     shared expert, ``shared.gate``, ``shared.up``, ``shared.down`` and, with its gate, ``shared.sg``.
     """
 
@@ -54,6 +55,7 @@ class RoutedExperts(FeedForward):
         self.correction = bool(g("correction", False))
         if self.correction and self.scores != "sigmoid":
             raise ValueError("a correction of the choice goes with sigmoid scores")
+        self.router_bias = bool(g("router_bias", False))
         self.group_score = str(g("group_score", "best"))
         if self.group_score not in ("best", "top2"):
             raise ValueError(f"unknown group_score {self.group_score!r}: 'best' or 'top2'")
@@ -77,6 +79,8 @@ class RoutedExperts(FeedForward):
     def param_decls(self):
         H, ff = self.hidden, self.ff
         decls = {"router": ParamDecl((self.experts, H))}
+        if self.router_bias:
+            decls["router.b"] = ParamDecl((self.experts,), "table")
         for e in range(self.experts):
             decls[f"e{e}.gate"] = ParamDecl((ff, H))
             decls[f"e{e}.up"] = ParamDecl((ff, H))
@@ -101,6 +105,7 @@ class RoutedExperts(FeedForward):
                 rows.append(torch.zeros((pad, self.hidden), dtype=self.router.dtype, device=self.router.device))
             self.router = torch.cat(rows).contiguous()
         self.choice_correction = tensors["correction"].to(torch.float32).contiguous() if self.correction else None
+        self.logit_bias = tensors["router.b"].to(torch.float32).contiguous() if self.router_bias else None
         # per expert its gate rows, then its up rows: one operand for a grouped product, two for the own kernels
         self.w_gate_up = torch.stack([torch.cat([_as_compute(tensors[f"e{e}.gate"], dtype),
                                                  _as_compute(tensors[f"e{e}.up"], dtype)]) for e in E]).contiguous()
@@ -125,7 +130,7 @@ class RoutedExperts(FeedForward):
         ids, weights, logits = ops.moe_route(x, self.router, self.top, scores=self.scores, groups=self.groups,
                                              keep_groups=self.keep_groups, scale=self.route_scale,
                                              correction=self.choice_correction, group_top2=self.group_score == "top2",
-                                             experts=self.experts, return_logits=True)
+                                             experts=self.experts, return_logits=True, bias=self.logit_bias)
         gate = logits[:, self.experts:self.experts + 1] if self.shared_gate else None
         return ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, self.limit, self.alpha, shared,
                                up_offset=self.up_offset, shared_gate=gate)

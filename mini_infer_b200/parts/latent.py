@@ -22,7 +22,7 @@ import torch
 from ..csrc import ops
 from .base import (KVNeed, LayerCache, ParamDecl, Part, PlanNeeds, StateNeed, StepContext, StreamPart, BranchSum,
                    register_embedding, register_mixer, register_stream_part)
-from .builtin import _as_compute
+from .builtin import Linear, _as_compute
 from .mixers import ProjectedMixer, _f32
 
 
@@ -42,14 +42,17 @@ class LatentAttention(ProjectedMixer):
     ``score_h(i, j) = (q_h,un(i) . W_uk,h c(j) + rotate(q_h,rot(i)) . r(j)) * scale``,
     ``out_h(i) = sum_j p_h(i, j) W_uv,h c(j)``, heads gated by ``sigmoid(W_g h)`` (``gate``), then ``W_o``.
 
-    The rotation is the half layout on the first ``rotary_dim`` of the ``rot_dim`` dimensions with base
-    ``theta``.  The cache holds ``[c, r]`` per token and nothing else; the kernel reads a key's value
+    The rotation is the half layout (``interleaved``: the pairs ``2i``, ``2i + 1``) on the first ``rotary_dim`` of the
+    ``rot_dim`` dimensions with base ``theta``.  With ``q_rank`` the queries go through a latent of their own,
+    ``q = W_uq (rmsnorm(W_dq h) * g_q)``, in the place of ``W_q h``.  With ``window`` position ``i`` sees ``j`` with ``0 <=
+    i - j < window``.  With ``gate_per_head`` the gate is one number per head.  The cache holds ``[c, r]`` per token and nothing else; the kernel reads a key's value
     from the key's own row.  Scores, softmax and sums are fp32 for either dtype.
 
     params: ``hidden_size``, ``num_heads``, ``head_dim``, ``rot_dim``, ``value_dim``, ``kv_rank``, ``theta``,
     ``rotary_dim``, ``scale``, ``eps``; optional ``sink`` (None, ``"learned"``, ``"zero"``), ``gate`` (None or
-    ``"sigmoid"`` / ``"silu"``).
-    tensors: ``q``, ``dkv``, ``dkv.norm``, ``uk``, ``uv``, ``o`` and, as asked, ``sink``, ``g``.
+    ``"sigmoid"`` / ``"silu"``), ``gate_per_head``, ``interleaved`` (default False), ``q_rank``, ``window``.
+    tensors: ``q`` (or, with ``q_rank``, ``dq``, ``dq.norm`` and ``uq``), ``dkv``, ``dkv.norm``, ``uk``, ``uv``, ``o`` and, as
+    asked, ``sink``, ``g``.
     """
 
     def __init__(self, spec):
@@ -71,34 +74,51 @@ class LatentAttention(ProjectedMixer):
             raise ValueError(f"{self.rot} rotated dimensions of a part of {self.rd}")
         if min(self.heads, self.d, self.dv, self.rank) <= 0 or self.rd < 0:
             raise ValueError("a latent attention needs positive sizes")
+        self.interleaved = bool(g("interleaved", False))
+        self.q_rank = int(g("q_rank") or 0)             # 0: the queries are projected from the input itself
+        self.window = int(g("window")) if g("window") else None
+        self.gate_width = 0 if not self.gate else (self.heads if g("gate_per_head") else self.heads * self.dv)
+        if self.q_rank < 0 or (self.window is not None and self.window <= 0):
+            raise ValueError(f"a query rank of {self.q_rank}, a window of {self.window}")
         self.qh = self.d + self.rd                      # a head's columns of the query projection
-        self.c_off = self.heads * self.qh
+        self.c_off = self.q_rank or self.heads * self.qh
         self.g_off = self.c_off + self.rank + self.rd
-        self.in_width = self.g_off + (self.heads * self.dv if self.gate else 0)
+        self.in_width = self.g_off + self.gate_width
         self.out_width = self.heads * self.dv
 
     def param_decls(self):
         H, n = self.hidden, self.heads
-        decls = {"q": ParamDecl((n * self.qh, H)), "dkv": ParamDecl((self.rank + self.rd, H)),
+        if self.q_rank:
+            decls = {"dq": ParamDecl((self.q_rank, H)), "dq.norm": ParamDecl((self.q_rank,), "gain"),
+                     "uq": ParamDecl((n * self.qh, self.q_rank))}
+        else:
+            decls = {"q": ParamDecl((n * self.qh, H))}
+        decls |= {"dkv": ParamDecl((self.rank + self.rd, H)),
                  "dkv.norm": ParamDecl((self.rank,), "gain"), "uk": ParamDecl((n * self.d, self.rank)),
                  "uv": ParamDecl((n * self.dv, self.rank)), "o": ParamDecl((H, n * self.dv))}
         if self.sink == "learned":
             decls["sink"] = ParamDecl((n,), "table")
         if self.gate:
-            decls["g"] = ParamDecl((n * self.dv, H))
+            decls["g"] = ParamDecl((self.gate_width, H))
         return decls
 
     def cache_need(self):
-        return KVNeed(1, self.rank + self.rd, None, 0)     # keys only: the latent is key and value
+        return KVNeed(1, self.rank + self.rd, self.window, 0)     # keys only: the latent is key and value
 
     def plan_needs(self):
         tiles = {ops.ATTENTION_TILE_TOKENS} | ops.rows_attention_tile_sizes(self.heads, 1, self.rank + self.rd, self.rank, True)
         return PlanNeeds(frozenset(tiles))
 
     def bind(self, tensors, dtype, device):
-        names = ["q", "dkv"] + (["g"] if self.gate else [])
-        self.w_in = torch.cat([_as_compute(tensors[n], dtype) for n in names], dim=0).contiguous()
+        names = ["dq" if self.q_rank else "q", "dkv"] + (["g"] if self.gate else [])
+        rows = [_as_compute(tensors[n], dtype) for n in names]
+        if self.q_rank and self.in_width % 8:      # rows of zeros up to a multiple of 8: the library's aligned products
+            rows.append(torch.zeros((-self.in_width % 8, self.hidden), dtype=dtype, device=device))
+            self.in_width += -self.in_width % 8
+        self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_out = _as_compute(tensors["o"], dtype).contiguous()
+        if self.q_rank:
+            self.uq, self.cq_gain = Linear(_as_compute(tensors["uq"], dtype).contiguous()), _f32(tensors["dq.norm"])
         n = self.heads
         # per head: W_uk^T [rank, head_dim] maps a query into the latent's space, W_uv [value_dim, rank]
         # expands a weighted sum of latents to the head's value
@@ -121,19 +141,31 @@ class LatentAttention(ProjectedMixer):
         M = ctx.n_tokens
         qfull = torch.empty((M, n, dk), dtype=proj.dtype, device=proj.device)
         group = ctx.groups[cache.group]
-        ops.latent_prepare(proj, 0, n, self.qh, self.d, self.c_off, rank, self.rd, self.rot,
-                           positions=ctx.positions, freq=self.freq, c_gain=self.c_gain, eps=self.eps, qfull=qfull,
-                           slots=group.slots if cache.writes else None, kcache=cache.k if cache.writes else None)
-        q_un = proj[:, :n * self.qh].unflatten(1, (n, self.qh))[:, :, :self.d]
+        common = dict(positions=ctx.positions, freq=self.freq, eps=self.eps, interleaved=self.interleaved)
+        row = dict(c_gain=self.c_gain, slots=group.slots if cache.writes else None,
+                   kcache=cache.k if cache.writes else None)
+        sizes = (self.c_off, rank, self.rd, self.rot)
+        if self.q_rank:
+            # the cache row and the queries' normed latent; then, from their product, the rotated query parts
+            cq = torch.empty((M, self.q_rank), dtype=proj.dtype, device=proj.device)
+            ops.latent_prepare(proj, 0, 0, self.qh, self.d, *sizes, qfull=None, cq_gain=self.cq_gain, cq_out=cq,
+                               **row, **common)
+            q = self.uq(cq)
+            ops.latent_prepare(q, 0, n, self.qh, self.d, *sizes, c_gain=None, qfull=qfull, **common)
+        else:
+            q = proj
+            ops.latent_prepare(proj, 0, n, self.qh, self.d, *sizes, qfull=qfull, **row, **common)
+        q_un = q[:, :n * self.qh].unflatten(1, (n, self.qh))[:, :, :self.d]
         ops.batched_linear(q_un, self.uk_t, qfull[:, :, :rank])
         latent = torch.empty((M, n * rank), dtype=proj.dtype, device=proj.device)
-        ops.attention_ext(qfull.view(M, n * dk), latent, cache, ctx, n, 1, dk, rank, self.scale, sinks=self.sinks,
-                          values_in_keys=True)
+        ops.attention_ext(qfull.view(M, n * dk), latent, cache, ctx, n, 1, dk, rank, self.scale,
+                          window=self.window or 0, sinks=self.sinks, values_in_keys=True)
         heads = torch.empty((M, n, self.dv), dtype=proj.dtype, device=proj.device)
         ops.batched_linear(latent.view(M, n, rank), self.uv, heads)
         heads = heads.view(M, n * self.dv)
         if self.gate:
-            ops.gate_mul(heads, proj[:, self.g_off:self.g_off + n * self.dv], out, self.gate, out_scale)
+            ops.gate_mul(heads, proj[:, self.g_off:self.g_off + self.gate_width], out, self.gate, out_scale,
+                         per=n * self.dv // self.gate_width)
         elif out_scale == 1.0:
             out.copy_(heads)
         else:

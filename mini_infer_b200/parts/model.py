@@ -59,6 +59,10 @@ class DecoderModel:
                 build_part("norm", layer.feed_forward_norm),
                 position,
             )
+            if layer.mixer_input is not None:
+                if not block.takes_mixer_input:
+                    raise ValueError(f"arrangement {layer.arrangement!r} runs no input part in front of its mixer")
+                block.mixer_input = build_part("input", layer.mixer_input)
             self.blocks.append(block)
         self.schedule = spec.schedule
         # stream parts that run before a schedule entry (None where an entry has none)
@@ -124,11 +128,21 @@ class DecoderModel:
                         f"{owner} does not fit its own {kv}"
                     )
         out = [needs[i] for i in range(self.spec.num_cache_layers)]
-        # an embedding that keeps something per request gets a state arena behind the cache layers'
+        # an embedding that keeps something per request gets a state arena behind the cache layers', and so
+        # does every run of a layer whose input part keeps something
         emb_state = getattr(self.embedding, "state_need", lambda: None)()
         if emb_state is not None:
             out.append(CacheLayerNeed(self.embedding_state_index, None, emb_state))
+        for i, e in enumerate(self.schedule):
+            part = self.blocks[e.layer].mixer_input
+            state = part.state_need() if part is not None else None
+            if state is not None:
+                out.append(CacheLayerNeed(self.input_state_index(i), None, state))
         return out
+
+    def input_state_index(self, entry: int) -> int:
+        """The index under which the cache manager keeps the state of the input part of schedule entry ``entry``."""
+        return self.spec.num_cache_layers + 1 + entry
 
     @property
     def embedding_state_index(self) -> int:
@@ -181,12 +195,16 @@ class DecoderModel:
         else:
             x = self.embedding.forward(ctx)
         embedded = x if self._keeps_embedding else None
+        if embedded is not None:
+            ctx.scratch["embedded"] = embedded      # a layer that updates its stream in place asks for it
         residual = None
         for i, (entry, cache) in enumerate(zip(self.schedule, caches)):
             if self.before[i] is not None:
                 x, residual = self.before[i].forward(x, residual, ctx, embedded)
-            block = self.blocks[entry.layer]
-            if block.entry() is None:
+            block, after = self.blocks[entry.layer], self.after[i]
+            if block.leaves_branch and after is not None and after.finishes_branch:
+                x, residual = block.forward(x, residual, ctx, cache, leave_branch=True)
+            elif block.entry() is None:
                 x, residual = block.forward(x, residual, ctx, cache)
             else:
                 # a layer that takes part in the hand-over of norms is told how the next one begins
@@ -195,8 +213,14 @@ class DecoderModel:
                 if i + 1 < len(self.schedule) and self.after[i] is None:
                     nxt = self.blocks[self.schedule[i + 1].layer].entry()
                 x, residual = block.forward(x, residual, ctx, cache, following=nxt)
-            if self.after[i] is not None:
-                x, residual = self.after[i].forward(x, residual, ctx, embedded)
+            if after is not None and after.prepares_input:
+                nxt = None
+                if i + 1 < len(self.schedule) and self.before[i + 1] is None:
+                    part = self.blocks[self.schedule[i + 1].layer].mixer_input
+                    nxt = None if part is None else (part, caches[i + 1])
+                x, residual = after.forward(x, residual, ctx, embedded, following=nxt)
+            elif after is not None:
+                x, residual = after.forward(x, residual, ctx, embedded)
         if n_want == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=ctx.device)
         z, _ = self.final_norm.forward(x, residual, rows=want_rows)

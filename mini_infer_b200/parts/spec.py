@@ -43,7 +43,8 @@ class LayerSpec:
 
     ``arrangement`` is a registered block-arrangement kind (where the norms and
     the residual additions stand).  ``position`` is the position encoding the
-    mixer applies (``None``: the mixer uses none).
+    mixer applies (``None``: the mixer uses none).  ``mixer_input``: a registered input part that
+    works on what the mixer reads, right before it (``None``: the mixer reads it as it is).
     """
 
     mixer: PartSpec
@@ -52,6 +53,7 @@ class LayerSpec:
     feed_forward_norm: PartSpec
     position: PartSpec | None = None
     arrangement: str = "prenorm"
+    mixer_input: PartSpec | None = None
 
 
 @dataclass(frozen=True)
