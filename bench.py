@@ -561,6 +561,101 @@ def run_ruburax_designs(args) -> int:
     return 0
 
 
+# The Zinesun architecture at the same widths: latent attention over a window with low-rank queries in every layer,
+# dense xIELU units and mixtures of experts alternating.  Beside it its closest model, Lilulix, with the same latent
+# attention (no window, full-rank queries, a gate per channel) in every layer and a gated unit with as many
+# parameters, and Llama with the same width, heads, layer count and feed-forward parameters.
+ZINESUN_SIZES = {
+    "2k": dict(q_rank=768, window=1024, dense_ff=8448, experts=32, top=4, ff=512),
+    "4k": dict(q_rank=1536, window=1024, dense_ff=16512, experts=64, top=4, ff=1024),
+}
+
+
+def zinesun_design(s: dict, z: dict, layers: int) -> tuple[dict, dict, dict]:
+    """(Zinesun, Lilulix, Llama) configurations."""
+    rot = {"base": 10000.0, "dims": s["rot_dim"]}
+    mixer = {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "kv_rank": s["kv_rank"],
+             "rot": rot, "scale": (s["dim"] + s["rot_dim"]) ** -0.5}
+    dense = {"kind": "dense", "ff": z["dense_ff"]}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["ff"]}}
+    raw = {"architecture": "Zinesun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "canon": {"taps": 3},
+           "embedding": {"scale": 1.0},
+           "layers": [{"type": "latent_attention", "mlp": moe if i % 2 else dense,
+                       "mixer": dict(mixer, q_rank=z["q_rank"], mask={"size": z["window"]})} for i in range(layers)]}
+    lilulix = {"architecture": "Lilulix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+               "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+               "layers": [{"type": "latent_attention", "mlp": {"kind": "dense", "ff": s["ff"]}, "mixer": mixer}] * layers}
+    llama = dict(LLAMA_8B, hidden_size=s["width"], num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"],
+                 head_dim=s["dim"], intermediate_size=s["ff"], vocab_size=s["vocab"], num_hidden_layers=layers)
+    return raw, lilulix, llama
+
+
+def zinesun_numbers(s: dict, z: dict, layers: int, batch: int, context: float, tokens: int) -> tuple[float, float]:
+    """(bytes a decode step must move, floating-point operations of a prefill of ``tokens``): weights once (of the
+    experts those that the batch's tokens choose in expectation), the cache rows of a window; products per token,
+    keys and values expanded from the latent once per token, the scores and sums inside the window."""
+    H, n, d, rd, dv, R = (s[k] for k in ("width", "heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    E, top, qr, W = z["experts"], z["top"], z["q_rank"], z["window"]
+    mix = H * (qr + R + rd + n) + qr * n * (d + rd) + n * (d + dv) * R + n * dv * H
+    hit = E * (1.0 - (1.0 - 1.0 / E) ** (batch * top))
+    n_moe = layers // 2
+    dense = (layers - n_moe) * 2 * H * z["dense_ff"]
+    experts = lambda used: n_moe * (H * E + used * 3 * H * z["ff"])
+    nbytes = 2.0 * (layers * mix + dense + experts(hit) + s["vocab"] * H) + 2.0 * layers * batch * min(W, context) * (R + rd)
+    w = min(W, tokens)
+    pairs = tokens * w - w * (w - 1) / 2.0
+    flops = 2.0 * tokens * (layers * mix + dense + experts(top)) + 2.0 * s["vocab"] * H \
+        + layers * 2.0 * pairs * n * (d + rd + dv)
+    return nbytes, flops
+
+
+def run_zinesun_designs(args) -> int:
+    import torch
+
+    from mini_infer_b200.engine import ModelRunner
+
+    peaks = load_peaks()
+    warmup = max(3, args.warmup)
+    out = {"scenario": "designs", "design": "zinesun", "dtype": "bf16", "data": "synthetic", "batch": args.batch,
+           "context": args.context, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks, "sizes": {}}
+    clocks = ClockSampler()
+    clocks.start()
+    for name in args.design_sizes.split(","):
+        s, z = LILULIX_SIZES[name], ZINESUN_SIZES[name]
+        layers = args.layers or 4
+        raw, lilulix, llama = zinesun_design(s, z, layers)
+        cap = args.batch * (args.context + args.steps + warmup + 64) + 2 * PREFILL_TOKENS
+        row = {"layers": layers}
+        for label, cfg in (("zinesun", raw), ("lilulix", lilulix), ("llama", llama)):
+            runner = ModelRunner.from_random(cfg, seed=0, gain_std=0.0, device="cuda:0", dtype="bfloat16",
+                                             num_blocks=cap // PAGE + 8, block_size=PAGE, max_requests=args.batch,
+                                             cuda_graph=True)
+            ms, launches = time_decode(runner, args.batch, args.context, args.steps, warmup)
+            pms = time_prefill(runner, PREFILL_TOKENS, repeats=3, warmup=2)
+            mid = args.context + warmup + args.steps / 2.0
+            if label == "zinesun":
+                nbytes, flops = zinesun_numbers(s, z, layers, args.batch, mid, PREFILL_TOKENS)
+            elif label == "lilulix":
+                nbytes, flops = lilulix_numbers(s, [0] * layers, args.batch, mid, PREFILL_TOKENS)
+            else:
+                flops = prefill_flops(cfg, layers, PREFILL_TOKENS)
+                nbytes = decode_bytes(cfg, layers, args.batch, mid)
+            row[label] = {
+                "decode_tok_s": round(args.batch * 1000.0 / ms, 1), "decode_ms": round(ms, 4),
+                "decode_gbs": round(nbytes / (ms * 1e-3) / 1e9, 1),
+                "decode_frac_of_hbm": round(nbytes / (ms * 1e-3) / 1e9 / peaks["hbm_gbs"], 4),
+                "prefill_tok_s": round(PREFILL_TOKENS * 1000.0 / pms, 1), "prefill_ms": round(pms, 3),
+                "prefill_frac_of_bf16": round(flops / (pms * 1e-3) / (peaks["bf16_tflops"] * 1e12), 4),
+                "launches_per_decode_step": launches // max(1, args.steps),
+            }
+            del runner
+            torch.cuda.empty_cache()
+        out["sizes"][name] = row
+    out["clocks"] = clocks.stop()
+    print(json.dumps(out))
+    return 0
+
+
 def run_vepevik_designs(args) -> int:
     import torch
 
@@ -1127,9 +1222,9 @@ def main() -> int:
                     help="decode: the contract line; long-mixed: many requests of very different lengths "
                          "through the scheduler (a line of its own); serving: the reference's published "
                          "workload, 1024 tokens in and 128 out, single requests and 16 together (a line of its own); "
-                         "designs: the Ruvurax (or, with --design, the Lilulix, the Vepevik or the Ruburax) architecture beside Llama at equal sizes, prefill and decode "
+                         "designs: the Ruvurax (or, with --design, the Lilulix, the Vepevik, the Ruburax or the Zinesun) architecture beside Llama at equal sizes, prefill and decode "
                          "(a line of its own)")
-    ap.add_argument("--design", default="ruvurax", choices=["ruvurax", "lilulix", "vepevik", "ruburax"],
+    ap.add_argument("--design", default="ruvurax", choices=["ruvurax", "lilulix", "vepevik", "ruburax", "zinesun"],
                     help="designs: which architecture stands beside Llama")
     ap.add_argument("--design-sizes", default="2k,4k", help="designs: which of the sizes " + ",".join(DESIGN_SIZES))
     ap.add_argument("--requests", type=int, default=64, help="long-mixed: requests started together")
@@ -1163,6 +1258,8 @@ def main() -> int:
             return run_vepevik_designs(args)
         if args.design == "ruburax":
             return run_ruburax_designs(args)
+        if args.design == "zinesun":
+            return run_zinesun_designs(args)
         return run_lilulix_designs(args) if args.design == "lilulix" else run_designs(args)
     warmup = max(3, args.warmup)
 
