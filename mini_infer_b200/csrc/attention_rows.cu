@@ -25,7 +25,8 @@
 //
 // Layouts as in attention_generic.cu: q [tokens, q_stride], out [tokens, out_stride], kcache
 // [pages, nkv, page_size, d], vcache [pages, nkv, page_size, dv] (null with v_prefix), block tables
-// and the per-request lists of a step; tile_req / tile_tok0 list tiles of `tile_tokens` tokens.
+// and the per-request lists of a step; tile_req / tile_tok0 list tiles of `tile_tokens` tokens (null: a
+// tile per request, from its first token; a null q_len: one token per request).
 #include "common.cuh"
 
 MI_DEFINE_ERROR_API()
@@ -152,8 +153,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   bid /= head_tiles;
   const int kvh = bid % nkv;
   const int tile = bid / nkv;
-  const int b = tile_req[tile], tok0 = tile_tok0[tile];
-  const int ql = q_len[b], kl = kv_len[b], qs = q_start[b];
+  const int b = tile_req ? tile_req[tile] : tile, tok0 = tile_req ? tile_tok0[tile] : 0;
+  const int ql = q_len ? q_len[b] : 1, kl = kv_len[b], qs = q_start[b];
   const int trow = table_rows ? table_rows[b] : b;
   const int nt = min(tile_tokens, ql - tok0);                   // tokens of this tile
   const int p0 = kl - ql + tok0;                                // position of the tile's first token
@@ -414,8 +415,8 @@ attention_rows_merge_kernel(const float* __restrict__ part_o, const float* __res
   const int kvh = bid % nkv;
   const int tile = bid / nkv;
   const RowMap rows{G, R, kvh, hs};
-  const int b = tile_req[tile], tok0 = tile_tok0[tile];
-  const int nt = min(tile_tokens, q_len[b] - tok0);
+  const int b = tile_req ? tile_req[tile] : tile, tok0 = tile_req ? tile_tok0[tile] : 0;
+  const int nt = min(tile_tokens, (q_len ? q_len[b] : 1) - tok0);
   if (rows.token(r) >= nt) return;
   const int head = rows.head(r);
   const float* pml = part_ml + ((size_t)unit * n_splits * R + r) * 2;

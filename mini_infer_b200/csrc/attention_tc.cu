@@ -619,6 +619,303 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   }
 }
 
+// ------------------------------------------------------------------------------------- expanded latent rows
+//
+// The same kernel for attention whose keys and values have been expanded from cached latents into
+// contiguous rows for this step (latent_gather in qk_prepare.cu, then one library product): row y of
+// `kv` [rows, n dn + n dv] holds every head's key part (dn numbers each), then every head's value
+// (dv each); row y of `lat` holds, from column r_col on, 64 columns of the key part that all heads
+// share (rd of them, then zeros).  A request's rows start at e_start[b] and stand for its positions
+// from e_first[b] on, a multiple of 64; they are whole chunks, and every row is finite.  One block
+// takes 128 tokens of one head (TMEM lane = token), its keys in chunks of 64: TMA box copies of
+// [64 rows x 64 columns] with the 128-byte swizzle.  A head's query is [dn, rd] at column
+// h (dn + rd) of q; query columns that do not exist are zero, so what a box brings beyond a head's
+// own columns does not count.  `gate` (optional): head h's output row is multiplied by
+// sigmoid(gate[token, h]).  Registers, tensor memory and the roles of the warps as above; kst / vst:
+// stages of the key and the value ring.
+#define BOX_BYTES (KC * 128)     // 64 keys x 64 columns
+#define XB_KFULL 0
+#define XB_VFULL 2
+#define XB_KEMPTY 4
+#define XB_VEMPTY 6
+#define XB_SFULL 8
+#define XB_PFULL 10
+#define XB_PVDONE 12
+#define XB_COUNT 14
+#define XTM_COLS 256             // two score buffers of 64 columns, then O of 128
+#define XTM_O 128
+
+__global__ void __launch_bounds__(256, 2)
+attention_expanded_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_lat,
+                             const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
+                             const int* __restrict__ e_start, const int* __restrict__ e_first,
+                             const int* __restrict__ q_start, const int* __restrict__ q_len,
+                             const int* __restrict__ kv_len, const int* __restrict__ tile_req,
+                             const int* __restrict__ tile_tok0, int n, int dn, int rd, int dv, int r_col, float scale,
+                             int window, const float* __restrict__ sinks, const bf16* __restrict__ gate,
+                             int gate_stride, int kst, int vst) {
+  mi_pdl_enter();
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
+  unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  const int kb = (dn + 63) >> 6, qb = kb + (rd > 0 ? 1 : 0), vb = (dv + 63) >> 6;   // boxes per row: own key part, key, value
+  unsigned char* Qs = smem;                                  // [qb][128 rows][128 B]
+  unsigned char* Ks = Qs + qb * (ROWS * 128);                // [kst][qb][64 keys][128 B]
+  unsigned char* Vs = Ks + kst * qb * BOX_BYTES;             // [vst][vb][64 keys][128 B]
+  __shared__ __align__(8) uint64_t bars[XB_COUNT];
+  __shared__ uint32_t tmem_base_holder;
+  __shared__ int give_up;
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tile = blockIdx.x / n, h = blockIdx.x - tile * n;
+  const int b = tile_req[tile], tok0 = tile_tok0[tile];
+  const int ql = q_len[b], kl = kv_len[b], qs = q_start[b];
+  const int ntok = min(ROWS, ql - tok0);
+  const int p_first = kl - ql + tok0;
+  const int hi = p_first + ntok;
+  const int lo = window > 0 ? max(0, p_first - window + 1) : 0;
+  const int c0 = lo / KC, c1 = (hi + KC - 1) / KC, n_chunks = c1 - c0;
+  volatile int* gu = &give_up;
+
+  if (tid == 0) {
+    for (int i = 0; i < XB_COUNT; ++i) mbar_init(&bars[i], (i >= XB_PFULL && i < XB_PVDONE) ? 4 : 1);
+    give_up = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  if (warp == 5) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(&tmem_base_holder)),
+                 "r"(XTM_COLS)
+                 : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
+  }
+  // the query tile: thread (row, half of the 16-byte pieces); pieces behind the head's part are zero
+  {
+    const int r = tid >> 1;
+    const bool there = r < ntok;
+    const bf16* src = q + (size_t)(qs + tok0 + (there ? r : 0)) * q_stride + (size_t)h * (dn + rd);
+    for (int u0 = tid & 1; u0 < qb * 8; u0 += 8) {           // four pieces in flight
+      uint4 v[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int u = u0 + 2 * k, box = u >> 3, c = (u & 7) * 8;
+        const int col = box < kb ? box * 64 + c : dn + c;    // of the head's query
+        const bool in = u < qb * 8 && there && (box < kb ? box * 64 + c < dn : c < rd);
+        v[k] = in ? *reinterpret_cast<const uint4*>(src + col) : make_uint4(0u, 0u, 0u, 0u);
+      }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int u = u0 + 2 * k, box = u >> 3, c = u & 7;
+        if (u < qb * 8) *reinterpret_cast<uint4*>(Qs + box * (ROWS * 128) + r * 128 + ((c ^ (r & 7)) << 4)) = v[k];
+      }
+    }
+    fence_async_smem();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_holder;
+
+  if (warp == 4 || warp == 6) {
+    // the copy threads, one for keys and one for values
+    REGS_GIVE();
+    if (lane == 0) {
+      const bool is_v = warp == 6;
+      const int y0 = e_start[b] - e_first[b];
+      const int boxes = is_v ? vb : qb, stages = is_v ? vst : kst;
+      const int full0 = is_v ? XB_VFULL : XB_KFULL, empty0 = is_v ? XB_VEMPTY : XB_KEMPTY;
+      unsigned char* ring = is_v ? Vs : Ks;
+      for (int it = 0; it < n_chunks; ++it) {
+        const int st = it % stages, round = it / stages;
+        if (round > 0 && !mbar_wait(&bars[empty0 + st], (round - 1) & 1, gu)) break;
+        mbar_expect_tx(&bars[full0 + st], (uint32_t)boxes * BOX_BYTES);
+        const int y = y0 + (c0 + it) * KC;
+        for (int j = 0; j < boxes; ++j) {
+          void* dst = ring + (st * boxes + j) * BOX_BYTES;
+          if (is_v) tma_load_2d(dst, &map_kv, n * dn + h * dv + j * 64, y, &bars[full0 + st]);
+          else if (j < kb) tma_load_2d(dst, &map_kv, h * dn + j * 64, y, &bars[full0 + st]);
+          else tma_load_2d(dst, &map_lat, r_col, y, &bars[full0 + st]);
+        }
+      }
+    }
+  } else if (warp == 5) {
+    // S = Q K^T of one chunk after the other
+    REGS_GIVE();
+    if (lane == 0) {
+      const uint32_t idesc_qk = idesc_bf16(ROWS, KC, 0);
+      const uint64_t qd = desc_sw128(smem_u32(Qs), 0), k_desc = desc_sw128(smem_u32(Ks), 0);
+      for (int it = 0; it < n_chunks; ++it) {
+        const int st = it % kst, round = it / kst, sb = it & 1, sround = it >> 1;
+        if (!mbar_wait(&bars[XB_KFULL + st], round & 1, gu)) break;
+        if (sround > 0 && !mbar_wait(&bars[XB_PVDONE + sb], (sround - 1) & 1, gu)) break;
+        tc_fence_after();
+        const uint64_t kd = k_desc + ((st * qb * BOX_BYTES) >> 4);
+        for (int j = 0; j < qb; ++j) {
+          const int steps = min(4, ((j < kb ? dn - j * 64 : rd) + 15) >> 4);
+          for (int k = 0; k < steps; ++k)
+            umma(tmem + sb * KC, qd + ((j * (ROWS * 128) + k * 32) >> 4), kd + ((j * BOX_BYTES + k * 32) >> 4), idesc_qk,
+                 (j | k) ? 1u : 0u);
+        }
+        umma_commit(&bars[XB_SFULL + sb]);
+        umma_commit(&bars[XB_KEMPTY + st]);
+      }
+    }
+  } else if (warp == 7) {
+    // O += P V
+    REGS_GIVE();
+    if (lane == 0) {
+      const uint32_t idesc_pv = idesc_bf16(ROWS, dv, 1);
+      const uint64_t v_desc = desc_sw128(smem_u32(Vs), BOX_BYTES);
+      for (int it = 0; it < n_chunks; ++it) {
+        const int st = it % vst, round = it / vst, sb = it & 1, sround = it >> 1;
+        if (!mbar_wait(&bars[XB_VFULL + st], round & 1, gu)) break;
+        if (!mbar_wait(&bars[XB_PFULL + sb], sround & 1, gu)) break;
+        tc_fence_after();
+        const uint64_t vd = v_desc + ((st * vb * BOX_BYTES) >> 4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          umma_ts(tmem + XTM_O, tmem + sb * KC + k * 8, vd + ((k * 2048) >> 4), idesc_pv, (it > 0 || k > 0) ? 1u : 0u);
+        umma_commit(&bars[XB_PVDONE + sb]);
+        umma_commit(&bars[XB_VEMPTY + st]);
+      }
+    }
+  } else {
+    // softmax, one token per thread (see attention_prefill_tc_kernel for how the reference moves)
+    REGS_TAKE();
+    const int r = tid;
+    const bool rvalid = r < ntok;
+    const int prow = p_first + r;
+    const int lorow = window > 0 ? max(0, prow - window + 1) : 0;
+    const int last_lo = window > 0 ? max(0, hi - window) : 0;       // the last row's bound, the highest of the block
+    const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
+    const uint32_t tmem_o = tmem + XTM_O;
+    const float sc = scale * LOG2E;
+    float m_run = -INFINITY, l_run = 0.f;
+    bool ok = true;
+    for (int it = 0; it < n_chunks; ++it) {
+      const int sb = it & 1, sround = it >> 1, key0 = (c0 + it) * KC;
+      if (!warp_wait(&bars[XB_SFULL + sb], sround & 1, gu)) { ok = false; break; }
+      tc_fence_after();
+      float s[64];
+      {
+        uint32_t ra[32], rb[32];
+        tmem_ld32_issue(tmem + lane_addr + sb * KC, ra);
+        tmem_ld32_issue(tmem + lane_addr + sb * KC + 32, rb);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          s[i] = __uint_as_float(ra[i]);
+          s[32 + i] = __uint_as_float(rb[i]);
+        }
+      }
+      const bool interior = key0 + KC - 1 <= p_first && key0 >= last_lo;
+      if (!interior || !rvalid) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j)
+          if (!(rvalid && key0 + j <= prow && key0 + j >= lorow)) s[j] = -INFINITY;
+      }
+      const uint64_t sc2 = pair_of(sc, sc);
+      uint32_t pk[32];
+      float sum = 0.f, mx4[4];
+      const bool ahead = __all_sync(0xffffffffu, m_run != -INFINITY);
+      if (ahead) {
+        const uint64_t mneg2 = pair_of(-m_run, -m_run);
+        uint64_t acc[2] = {pair_of(0.f, 0.f), pair_of(0.f, 0.f)};
+#pragma unroll
+        for (int j = 0; j < 64; j += 2) {
+          float x0, x1;
+          unpair(fma2(pair_of(s[j], s[j + 1]), sc2, mneg2), x0, x1);
+          const float p0 = fast_exp2(x0), p1 = fast_exp2(x1);
+          acc[(j >> 1) & 1] = add2(acc[(j >> 1) & 1], pair_of(p0, p1));
+          pk[j >> 1] = pack_bf16(p0, p1);
+          mx4[j >> 4] = (j & 15) ? max3(mx4[j >> 4], s[j], s[j + 1]) : fmaxf(s[j], s[j + 1]);
+        }
+        float a0, a1;
+        unpair(add2(acc[0], acc[1]), a0, a1);
+        sum = a0 + a1;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 64; j += 2)
+          mx4[j >> 4] = (j & 15) ? max3(mx4[j >> 4], s[j], s[j + 1]) : fmaxf(s[j], s[j + 1]);
+      }
+      const float mx = fmaxf(max3(mx4[0], mx4[1], mx4[2]), mx4[3]) * sc;
+      const bool moved = __any_sync(0xffffffffu, mx > m_run + RESCALE_LOG2);
+      const float m_new = moved ? fmaxf(m_run, mx) : m_run;
+      float alpha = 1.f;
+      if (!ahead || moved) {
+        sum = 0.f;
+        if (m_new != -INFINITY) {
+          alpha = fast_exp2(m_run - m_new);
+          const uint64_t mneg2 = pair_of(-m_new, -m_new);
+          uint64_t acc[2] = {pair_of(0.f, 0.f), pair_of(0.f, 0.f)};
+#pragma unroll
+          for (int j = 0; j < 64; j += 2) {
+            float x0, x1;
+            unpair(fma2(pair_of(s[j], s[j + 1]), sc2, mneg2), x0, x1);
+            const float p0 = fast_exp2(x0), p1 = fast_exp2(x1);
+            acc[(j >> 1) & 1] = add2(acc[(j >> 1) & 1], pair_of(p0, p1));
+            pk[j >> 1] = pack_bf16(p0, p1);
+          }
+          float a0, a1;
+          unpair(add2(acc[0], acc[1]), a0, a1);
+          sum = a0 + a1;
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) pk[j] = 0u;
+        }
+      }
+      m_run = m_new;
+      l_run = l_run * alpha + sum;
+      if (it > 0 && moved) {
+        if (!warp_wait(&bars[XB_PVDONE + (sb ^ 1)], ((it - 1) >> 1) & 1, gu)) { ok = false; break; }
+        tc_fence_after();
+        for (int c32 = 0; c32 < dv; c32 += 32) {
+          float o32[32];
+          tmem_ld32(tmem_o + lane_addr + c32, o32);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o32[i] *= alpha;
+          tmem_st32(tmem_o + lane_addr + c32, o32);
+        }
+        tmem_st_wait();
+      }
+      tmem_st32_bits(tmem + lane_addr + sb * KC, pk);
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars[XB_PFULL + sb]);
+    }
+    if (ok && n_chunks > 0 && warp_wait(&bars[XB_PVDONE + ((n_chunks - 1) & 1)], ((n_chunks - 1) >> 1) & 1, gu)) {
+      tc_fence_after();
+      if (sinks && rvalid && m_run != -INFINITY) l_run += fast_exp2(sinks[h] * LOG2E - m_run);
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      const int row = qs + tok0 + (rvalid ? r : 0);
+      if (gate) inv *= 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)row * gate_stride + h])));
+      bf16* orow = out + (size_t)row * out_stride + (size_t)h * dv;
+      for (int c32 = 0; c32 < dv; c32 += 32) {
+        float o32[32];
+        tmem_ld32(tmem_o + lane_addr + c32, o32);   // every thread of the warp takes part in the load
+        if (rvalid) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            if (c32 + i < dv) {
+              uint4 v;
+              v.x = pack_bf16(o32[i] * inv, o32[i + 1] * inv);
+              v.y = pack_bf16(o32[i + 2] * inv, o32[i + 3] * inv);
+              v.z = pack_bf16(o32[i + 4] * inv, o32[i + 5] * inv);
+              v.w = pack_bf16(o32[i + 6] * inv, o32[i + 7] * inv);
+              *reinterpret_cast<uint4*>(orow + c32 + i) = v;
+            }
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 5) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem_base_holder), "r"(XTM_COLS) : "memory");
+  }
+}
+
 // ------------------------------------------------------------------------------------- host
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
@@ -755,4 +1052,63 @@ extern "C" int mi_attention_prefill_tc(const void* q, int q_stride, void* out, i
   return mi_attention_prefill_tc_ext(q, q_stride, out, out_stride, kcache, vcache, n_pages, block_table, bt_stride,
                                      table_rows, page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles,
                                      tile_tokens, nq, nkv, d, scale, window, nullptr, nullptr, stream);
+}
+
+// rows [rows, cols] bf16 read in boxes of 64 rows x 64 columns with the 128-byte swizzle
+static bool make_rows_map(CUtensorMap* map, const void* base, long long rows, long long cols) {
+  EncodeTiledFn fn = encode_fn();
+  if (!fn) return false;
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  cuuint32_t box[2] = {64, KC};
+  cuuint32_t estr[2] = {1, 1};
+  return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+#define EXPANDED_SMEM_PAIR (112 * 1024)   // of dynamic shared memory, so that two blocks share an SM
+
+// 1 if the kernel on expanded latent rows takes these sizes
+extern "C" int mi_attention_expanded_supported(int n, int dn, int rd, int dv) {
+  return n > 0 && n <= 65535 && dn >= 8 && dn <= 128 && dn % 8 == 0 && rd >= 0 && rd <= 64 && rd % 8 == 0 && dv >= 16 &&
+         dv <= 128 && dv % 16 == 0;
+}
+
+// Tokens per tile of that kernel (a block takes the tile for one head).
+extern "C" int mi_attention_expanded_tile_tokens() { return ROWS; }
+
+extern "C" int mi_attention_expanded(const void* q, int q_stride, void* out, int out_stride, const void* kv,
+                                     const void* lat, int lat_cols, int r_col, long long rows, const int* e_start,
+                                     const int* e_first, const int* q_start, const int* q_len, const int* kv_len,
+                                     const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens, int n,
+                                     int dn, int rd, int dv, float scale, int window, const float* sinks,
+                                     const void* gate, int gate_stride, cudaStream_t stream) {
+  if (n_tiles <= 0) return 0;
+  if (!mi_attention_expanded_supported(n, dn, rd, dv))
+    MI_REFUSE("attention_expanded: sizes not taken (%d heads, keys of %d + %d, values of %d)", n, dn, rd, dv);
+  if (tile_tokens != ROWS) MI_REFUSE("attention_expanded: tiles of %d tokens, the kernel wants %d", tile_tokens, ROWS);
+  if (!(scale > 0.f) || window < 0) MI_REFUSE("attention_expanded: the scale must be positive and the window not negative");
+  if (rows <= 0 || rows % KC) MI_REFUSE("attention_expanded: %lld expanded rows are no whole chunks", rows);
+  if (lat_cols % 8 || r_col % 8 || r_col + 64 > lat_cols) MI_REFUSE("attention_expanded: columns %d to %d of latent rows of %d", r_col, r_col + 64, lat_cols);
+  if (!mi_aligned(q, 16) || q_stride % 8 || (dn + rd) % 8 || !mi_aligned(out, 16) || out_stride % 8 || !mi_aligned(kv, 16) ||
+      !mi_aligned(lat, 16))
+    MI_REFUSE("attention_expanded: rows must be 16-byte aligned");
+  const int kb = (dn + 63) / 64, qb = kb + (rd > 0 ? 1 : 0), vb = (dv + 63) / 64;
+  const size_t q_bytes = (size_t)qb * ROWS * 128, k_bytes = (size_t)qb * BOX_BYTES, v_bytes = (size_t)vb * BOX_BYTES;
+  int kst = 2, vst = 2;
+  if (q_bytes + kst * k_bytes + vst * v_bytes + 1024 > EXPANDED_SMEM_PAIR) kst = 1;
+  const size_t smem = q_bytes + kst * k_bytes + vst * v_bytes + 1024;
+  CUtensorMap map_kv, map_lat;
+  if (!make_rows_map(&map_kv, kv, rows, (long long)n * (dn + dv)) || !make_rows_map(&map_lat, lat, rows, lat_cols))
+    MI_REFUSE("attention_expanded: the driver refused a tensor map");
+  auto kern = attention_expanded_tc_kernel;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  const long long n_blocks = (long long)n_tiles * n;
+  if (n_blocks > 0x7fffffffLL) MI_REFUSE("attention_expanded: too many blocks for one launch");
+  MI_LAUNCH((kern), (unsigned)n_blocks, 256, smem, stream, map_kv, map_lat, (const bf16*)q, q_stride, (bf16*)out, out_stride,
+            e_start, e_first, q_start, q_len, kv_len, tile_req, tile_tok0, n, dn, rd, dv, r_col, scale, window, sinks,
+            (const bf16*)gate, gate_stride, kst, vst);
+  MI_RETURN_LAUNCH_STATUS();
 }

@@ -219,6 +219,14 @@ def _sig_attention_tc(lib: ctypes.CDLL) -> None:
     lib.mi_attention_prefill_tc_supported.argtypes = [c_int, c_int, c_int, c_int]
     lib.mi_attention_tc_status.argtypes = [c_int]
     lib.mi_set_status_word.argtypes = [c_void_p]
+    _sig_expanded(lib)
+
+
+def _sig_expanded(lib: ctypes.CDLL) -> None:
+    lib.mi_attention_expanded.argtypes = [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, ctypes.c_longlong, c_void_p, c_void_p, c_void_p,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+        c_int, c_void_p]
 
 
 def _sig_layernorm(lib: ctypes.CDLL) -> None:
@@ -320,6 +328,10 @@ def _sig_qk_prepare(lib: ctypes.CDLL) -> None:
                                           c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_float, c_float,
                                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                           c_void_p, c_int, c_void_p, c_int, c_void_p]
+
+
+    lib.mi_latent_gather.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                     c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p]
 
 
 def _sig_attention_rows(lib: ctypes.CDLL) -> None:
@@ -2200,6 +2212,26 @@ def latent_prepare(packed: torch.Tensor, q_off: int, nq: int, q_head: int, q_rot
     _finish(lib, rc, "latent_prepare")
 
 
+def latent_rotate_queries(q: torch.Tensor, nq: int, q_head: int, rot_off: int, rot_dim: int, rot: int, *,
+                          positions: torch.Tensor, freq: torch.Tensor, interleaved: bool) -> None:
+    """Rotates, in place, the part at ``rot_off`` of every head (``q_head`` columns) of ``q [M, nq * q_head]`` as
+    ``latent_prepare`` does."""
+    if not rot:
+        return
+    _cuda(q, positions, freq)
+    _cols(q, "latent_prepare")
+    M = q.shape[0]
+    if q.shape[1] != nq * q_head or positions.dtype != torch.int32 or positions.shape != (M,):
+        raise KernelError("latent_prepare: q must be [M, heads * head columns], positions int32 [M]")
+    if freq.dtype != torch.float64 or freq.shape != (rot // 2,) or not freq.is_contiguous():
+        raise KernelError("latent_prepare: freq must be float64 [rot / 2]")
+    lib = _lib("qk_prepare")
+    rc = lib.mi_latent_prepare(_ptr(q), q.stride(0), 0, M, nq, q_head, rot_off, 0, rot_off, rot_dim, int(rot),
+                               _ptr(positions), _ptr(freq), None, 0.0, _ptr(q), q.stride(0), q_head, None, None, 0, 0,
+                               1 if interleaved else 0, 0, 0, None, None, _code(q.dtype), _stream())
+    _finish(lib, rc, "latent_prepare")
+
+
 USE_ROWS_ATTENTION = os.environ.get("MINI_INFER_ROWS_ATTENTION", "1") != "0"
 ROWS_ATTENTION_ROWS = (16, 32, 64)   # query rows per block of attention_rows.cu: steps of single tokens; prompt portions
 
@@ -2258,11 +2290,15 @@ def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys
         return 16, rows_attention_tile_tokens(group, 16), 1, 1
     tt = rows_attention_tile_tokens(group, 16)
     units = ctx.tiles[tt][2] * nkv * max(1, -(-group // 16))
+    return 16, tt, _rows_attention_runs(ctx, units, window, device), 1
+
+
+def _rows_attention_runs(ctx, units: int, window: int, device) -> int:
+    """Runs of keys per tile in a step of ``units`` tiles of single tokens, so that the blocks fill the GPU."""
     chunks = max(1, -(-int(getattr(ctx, "max_kv_len", 0) or 64) // 64))
     if window:                       # the keys of one window touch at most this many chunks
         chunks = min(chunks, -(-(window - 1) // 64) + 1)
-    splits = max(1, min(-(-4 * _sms(device) // units), chunks, 64))
-    return 16, tt, splits, 1
+    return max(1, min(-(-4 * _sms(device) // units), chunks, 64))
 
 
 def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: int, d: int, dv: int, scale: float, *,
@@ -2335,6 +2371,116 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
         _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len),
         _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), nq, nkv, d, dv, float(scale), int(window), int(chunk),
         _ptr(sinks), _ptr(slopes), 1 if values_in_keys else 0, _code(q.dtype), _stream())
+    _finish(lib, rc, "attention")
+
+
+def attention_latent_singles(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, d: int, dv: int, scale: float, *,
+                             window: int = 0, sinks: torch.Tensor | None = None) -> None:
+    """``attention_ext`` with ``values_in_keys`` for the requests of a mixed step that bring one token, alone: the
+    tensor-core kernel with every request's keys cut into runs.  Only their rows of ``out`` are written."""
+    global launch_count
+    group = ctx.groups[cache.group]
+    kc, bt = cache.k, group.block_table
+    _cuda(q, out, kc)
+    if (q.dtype != torch.bfloat16 or not rows_attention_supported(nq, 1, d, dv, True) or kc.dtype != q.dtype
+            or kc.shape[1:] != (1, group.page_size, d) or not kc.is_contiguous() or not ctx.n_single):
+        raise KernelError("attention: single tokens of a mixed step need bfloat16 rows that attention_rows takes")
+    _opt_f32(sinks, nq, "attention (sinks)")
+    units = ctx.n_single * max(1, -(-nq // 16))
+    splits = _rows_attention_runs(ctx, units, int(window), q.device)
+    part_o = part_ml = None
+    if splits > 1:
+        part_o = torch.empty(units * splits * 16 * dv, dtype=torch.float32, device=q.device)
+        part_ml = torch.empty(units * splits * 16 * 2, dtype=torch.float32, device=q.device)
+    lib = _lib("attention_rows")
+    rc = lib.mi_attention_rows(
+        _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), None, _ptr(bt), bt.stride(0), _ptr(ctx.single_rows),
+        int(group.page_size), _ptr(ctx.single_q_start), None, _ptr(ctx.single_kv_len), None, None, int(ctx.n_single),
+        rows_attention_tile_tokens(nq, 16), 16, nq, 1, d, dv, float(scale), _ptr(sinks), None, 1, splits, _ptr(part_o),
+        _ptr(part_ml), 1, int(window), _stream())
+    _finish(lib, rc, "attention")
+    if splits > 1:
+        launch_count += 1
+
+
+# --------------------------------------------------------------------------------------- prompt portions over expanded latents
+
+
+USE_EXPANDED_LATENT = os.environ.get("MINI_INFER_EXPANDED_LATENT", "1") != "0"
+EXPANDED_TILE_TOKENS = 128     # the kernel's mi_attention_expanded_tile_tokens()
+EXPANDED_MIN_TOKENS = 32       # prompt tokens of a step from which expanding the keys pays
+
+
+def expanded_latent_supported(n: int, dn: int, rd: int, dv: int, rank: int) -> bool:
+    """Whether the tcgen05 kernel on expanded latent rows takes these sizes (the library's
+    ``mi_attention_expanded_supported``, made here so that a model it does not take never compiles it)."""
+    return (USE_EXPANDED_LATENT and 0 < n <= 65535 and 8 <= dn <= 128 and dn % 8 == 0 and 0 <= rd <= 64 and rd % 8 == 0
+            and 16 <= dv <= 128 and dv % 16 == 0 and rank % 8 == 0)
+
+
+class ExpandedRows:
+    """The cached latent rows that a step's prompt portions see, side by side (``latent_gather``)."""
+
+    __slots__ = ("rows", "start", "first", "rank")
+
+    def __init__(self, rows, start, first, rank):
+        self.rows, self.start, self.first, self.rank = rows, start, first, rank
+
+
+def latent_gather(cache, ctx, rank: int, rot_dim: int, window: int = 0) -> ExpandedRows:
+    """The cache rows ``[latent, shared key part]`` of every position that this step's portions of more than one
+    token see, one request after the other, each from a multiple of 64 positions on and a multiple of 64 rows
+    long (rows of zeros where nobody sees anything), the shared part padded with zeros to 64 columns."""
+    group = ctx.groups[cache.group]
+    kc, bt = cache.k, group.block_table
+    _cuda(kc, bt)
+    width = rank + rot_dim
+    if kc.dtype != torch.bfloat16 or kc.shape[1:] != (1, group.page_size, width) or not kc.is_contiguous():
+        raise KernelError("latent_gather: the cache must be contiguous bfloat16 [pages, 1, page_size, rank + rot_dim]")
+    total = longest = 0
+    for n, kl in zip(ctx.host_q_len, ctx.host_kv_len):
+        if n == 1:
+            continue
+        lo = max(0, kl - n - window + 1) if window else 0
+        count = -(-(kl - lo // 64 * 64) // 64) * 64
+        total, longest = total + count, max(longest, count)
+    rows = torch.empty((total, rank + 64), dtype=kc.dtype, device=kc.device)
+    where = torch.empty((2, ctx.n_requests), dtype=torch.int32, device=kc.device)
+    lib = _lib("qk_prepare")
+    rc = lib.mi_latent_gather(_ptr(kc), _ptr(bt), bt.stride(0), _ptr(group.table_rows), int(group.page_size),
+                              _ptr(ctx.q_len), _ptr(ctx.kv_len), ctx.n_requests, longest, int(window), 1, width, _ptr(rows),
+                              rank + 64, _ptr(where[0]), _ptr(where[1]), _code(kc.dtype), _stream())
+    _finish(lib, rc, "latent_gather")
+    return ExpandedRows(rows, where[0], where[1], rank)
+
+
+def attention_expanded(q: torch.Tensor, out: torch.Tensor, lat: ExpandedRows, w_kv: torch.Tensor, ctx, n: int, dn: int,
+                       rd: int, dv: int, scale: float, *, window: int = 0, sinks: torch.Tensor | None = None,
+                       gate: torch.Tensor | None = None) -> None:
+    """Attention of this step's prompt portions (requests of more than one token) over gathered latent rows:
+    ``w_kv [n dn + n dv, rank]`` (every head's key expansion, then every head's value expansion) is multiplied
+    with the latents once (a library product), then the tcgen05 kernel runs on the expanded rows.  ``q [M, n (dn +
+    rd)]`` with the ``rd`` part of every head rotated, ``out [M, n dv]``; ``gate`` (``[M, n]``): a head's output times
+    ``sigmoid(gate)``."""
+    _cuda(q, out, w_kv, sinks, gate)
+    _cols(q, "attention")
+    _cols(out, "attention")
+    if q.shape[1] != n * (dn + rd) or out.shape[1] != n * dv or q.dtype != torch.bfloat16 or out.dtype != q.dtype:
+        raise KernelError("attention: q must be bfloat16 [M, n * (dn + rd)] and out [M, n * dv]")
+    _opt_f32(sinks, n, "attention (sinks)")
+    if gate is not None:
+        _cols(gate, "attention (gate)")
+        if gate.shape != (q.shape[0], n) or gate.dtype != q.dtype:
+            raise KernelError("attention: the gate must be [M, heads] in q's dtype")
+    kv = linear(lat.rows[:, :lat.rank], w_kv)
+    tt = EXPANDED_TILE_TOKENS
+    tile_req, tile_tok0, n_tiles = (ctx.tiles_multi if ctx.n_single else ctx.tiles)[tt]
+    lib = _waiting_lib("attention_tc", q.device)
+    rc = lib.mi_attention_expanded(
+        _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kv), _ptr(lat.rows), lat.rows.shape[1], lat.rank, kv.shape[0],
+        _ptr(lat.start), _ptr(lat.first), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len), _ptr(tile_req),
+        _ptr(tile_tok0), int(n_tiles), tt, n, dn, rd, dv, float(scale), int(window), _ptr(sinks), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, _stream())
     _finish(lib, rc, "attention")
 
 

@@ -137,10 +137,10 @@ extern "C" int mi_qk_bias_norm_store(void* packed, int stride, int q_off, int k_
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_prepare_kernel(const T* __restrict__ packed, int stride, int q_off, int nq, int q_head, int q_rot_off, int c_off,
+latent_prepare_kernel(const T* packed, int stride, int q_off, int nq, int q_head, int q_rot_off, int c_off,
                       int rank, int rot_dim, int rot, const int* __restrict__ positions,
                       const double* __restrict__ freq, const float* __restrict__ c_gain, float eps,
-                      T* __restrict__ qfull, int qfull_stride, int qfull_head, const int* __restrict__ slots,
+                      T* qfull, int qfull_stride, int qfull_head, const int* __restrict__ slots,
                       T* __restrict__ kcache, int page_size, int writes, int interleaved, int cq_off, int cq_rank,
                       const float* __restrict__ cq_gain, T* __restrict__ cq_out) {
   mi_pdl_enter();
@@ -203,10 +203,22 @@ latent_prepare_kernel(const T* __restrict__ packed, int stride, int q_off, int n
     for (int k = tid; k < rot_dim; k += blockDim.x)
       kdst[mi_swizzled(rank + k, offset, mk, EPC)] = mi_from_float<T>(rotated(kr, k));
   }
-  for (int idx = tid; idx < nq * rot_dim; idx += blockDim.x) {
-    const int h = idx / rot_dim, k = idx - h * rot_dim;
+  // the queries' rotated parts, a pair per thread (qfull may be the packed projection itself)
+  const int q_pairs = half + (rot_dim - rot);            // pairs, then the dimensions that pass one by one
+  for (int idx = tid; idx < nq * q_pairs; idx += blockDim.x) {
+    const int h = idx / q_pairs, i = idx - h * q_pairs;
     const T* qr = row + q_off + h * q_head + q_rot_off;
-    qfull[(size_t)t * qfull_stride + h * qfull_head + rank + k] = mi_from_float<T>(rotated(qr, k));
+    T* dst = qfull + (size_t)t * qfull_stride + h * qfull_head + rank;
+    if (i < half) {
+      const int k1 = interleaved ? 2 * i : i, k2 = interleaved ? 2 * i + 1 : i + half;
+      float y1, y2;
+      mi_rotate(mi_to_float(qr[k1]), mi_to_float(qr[k2]), sn[i], cs[i], y1, y2);
+      dst[k1] = mi_from_float<T>(y1);
+      dst[k2] = mi_from_float<T>(y2);
+    } else {
+      const int k = rot + (i - half);
+      dst[k] = qr[k];
+    }
   }
 }
 
@@ -238,6 +250,74 @@ extern "C" int mi_latent_prepare(const void* packed, int stride, int q_off, int 
   MI_RETURN_LAUNCH_STATUS();
 }
 
+
+// Cached latent rows of this step's requests, side by side in one tensor, for an attention that
+// expands them: row e_start[b] + (j - e_first[b]) of `rows` holds the cache row of position j of
+// request b ([rank + rot_dim] numbers, un-permuted), then zeros up to `cols` columns.  A request's rows
+// start at e_first[b], the multiple of 64 at or below the first key its portion sees, and are a
+// multiple of 64 in number; positions that nobody sees or that do not exist yet are rows of zeros.
+// Requests of one token have no rows with skip_single.  The first block of a request leaves
+// e_start and e_first for the kernels behind.  grid = (tiles of GATHER_ROWS rows, requests)
+#define GATHER_ROWS 16
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const T* __restrict__ kcache, const int* __restrict__ block_table, int bt_stride,
+                     const int* __restrict__ table_rows, int page_size, const int* __restrict__ q_len,
+                     const int* __restrict__ kv_len, int window, int skip_single, int width, T* __restrict__ rows,
+                     int cols, int* __restrict__ e_start, int* __restrict__ e_first) {
+  mi_pdl_enter();
+  const int b = blockIdx.y, tid = threadIdx.x;
+  auto first_seen = [&](int r) { return window > 0 ? max(0, kv_len[r] - q_len[r] - window + 1) : 0; };
+  auto count = [&](int r) {
+    if (skip_single && q_len[r] == 1) return 0;
+    const int f = first_seen(r) / 64 * 64;
+    return (kv_len[r] - f + 63) / 64 * 64;
+  };
+  __shared__ int start_sh;
+  if (tid < 32) {                      // rows of the requests before this one
+    int s = 0;
+    for (int r = tid; r < b; r += 32) s += count(r);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (tid == 0) start_sh = s;
+  }
+  __syncthreads();
+  const int start = start_sh, lo = first_seen(b), first = lo / 64 * 64, n = count(b), kl = kv_len[b];
+  if (blockIdx.x == 0 && tid == 0) {
+    e_start[b] = start;
+    e_first[b] = first;
+  }
+  const int trow = table_rows ? table_rows[b] : b;
+  constexpr int EPC = 16 / (int)sizeof(T);
+  const int mk = mi_swizzle_mask_rows(width, (int)sizeof(T));
+  const int pieces = cols / EPC, own = width / EPC;      // whole 16-byte pieces (the host checks)
+  for (int idx = tid; idx < GATHER_ROWS * pieces; idx += blockDim.x) {
+    const int r = blockIdx.x * GATHER_ROWS + idx / pieces, c = idx % pieces;
+    if (r >= n) continue;
+    const int j = first + r;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (c < own && j >= lo && j < kl) {
+      const int page = block_table[(size_t)trow * bt_stride + j / page_size], off = j % page_size;
+      v = *reinterpret_cast<const uint4*>(kcache + ((size_t)page * page_size + off) * width + ((c ^ (off & mk)) * EPC));
+    }
+    *reinterpret_cast<uint4*>(rows + (size_t)(start + r) * cols + c * EPC) = v;
+  }
+}
+
+extern "C" int mi_latent_gather(const void* kcache, const int* block_table, int bt_stride, const int* table_rows,
+                                int page_size, const int* q_len, const int* kv_len, int n_requests, int max_rows,
+                                int window, int skip_single, int width, void* rows, int cols, int* e_start, int* e_first,
+                                int dtype, cudaStream_t stream) {
+  if (n_requests <= 0 || max_rows <= 0) return 0;
+  if (n_requests > 65535) MI_REFUSE("latent_gather: %d requests in one step", n_requests);
+  if (dtype != MI_DTYPE_BF16) MI_REFUSE("latent_gather: bfloat16 rows only");
+  if (page_size <= 0 || width <= 0 || width % 8 || cols % 8 || cols < width || !mi_aligned(kcache, 16) || !mi_aligned(rows, 16))
+    MI_REFUSE("latent_gather: rows of %d in rows of %d must be whole 16-byte pieces", width, cols);
+  const dim3 grid((unsigned)((max_rows + GATHER_ROWS - 1) / GATHER_ROWS), (unsigned)n_requests);
+  MI_LAUNCH((latent_gather_kernel<bf16>), grid, 256, 0, stream, (const bf16*)kcache, block_table, bt_stride, table_rows,
+            page_size, q_len, kv_len, window, skip_single, width, (bf16*)rows, cols, e_start, e_first);
+  MI_RETURN_LAUNCH_STATUS();
+}
 
 #define ROPE_MAX_D 1024
 

@@ -107,7 +107,14 @@ class LatentAttention(ProjectedMixer):
 
     def plan_needs(self):
         tiles = {ops.ATTENTION_TILE_TOKENS} | ops.rows_attention_tile_sizes(self.heads, 1, self.rank + self.rd, self.rank, True)
+        if self._expands():
+            tiles.add(ops.EXPANDED_TILE_TOKENS)
         return PlanNeeds(frozenset(tiles))
+
+    def _expands(self) -> bool:
+        """Whether prompt portions may run on expanded keys and values (bfloat16; single tokens never do)."""
+        return (ops.expanded_latent_supported(self.heads, self.d, self.rd, self.dv, self.rank) and self.scale > 0
+                and ops.rows_attention_supported(self.heads, 1, self.rank + self.rd, self.rank, True))
 
     def bind(self, tensors, dtype, device):
         names = ["dq" if self.q_rank else "q", "dkv"] + (["g"] if self.gate else [])
@@ -124,6 +131,9 @@ class LatentAttention(ProjectedMixer):
         # expands a weighted sum of latents to the head's value
         self.uk_t = _as_compute(tensors["uk"], dtype).reshape(n, self.d, self.rank).transpose(1, 2).contiguous()
         self.uv = _as_compute(tensors["uv"], dtype).reshape(n, self.dv, self.rank).contiguous()
+        self.w_kv = None                # both expansions as one matrix, for prompt portions
+        if dtype == torch.bfloat16 and self._expands():
+            self.w_kv = torch.cat([_as_compute(tensors["uk"], dtype), _as_compute(tensors["uv"], dtype)]).contiguous()
         self.c_gain = _f32(tensors["dkv.norm"])
         self.sinks = None
         if self.sink == "learned":
@@ -139,33 +149,56 @@ class LatentAttention(ProjectedMixer):
             raise ValueError("a latent attention rotates by itself and takes no position part")
         n, rank, dk = self.heads, self.rank, self.rank + self.rd
         M = ctx.n_tokens
-        qfull = torch.empty((M, n, dk), dtype=proj.dtype, device=proj.device)
         group = ctx.groups[cache.group]
         common = dict(positions=ctx.positions, freq=self.freq, eps=self.eps, interleaved=self.interleaved)
         row = dict(c_gain=self.c_gain, slots=group.slots if cache.writes else None,
                    kcache=cache.k if cache.writes else None)
         sizes = (self.c_off, rank, self.rd, self.rot)
+        gate = proj[:, self.g_off:self.g_off + self.gate_width] if self.gate else None
+        # a step's prompt portions expand the keys and values they see once and attend per head; single tokens (and
+        # short portions) attend in the latent's space
+        prompt_tokens = 0 if ctx.decode_only or self.w_kv is None else M - ctx.n_single
+        if not self.q_rank and (proj.stride(0) % 8 or proj.data_ptr() % 16):
+            prompt_tokens = 0                       # the kernel reads a head's query in 16-byte pieces
+        expand = prompt_tokens >= ops.EXPANDED_MIN_TOKENS
+        in_latent_space = not expand or ctx.n_single > 0
+        q = proj[:, :n * self.qh]
         if self.q_rank:
-            # the cache row and the queries' normed latent; then, from their product, the rotated query parts
+            # the cache row and the queries' normed latent; then their product
             cq = torch.empty((M, self.q_rank), dtype=proj.dtype, device=proj.device)
             ops.latent_prepare(proj, 0, 0, self.qh, self.d, *sizes, qfull=None, cq_gain=self.cq_gain, cq_out=cq,
                                **row, **common)
             q = self.uq(cq)
-            ops.latent_prepare(q, 0, n, self.qh, self.d, *sizes, c_gain=None, qfull=qfull, **common)
-        else:
-            q = proj
-            ops.latent_prepare(proj, 0, n, self.qh, self.d, *sizes, qfull=qfull, **row, **common)
-        q_un = q[:, :n * self.qh].unflatten(1, (n, self.qh))[:, :, :self.d]
-        ops.batched_linear(q_un, self.uk_t, qfull[:, :, :rank])
-        latent = torch.empty((M, n * rank), dtype=proj.dtype, device=proj.device)
-        ops.attention_ext(qfull.view(M, n * dk), latent, cache, ctx, n, 1, dk, rank, self.scale,
-                          window=self.window or 0, sinks=self.sinks, values_in_keys=True)
-        heads = torch.empty((M, n, self.dv), dtype=proj.dtype, device=proj.device)
-        ops.batched_linear(latent.view(M, n, rank), self.uv, heads)
-        heads = heads.view(M, n * self.dv)
+            row = dict(c_gain=None)
+        heads = torch.empty((M, n * self.dv), dtype=proj.dtype, device=proj.device)
+        qfull = torch.empty((M, n, dk), dtype=proj.dtype, device=proj.device) if in_latent_space else None
+        if row["c_gain"] is not None or in_latent_space:
+            packed = q if self.q_rank else proj
+            ops.latent_prepare(packed, 0, n if in_latent_space else 0, self.qh, self.d, *sizes, qfull=qfull, **row, **common)
+        if in_latent_space:
+            q_un = q.unflatten(1, (n, self.qh))[:, :, :self.d]
+            ops.batched_linear(q_un, self.uk_t, qfull[:, :, :rank])
+            latent = torch.empty((M, n * rank), dtype=proj.dtype, device=proj.device)
+            attend = dict(window=self.window or 0, sinks=self.sinks)
+            if expand:
+                ops.attention_latent_singles(qfull.view(M, n * dk), latent, cache, ctx, n, dk, rank, self.scale, **attend)
+            else:
+                ops.attention_ext(qfull.view(M, n * dk), latent, cache, ctx, n, 1, dk, rank, self.scale,
+                                  values_in_keys=True, **attend)
+            ops.batched_linear(latent.view(M, n, rank), self.uv, heads.view(M, n, self.dv))
+        fused_gate = expand and not in_latent_space and self.gate == "sigmoid" and self.gate_width == n and out_scale == 1.0
+        if expand:
+            lat = ops.latent_gather(cache, ctx, rank, self.rd, self.window or 0)
+            ops.latent_rotate_queries(q, n, self.qh, self.d, self.rd, self.rot, positions=ctx.positions, freq=self.freq,
+                                      interleaved=self.interleaved)
+            to = out if fused_gate and out.is_contiguous() else heads
+            fused_gate = to is out
+            ops.attention_expanded(q, to, lat, self.w_kv, ctx, n, self.d, self.rd, self.dv, self.scale,
+                                   window=self.window or 0, sinks=self.sinks, gate=gate if fused_gate else None)
+            if fused_gate:
+                return
         if self.gate:
-            ops.gate_mul(heads, proj[:, self.g_off:self.g_off + self.gate_width], out, self.gate, out_scale,
-                         per=n * self.dv // self.gate_width)
+            ops.gate_mul(heads, gate, out, self.gate, out_scale, per=n * self.dv // self.gate_width)
         elif out_scale == 1.0:
             out.copy_(heads)
         else:

@@ -559,6 +559,80 @@ def test_windows_page_borders_and_far_keys(dtype, sizes):
         run(420, 67, 16, 301, portions)                      # the window's edge lies 300 tokens behind
 
 
+@pytest.mark.parametrize("n,dn,rd,dv,rank", [(2, 64, 32, 64, 64), (3, 128, 64, 128, 96), (16, 8, 8, 16, 32), (1, 72, 16, 96, 40),
+                                             (5, 24, 0, 48, 24), (4, 120, 40, 80, 512)])
+@pytest.mark.parametrize("window,sink", [(0, False), (1, False), (50, True), (200, False), (333, True)])
+def test_prompt_portions_on_expanded_rows(n, dn, rd, dv, rank, window, sink):
+    """The tcgen05 kernel on keys and values expanded from gathered cache rows: three requests of unequal portions
+    in one step, one of them a single token that stays out of it, pages handed out from the far end and NaN
+    everywhere else; per-head gates, sinks, and a key that stands out at the window's first position of one token,
+    against the plain softmax over expanded keys."""
+    o = ops()
+    page, scale = 8, 0.7
+    assert o.expanded_latent_supported(n, dn, rd, dv, rank)
+    starts, portions = [0, 77, 301], [131, 1, 200]              # tokens held before, tokens brought
+    lens = [a + b for a, b in zip(starts, portions)]
+    width = rank + rd
+    kc = torch.full((sum(-(-x // page) for x in lens) + 2, 1, page, width), float("nan"), dtype=torch.bfloat16, device=DEV)
+    table = torch.full((4, 80), -1, dtype=torch.int32, device=DEV)
+    table_rows, free = [2, 0, 3], list(range(kc.shape[0] - 1, 0, -1))
+    w_k = rnd(n * dn, rank, seed=90, scale=rank ** -0.5).bfloat16()
+    w_v = rnd(n * dv, rank, seed=91, scale=rank ** -0.5).bfloat16()
+    M = sum(portions)
+    q = rnd(M, n, dn + rd, seed=92, scale=(dn + rd) ** -0.5).bfloat16()
+    gate = rnd(M, n, seed=93).bfloat16()
+    sinks = torch.linspace(-2.0, 3.0, n, dtype=torch.float64) if sink else None
+    rows = [rnd(x, width, seed=94 + i).bfloat16() for i, x in enumerate(lens)]
+    if window > 1:      # request 2: the token at 301 + 150 points at the first key of its window, which stands out
+        target = 451 - window + 1
+        k = (w_k.double() @ rows[2][target, :rank].double()).reshape(n, dn)
+        q[portions[0] + 1 + 150, :, :dn] = (k * 12.0 / (k * k).sum(dim=1, keepdim=True)).bfloat16()
+    by_slot = o.unpack_cache_pages(kc)
+    for i, x in enumerate(lens):
+        first = max(0, starts[i] - window + 1) if window else 0
+        held = []
+        for p in range(-(-x // page)):
+            held.append(free.pop())
+            table[table_rows[i], p] = held[-1]
+        slots = [held[j // page] * page + j % page for j in range(x)]
+        keep = list(range(first, x))                             # what lies before every window was given back
+        by_slot[[slots[j] for j in keep], 0] = rows[i][keep].to(DEV)
+    kc.copy_(o.pack_cache_pages(by_slot, page))
+    tiles = [(i, t) for i, x in enumerate(portions) if x > 1 for t in range(0, x, 128)][::-1]
+    ctx = SimpleNamespace(
+        groups=[SimpleNamespace(block_table=table, page_size=page, table_rows=i32(table_rows))], n_requests=3, n_single=1,
+        q_start=i32(np.cumsum([0] + portions[:-1])), q_len=i32(portions), kv_len=i32(lens), host_q_len=portions, host_kv_len=lens,
+        tiles={}, tiles_multi={128: (i32([t[0] for t in tiles]), i32([t[1] for t in tiles]), len(tiles))})
+    lat = o.latent_gather(SimpleNamespace(group=0, k=kc), ctx, rank, rd, window)
+    assert lat.rows.shape[0] % 64 == 0 and torch.isfinite(lat.rows).all()
+    out = torch.full((M, n * dv), float("nan"), dtype=torch.bfloat16, device=DEV)
+    o.attention_expanded(q.reshape(M, -1).to(DEV), out, lat, torch.cat([w_k, w_v]).to(DEV), ctx, n, dn, rd, dv, scale,
+                         window=window, sinks=sinks.float().to(DEV) if sink else None, gate=gate.to(DEV))
+    assert o.attention_tc_status() == 0
+    got = out.float().cpu().double().reshape(M, n, dv)
+    t0 = 0
+    for i, (a, b) in enumerate(zip(starts, portions)):
+        if b == 1:
+            assert torch.isnan(got[t0]).all()                    # a single token's row is somebody else's
+            t0 += b
+            continue
+        c, r = rows[i][:, :rank].double(), rows[i][:, rank:].double()
+        k = (c @ w_k.double().T).reshape(-1, n, dn)
+        v = (c @ w_v.double().T).reshape(-1, n, dv)
+        qq = q[t0:t0 + b].double()
+        s = (torch.einsum("thd,jhd->thj", qq[..., :dn], k) + torch.einsum("thd,jd->thj", qq[..., dn:], r)) * scale
+        pos, j = torch.arange(a, a + b)[:, None], torch.arange(a + b)[None]
+        seen = (j <= pos) & ((pos - j < window) if window else torch.ones_like(j <= pos))
+        s = s.masked_fill(~seen[:, None], float("-inf"))
+        if sink:
+            s = torch.cat([s, sinks[None, :, None].expand(b, n, 1)], dim=2)
+        p = torch.softmax(s, dim=2)[..., :a + b]
+        want = torch.einsum("thj,jhd->thd", p, v) * torch.sigmoid(gate[t0:t0 + b].double())[..., None]
+        err = (got[t0:t0 + b] - want).abs().amax(dim=(1, 2))
+        assert err.max() <= 2e-2 * max(1.0, want.abs().max()), (i, torch.nonzero(err > 2e-2).ravel()[:5].tolist(), float(err.max()))
+        t0 += b
+
+
 def test_configurations_take_both_attention_kernels():
     o = ops()
     taken = {which: [o.rows_attention_supported(l["mixer"]["heads"], 1, l["mixer"]["kv_rank"] + l["mixer"]["rot_dim"],
