@@ -360,8 +360,9 @@ class CacheManager:
                 if n_new == 1:
                     slots.append(table[start // ps] * ps + start % ps)
                 else:
-                    for p in range(start, total):
-                        slots.append(table[p // ps] * ps + p % ps)
+                    for idx in range(start // ps, -(-total // ps)):      # page by page
+                        base = table[idx] * ps
+                        slots.extend(range(base + max(0, start - idx * ps), base + min(ps, total - idx * ps)))
             req.length = total
         return plan
 

@@ -235,11 +235,19 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
       __syncthreads();                                          // the chunk before is consumed (first time: Qs written)
       list_rows(j0, 0);
       __syncthreads();
-      // four 16-byte pieces per thread are asked for before the first is stored, so that they fly together
       bf16* kdst = KV;
+      if (MT == 1) {     // few warps: every piece of the chunk is asked for at once (cp.async)
+        gather_rows_async<NT>(kdst, dp, kcache, d, mk, rowbase_all, rowoff_all, tid);
+        if (!v_prefix) gather_rows_async<NT>(kdst + CHUNK * dp, dvp, vcache, dv, mv, rowbase_all, rowoff_all, tid);
+        cp_async_commit();
+        cp_async_wait_all();
+        __syncthreads();
+      } else {
+      // four 16-byte pieces per thread are asked for before the first is stored, so that they fly together
       gather_rows<NT>(kdst, dp, kcache, d, mk, rowbase_all, rowoff_all, tid);
       if (!v_prefix) gather_rows<NT>(kdst + CHUNK * dp, dvp, vcache, dv, mv, rowbase_all, rowoff_all, tid);
       __syncthreads();
+      }
     }
 
     // ---- S = Q K^T for this warp's 16 keys: two tiles of 8 keys

@@ -199,4 +199,12 @@ __device__ __forceinline__ float mi_xielu(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
 
+// The same for a result that is rounded to bfloat16: the exponential is the hardware's, and close to zero,
+// where e^z - 1 - z would cancel, its power series z^2 / 2 + z^3 / 6 + z^4 / 24 takes its place.
+__device__ __forceinline__ float mi_xielu_bf16(float z, float a, float b) {
+  const float series = z * z * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f);
+  const float e = z > -0.125f ? series : __expf(z) - 1.f - z;
+  return fmaf(z > 0.f ? a * z : b, z > 0.f ? z : e, 0.5f * z);
+}
+
 static inline bool mi_aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) % a) == 0; }

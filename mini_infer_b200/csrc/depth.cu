@@ -202,17 +202,19 @@ extern "C" int mi_branch_depth(const float* stream, const void* branch, int bran
   MI_RETURN_LAUNCH_STATUS();
 }
 
-// One thread: V channels of a tile of tokens of one request.  The threads of a request's first tile read the
+// One thread: V channels of a tile of CONV_TILE tokens of one request; with TAPS > 0 (that many taps) all of
+// the tile's inputs are asked for before the first sum.  The threads of a request's first tile read the
 // state and, behind that, replace it (nobody else touches it).
-template <typename TX, typename T, int V>
+#define CONV_TILE 8
+template <typename TX, typename T, int V, int TAPS>
 __global__ void input_conv_kernel(const TX* __restrict__ x, int x_stride, const float* __restrict__ w, int taps,
                                   float* __restrict__ state, long long state_stride, const int* __restrict__ q_start,
                                   const int* __restrict__ q_len, const int* __restrict__ state_slot,
-                                  T* __restrict__ out, int H, int tile) {
+                                  T* __restrict__ out, int H) {
   mi_pdl_enter();
   const int k = V * (blockIdx.x * blockDim.x + threadIdx.x);
-  const int req = blockIdx.z, len = q_len[req], t0 = blockIdx.y * tile;
-  if (k >= H || t0 >= len) return;
+  const int req = blockIdx.z, len = q_len[req];
+  if (k >= H) return;
   const int row0 = q_start[req], before = taps - 1;
   float* tail = before > 0 ? state + (size_t)state_slot[req] * state_stride + k : nullptr;
   const TX* xr = x + (size_t)row0 * x_stride + k;
@@ -220,22 +222,51 @@ __global__ void input_conv_kernel(const TX* __restrict__ x, int x_stride, const 
     if (t >= 0) Pack<TX, V>::load(xr + (size_t)t * x_stride, f);
     else Pack<float, V>::load(tail + (size_t)(before + t) * H, f);
   };
-  const int t1 = min(len, t0 + tile);
-  for (int t = t0; t < t1; ++t) {
-    float acc[V], wj[V], f[V];
+  // the first block walks the first two tiles: nobody else's reach back into the state (at most 15 inputs)
+  const int tile0 = blockIdx.y == 0 ? 0 : blockIdx.y + 1, tiles = blockIdx.y == 0 ? 2 : 1;
+  for (int t0 = tile0 * CONV_TILE; t0 < min(len, (tile0 + tiles) * CONV_TILE); t0 += CONV_TILE) {
+    if (TAPS > 0) {
+      constexpr int N = TAPS > 0 ? TAPS : 1;
+      float in[CONV_TILE + N - 1][V], wj[N][V];
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = 0.f;
-    for (int j = 0; j < taps; ++j) {
-      input(t - before + j, f);
-      Pack<float, V>::load(w + (size_t)j * H + k, wj);
+      for (int i = 0; i < CONV_TILE + TAPS - 1; ++i)
+        if (t0 + i - (TAPS - 1) < len) input(t0 + i - (TAPS - 1), in[i]);
 #pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i], f[i], acc[i]);
+      for (int j = 0; j < TAPS; ++j) Pack<float, V>::load(w + (size_t)j * H + k, wj[j]);
+#pragma unroll
+      for (int t = 0; t < CONV_TILE; ++t) {
+        if (t0 + t < len) {
+          float acc[V];
+#pragma unroll
+          for (int i = 0; i < V; ++i) acc[i] = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[j][i], in[t + j][i], acc[i]);
+#pragma unroll
+          for (int i = 0; i < V; ++i) acc[i] = in[t + TAPS - 1][i] + acc[i];
+          Pack<T, V>::store(out + (size_t)(row0 + t0 + t) * H + k, acc);
+        }
+      }
+    } else {
+      const int t1 = min(len, t0 + CONV_TILE);
+      for (int t = t0; t < t1; ++t) {
+        float acc[V], wj[V], f[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = 0.f;
+        for (int j = 0; j < taps; ++j) {
+          input(t - before + j, f);
+          Pack<float, V>::load(w + (size_t)j * H + k, wj);
+#pragma unroll
+          for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i], f[i], acc[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = f[i] + acc[i];          // f: the current token, read last
+        Pack<T, V>::store(out + (size_t)(row0 + t) * H + k, acc);
+      }
     }
-#pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = f[i] + acc[i];          // f: the current token, read last
-    Pack<T, V>::store(out + (size_t)(row0 + t) * H + k, acc);
   }
-  if (t0 == 0)
+  if (blockIdx.y == 0)
     for (int j = 0; j < before; ++j) {                 // ascending: a slot is read before it is replaced
       float f[V];
       input(len - before + j, f);
@@ -255,17 +286,19 @@ extern "C" int mi_input_conv(const void* x, int x_stride, int x_dtype, const flo
                    mi_aligned(state, 16) && mi_aligned(out, 16);
   const int per = vec ? H / 4 : H;
   const int threads = 128;
-  const int tile = max_len >= 16 ? 16 : max_len;
-  const long long tiles = (max_len + tile - 1) / tile;
+  const long long tiles = (max_len + CONV_TILE - 1) / CONV_TILE;
   if (tiles > 65535) MI_REFUSE("input_conv: a portion of %d tokens", max_len);
-  const dim3 grid((unsigned)((per + threads - 1) / threads), (unsigned)tiles, (unsigned)n_requests);
-#define MI_GO(TX, T, V)                                                                                       \
-  MI_LAUNCH((input_conv_kernel<TX, T, V>), grid, threads, 0, stream, (const TX*)x, x_stride, w, taps, state, \
-            state_stride, q_start, q_len, state_slot, (T*)out, H, tile)
-#define MI_PICK(TX, T)                        \
-  do {                                        \
-    if (vec) MI_GO(TX, T, 4);                 \
-    else MI_GO(TX, T, 1);                     \
+  const dim3 grid((unsigned)((per + threads - 1) / threads), (unsigned)(tiles > 2 ? tiles - 1 : 1), (unsigned)n_requests);
+#define MI_GO(TX, T, V, TAPS)                                                                                      \
+  MI_LAUNCH((input_conv_kernel<TX, T, V, TAPS>), grid, threads, 0, stream, (const TX*)x, x_stride, w, taps, state, \
+            state_stride, q_start, q_len, state_slot, (T*)out, H)
+#define MI_PICK(TX, T)                          \
+  do {                                          \
+    if (vec && taps == 2) MI_GO(TX, T, 4, 2);   \
+    else if (vec && taps == 3) MI_GO(TX, T, 4, 3); \
+    else if (vec && taps == 4) MI_GO(TX, T, 4, 4); \
+    else if (vec) MI_GO(TX, T, 4, 0);           \
+    else MI_GO(TX, T, 1, 0);                    \
   } while (0)
   if (dtype == MI_DTYPE_F32 && x_dtype == MI_DTYPE_F32) MI_PICK(float, float);
   else if (dtype == MI_DTYPE_BF16 && x_dtype == MI_DTYPE_F32) MI_PICK(float, bf16);

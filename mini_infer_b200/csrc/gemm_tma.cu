@@ -425,7 +425,8 @@ gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
         if (n < N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(mi_xielu(v[j], fus.act_a, fus.act_b));
+            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(sizeof(OutT) == 2 ? mi_xielu_bf16(v[j], fus.act_a, fus.act_b)
+                                                                                                : mi_xielu(v[j], fus.act_a, fus.act_b));
         }
       } else if (swiglu) {
         // rows alternate gate, up: the even lane of a pair has the gate, its neighbour the up

@@ -26,6 +26,20 @@ __global__ void embedding_scaled_kernel(const T* __restrict__ table, const int* 
     return;
   }
   const T* src = table + (size_t)id * H;
+  if (H % 4 == 0) {                    // rows of whole aligned pieces (the host's tensors start aligned)
+    for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
+      Vec4<T> a;
+      float f[4];
+      a.load(src + i);
+      a.get(f);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[j] *= scale;
+      Vec4<float> o;
+      o.set(f);
+      o.store(dst + i);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = mi_to_float(src[i]) * scale;
 }
 
@@ -33,6 +47,7 @@ extern "C" int mi_embedding_scaled(const void* table, const int* ids, float* out
                                    float scale, int dtype, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (H <= 0 || V <= 0) MI_REFUSE("embedding: bad sizes H=%d V=%d", H, V);
+  if (!mi_aligned(table, 16) || !mi_aligned(out, 16)) MI_REFUSE("embedding: the table and the stream must be 16-byte aligned");
   const int threads = H >= 1024 ? 256 : 128;
   if (dtype == MI_DTYPE_F32)
     MI_LAUNCH((embedding_scaled_kernel<float>), M, threads, 0, stream, (const float*)table, ids, out, H, V, scale);

@@ -658,12 +658,68 @@ __global__ void moe_combine_kernel(const YT* __restrict__ y, const int* __restri
   }
 }
 
+// the same with four columns per access (sums in the same order)
+template <typename T, typename YT>
+__global__ void moe_combine4_kernel(const YT* __restrict__ y, const int* __restrict__ inv,
+                                    const float* __restrict__ weights, const T* __restrict__ shared, int shared_stride,
+                                    T* __restrict__ out, int H, int top, const float* __restrict__ shared_gate,
+                                    int gate_stride) {
+  mi_pdl_enter();
+  __shared__ int rows[32];
+  __shared__ float wts[32];
+  const int t = blockIdx.x;
+  if (threadIdx.x < top) {
+    rows[threadIdx.x] = inv[(size_t)t * top + threadIdx.x];
+    wts[threadIdx.x] = weights[(size_t)t * top + threadIdx.x];
+  }
+  const float sg = (shared && shared_gate) ? 1.f / (1.f + expf(-shared_gate[(size_t)t * gate_stride])) : 1.f;
+  __syncthreads();
+  for (int c = 4 * threadIdx.x; c < H; c += 4 * blockDim.x) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, f[4];
+    for (int k0 = 0; k0 < top; k0 += 4) {              // four experts' pieces in flight
+      Vec4<YT> v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (k0 + u < top) v[u].load(y + (size_t)rows[k0 + u] * H + c);
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (k0 + u < top) {
+          v[u].get(f);
+          const float w = wts[k0 + u];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[i] = fmaf(w, f[i], acc[i]);
+        }
+    }
+    if (shared) {
+      Vec4<T> v;
+      v.load(shared + (size_t)t * shared_stride + c);
+      v.get(f);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = fmaf(sg, f[i], acc[i]);
+    }
+    Vec4<T> o;
+    o.set(acc);
+    o.store(out + (size_t)t * H + c);
+  }
+}
+
 // y_dtype: the experts' outputs are fp32 (own products) or in the compute dtype (a library's grouped product)
 extern "C" int mi_moe_combine(const void* y, int y_dtype, const int* inv, const float* weights, const void* shared,
                               int shared_stride, void* out, int M, int H, int top, const float* shared_gate,
                               int gate_stride, int dtype, cudaStream_t stream) {
   if (M <= 0) return 0;
   const int threads = H >= 1024 ? 256 : 128;
+  if (dtype == MI_DTYPE_BF16 && H % 4 == 0 && top <= 32 && mi_aligned(y, 16) && mi_aligned(out, 8) && mi_aligned(shared, 8) &&
+      (!shared || shared_stride % 4 == 0) && (y_dtype == MI_DTYPE_F32 || y_dtype == MI_DTYPE_BF16)) {
+    const int t4 = H >= 4096 ? 512 : (H >= 1024 ? 256 : 128);
+    if (y_dtype == MI_DTYPE_F32)
+      MI_LAUNCH((moe_combine4_kernel<bf16, float>), M, t4, 0, stream, (const float*)y, inv, weights, (const bf16*)shared,
+                shared_stride, (bf16*)out, H, top, shared_gate, gate_stride);
+    else
+      MI_LAUNCH((moe_combine4_kernel<bf16, bf16>), M, t4, 0, stream, (const bf16*)y, inv, weights, (const bf16*)shared,
+                shared_stride, (bf16*)out, H, top, shared_gate, gate_stride);
+    MI_RETURN_LAUNCH_STATUS();
+  }
   if (dtype == MI_DTYPE_F32 && y_dtype == MI_DTYPE_F32)
     MI_LAUNCH((moe_combine_kernel<float, float>), M, threads, 0, stream, (const float*)y, inv, weights,
               (const float*)shared, shared_stride, (float*)out, H, top, shared_gate, gate_stride);
@@ -691,10 +747,36 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, int stride, T* __re
   }
 }
 
+// the same with four outputs per access (grid: column groups x rows)
+template <typename T>
+__global__ void clamped_glu4_kernel(const T* __restrict__ gu, int stride, T* __restrict__ out, int M, int I,
+                                    float limit, float alpha, float offset) {
+  mi_pdl_enter();
+  const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+  if (c >= I) return;
+  for (int t = blockIdx.y; t < M; t += gridDim.y) {
+    Vec4<T> a, b;
+    a.load(gu + (size_t)t * stride + c);
+    b.load(gu + (size_t)t * stride + I + c);
+    float g[4], u[4];
+    a.get(g);
+    b.get(u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) g[i] = mi_clamped_glu_value(g[i], u[i], limit, alpha, offset);
+    a.set(g);
+    a.store(out + (size_t)t * I + c);
+  }
+}
+
 extern "C" int mi_clamped_glu(const void* gu, int stride, void* out, int M, int I, float limit, float alpha,
                               float offset, int dtype, cudaStream_t stream) {
   if (M <= 0 || I <= 0) return 0;
   const size_t n = (size_t)M * I;
+  if (dtype == MI_DTYPE_BF16 && I % 4 == 0 && stride % 4 == 0 && mi_aligned(gu, 8) && mi_aligned(out, 8)) {
+    const dim3 grid((unsigned)((I / 4 + 127) / 128), (unsigned)(M < 16384 ? M : 16384));
+    MI_LAUNCH((clamped_glu4_kernel<bf16>), grid, 128, 0, stream, (const bf16*)gu, stride, (bf16*)out, M, I, limit, alpha, offset);
+    MI_RETURN_LAUNCH_STATUS();
+  }
   const int blocks = (int)((n + 255) / 256 < 4096 ? (n + 255) / 256 : 4096);
   if (dtype == MI_DTYPE_F32)
     MI_LAUNCH((clamped_glu_kernel<float>), blocks, 256, 0, stream, (const float*)gu, stride, (float*)out, M, I, limit, alpha, offset);

@@ -32,7 +32,7 @@ def _ptr(t: torch.Tensor | None) -> c_void_p:
 
 
 def _stream() -> c_void_p:
-    return c_void_p(torch.cuda.current_stream().cuda_stream)
+    return c_void_p(torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice()))
 
 
 def _cuda(*tensors: torch.Tensor | None) -> None:

@@ -391,12 +391,13 @@ __global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, size_
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
-        const __nv_bfloat162 o = __floats2bfloat162_rn(mi_xielu(f.x, a, b), mi_xielu(f.y, a, b));
+        const __nv_bfloat162 o = __floats2bfloat162_rn(mi_xielu_bf16(f.x, a, b), mi_xielu_bf16(f.y, a, b));
         w[j] = *reinterpret_cast<const uint32_t*>(&o);
       }
       reinterpret_cast<uint4*>(out)[idx] = v;
     } else {
-      out[idx] = mi_from_float<T>(mi_xielu(mi_to_float(x[idx]), a, b));
+      const float z = mi_to_float(x[idx]);
+      out[idx] = mi_from_float<T>(sizeof(T) == 2 ? mi_xielu_bf16(z, a, b) : mi_xielu(z, a, b));
     }
   }
 }

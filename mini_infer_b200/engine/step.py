@@ -112,9 +112,14 @@ class StepRunner:
         for e in entries:
             if len(e.tokens) == 0:
                 raise StepError(f"request {e.rid!r}: no tokens in this step")
-            for t in e.tokens:
-                if not 0 <= int(t) < V:
-                    raise StepError(f"request {e.rid!r}: token id {t} is outside [0, {V})")
+            check = True
+            if len(e.tokens) > 8:                # a long portion: one pass, and the loop only to name the token
+                ids = np.asarray(e.tokens)
+                check = ids.dtype.kind not in "iu" or ids.min() < 0 or ids.max() >= V
+            if check:
+                for t in e.tokens:
+                    if not 0 <= int(t) < V:
+                        raise StepError(f"request {e.rid!r}: token id {t} is outside [0, {V})")
             for w in e.want:
                 if not 0 <= int(w) < len(e.tokens):
                     raise StepError(f"request {e.rid!r}: wanted place {w} is outside its {len(e.tokens)} tokens")
@@ -150,10 +155,9 @@ class StepRunner:
                     want_rows.append(i)
                     rows.append((e.rid, int(w)))
         else:
-            tokens, positions = [], []
+            tokens = np.concatenate([np.asarray(e.tokens, dtype=np.int64) for e in entries])
+            positions = np.concatenate([np.arange(plan.start[i], kv_len[i]) for i in range(B)])
             for i, e in enumerate(entries):
-                tokens.extend(int(t) for t in e.tokens)
-                positions.extend(range(plan.start[i], kv_len[i]))
                 for w in e.want:
                     want_rows.append(q_start[i] + int(w))
                     rows.append((e.rid, int(w)))
@@ -197,18 +201,20 @@ class StepRunner:
                 # Tiles with the most keys to walk come first: the attention kernels start their
                 # blocks in this order, so the long ones are under way when the short ones fill
                 # what is left (a tile of tokens t0.. of request i sees its keys up to the tile's end).
-                tiles = [(i, t0) for i in range(B) for t0 in range(0, q_len[i], n)]
-                tiles.sort(key=lambda it: -(kv_len[it[0]] - q_len[it[0]] + min(q_len[it[0]], it[1] + n)))
-                treq = [i for i, _ in tiles]
-                ttok = [t0 for _, t0 in tiles]
+                first = [np.arange(0, q_len[i], n) for i in range(B)]
+                ttok = np.concatenate(first)
+                treq = np.repeat(np.arange(B), [len(f) for f in first])
+                ends = np.concatenate([kv_len[i] - q_len[i] + np.minimum(q_len[i], f + n) for i, f in enumerate(first)])
+                order = np.argsort(-ends, kind="stable")
+                treq, ttok = treq[order], ttok[order]
             tile_counts[n] = len(treq)
             parts.append((f"tile_req{n}", treq))
             parts.append((f"tile_tok{n}", ttok))
             if singles:
-                keep = [j for j, i in enumerate(treq) if q_len[i] > 1]
-                multi_counts[n] = len(keep)
-                parts.append((f"multi_req{n}", [treq[j] for j in keep]))
-                parts.append((f"multi_tok{n}", [ttok[j] for j in keep]))
+                keep = np.asarray(q_len)[treq] > 1
+                multi_counts[n] = int(keep.sum())
+                parts.append((f"multi_req{n}", treq[keep]))
+                parts.append((f"multi_tok{n}", ttok[keep]))
 
         offsets: dict[str, tuple[int, int]] = {}
         total = 0
