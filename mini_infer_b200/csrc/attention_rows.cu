@@ -21,7 +21,8 @@
 //
 // With n_splits > 1 the keys of every tile are cut into that many runs of whole chunks, one block
 // each; the blocks leave unnormalised sums with their maxima and denominators in `part_o` / `part_ml`
-// and attention_rows_merge_kernel adds them up (and the sink) in a fixed order.
+// and attention_rows_merge_kernel adds them up (and the sink) in a fixed order, or, without `merge`, whoever
+// reads them does.
 //
 // Layouts as in attention_generic.cu: q [tokens, q_stride], out [tokens, out_stride], kcache
 // [pages, nkv, page_size, d], vcache [pages, nkv, page_size, dv] (null with v_prefix), block tables
@@ -508,7 +509,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
                                  const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens, int rows,
                                  int nq, int nkv, int d, int dv, float scale, const float* sinks, const float* slopes,
                                  int v_prefix, int n_splits, float* part_o, float* part_ml, int stages,
-                                 int window, cudaStream_t stream) {
+                                 int window, int merge, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (stages != 1 && stages != 2) MI_REFUSE("attention_rows: one or two buffers for a chunk, not %d", stages);
   if ((rows == 2 * ROWS && stages != 2) || (rows == ROWS && stages != 1))
@@ -570,7 +571,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
       return (int)e;
     }
   }
-  if (n_splits > 1)
+  if (n_splits > 1 && merge)
     MI_LAUNCH(attention_rows_merge_kernel, (unsigned)(units * rows), 128, 0, stream, (const float*)part_o,
               (const float*)part_ml, (bf16*)out, out_stride, q_start, q_len, tile_req, tile_tok0, tile_tokens, nq, nkv,
               dv, sinks, n_splits, rows);

@@ -46,6 +46,7 @@ LIBRARIES: dict[str, tuple[list[str], list[str], list[str]]] = {
     "qk_prepare": (["qk_prepare.cu"], ["common.cuh"], []),
     "attention_rows": (["attention_rows.cu"], ["common.cuh"], []),
     "depth": (["depth.cu"], ["common.cuh"], []),
+    "latent_decode": (["latent_decode.cu"], ["common.cuh"], []),
 }
 
 

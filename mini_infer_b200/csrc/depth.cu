@@ -159,6 +159,93 @@ __global__ void branch_depth_kernel(const BranchDepthArgs a) {
   }
 }
 
+// The same for rows of up to 4096 channels in whole 16-byte pieces: a thread holds four channels from the first
+// load to the last store, and everything that does not depend on the row's statistics is asked for before them.
+#define ROW_MAX_THREADS 1024
+template <typename T>
+__global__ void __launch_bounds__(ROW_MAX_THREADS)
+branch_depth_row_kernel(const BranchDepthArgs a) {
+  mi_pdl_launch_dependents();
+  __shared__ float red[32];
+  const int t = blockIdx.x, H = a.H, k = 4 * threadIdx.x;
+  const bool on = k < H;
+  const size_t at = (size_t)t * H + k;
+  float g[4] = {}, c[4] = {}, y[4] = {}, x[4] = {}, acc[4] = {};
+  if (on && a.branch) {                // immutable: may be read before the kernels in front have finished
+    Pack<float, 4>::load(a.w + k, g);
+    Pack<float, 4>::load(a.b + k, c);
+  }
+  mi_pdl_wait();
+  if (on) {
+    if (a.branch) Pack<T, 4>::load(reinterpret_cast<const T*>(a.branch) + (size_t)t * a.branch_stride + k, y);
+    Pack<float, 4>::load(a.stream + at, x);
+    if (a.n_prev > 0) {
+      float f[4];
+      Pack<float, 4>::load(a.first + at, f);
+      const float a0 = a.avg[0];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] = a0 * f[i];
+      const float* res = a.results + at;
+      const size_t pitch = (size_t)a.M * H;
+      int j = 1;
+      for (; j + 4 <= a.n_prev; j += 4) {             // four results in flight; added in order
+        float r[4][4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) Pack<float, 4>::load(res + (size_t)(j - 1 + u) * pitch, r[u]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const float wj = a.avg[j + u];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[i] = fmaf(wj, r[u][i], acc[i]);
+        }
+      }
+      for (; j < a.n_prev; ++j) {
+        Pack<float, 4>::load(res + (size_t)(j - 1) * pitch, f);
+        const float wj = a.avg[j];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[i] = fmaf(wj, f[i], acc[i]);
+      }
+    }
+  }
+  if (a.branch) {
+    const float mean = mi_block_sum((y[0] + y[1]) + (y[2] + y[3]), red) / (float)H;
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      y[i] -= mean;
+      sq += y[i] * y[i];
+    }
+    const float rstd = 1.f / sqrtf(mi_block_sum(on ? sq : 0.f, red) / (float)H + a.eps);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) x[i] += y[i] * rstd * g[i] + c[i];
+  }
+  if (!on) return;
+  if (a.stream_out) Pack<float, 4>::store(a.stream_out + at, x);
+  if (a.n_prev > 0) {
+    const float an = a.avg[a.n_prev];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) x[i] = fmaf(an, x[i], acc[i]);
+    if (a.avg_out) Pack<float, 4>::store(a.avg_out + at, x);
+  }
+  if (a.copy) Pack<T, 4>::store(reinterpret_cast<T*>(a.copy) + at, x);
+  if (a.conv_w) {
+    float* tail = a.taps > 1 ? a.conv_state + (size_t)a.state_slot[t] * a.conv_stride + k : nullptr;
+    float s[4] = {}, w[4], in[4];
+    for (int j = 0; j < a.taps - 1; ++j) {
+      Pack<float, 4>::load(a.conv_w + (size_t)j * H + k, w);
+      Pack<float, 4>::load(tail + (size_t)j * H, in);
+      if (j > 0) Pack<float, 4>::store(tail + (size_t)(j - 1) * H, in);     // the state moves on by one token
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[i] = fmaf(w[i], in[i], s[i]);
+    }
+    Pack<float, 4>::load(a.conv_w + (size_t)(a.taps - 1) * H + k, w);
+    if (a.taps > 1) Pack<float, 4>::store(tail + (size_t)(a.taps - 2) * H, x);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) s[i] = x[i] + fmaf(w[i], x[i], s[i]);
+    Pack<T, 4>::store(reinterpret_cast<T*>(a.conv_out) + at, s);
+  }
+}
+
 extern "C" int mi_branch_depth(const float* stream, const void* branch, int branch_stride, const float* w,
                                const float* b, float eps, float* stream_out, void* copy, const float* first,
                                const float* results, int n_prev, const float* avg, float* avg_out,
@@ -181,6 +268,13 @@ extern "C" int mi_branch_depth(const float* stream, const void* branch, int bran
                    mi_aligned(copy, 16) && mi_aligned(first, 16) && mi_aligned(results, 16) && mi_aligned(avg_out, 16) &&
                    mi_aligned(conv_w, 16) && mi_aligned(conv_state, 16) && mi_aligned(conv_out, 16);
   const int per = vec ? H / 4 : H;
+  if (vec && per <= ROW_MAX_THREADS) {      // (the choice depends on the width alone: a row's bits do not depend on the step)
+    const int row_threads = (per + 31) / 32 * 32;
+    if (dtype == MI_DTYPE_F32) MI_LAUNCH((branch_depth_row_kernel<float>), M, row_threads, 0, cu_stream, a);
+    else if (dtype == MI_DTYPE_BF16) MI_LAUNCH((branch_depth_row_kernel<bf16>), M, row_threads, 0, cu_stream, a);
+    else MI_REFUSE("branch_depth: unknown dtype %d", dtype);
+    MI_RETURN_LAUNCH_STATUS();
+  }
   const int threads = per >= 1024 ? 512 : (per >= 256 ? 256 : 128);
 #define MI_GO(T, V)                                                                                         \
   do {                                                                                                      \

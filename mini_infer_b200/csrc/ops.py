@@ -334,11 +334,18 @@ def _sig_qk_prepare(lib: ctypes.CDLL) -> None:
                                      c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p]
 
 
+def _sig_latent_decode(lib: ctypes.CDLL) -> None:
+    lib.mi_latent_query.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                    c_void_p, c_void_p, c_void_p]
+    lib.mi_latent_value.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                    c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p]
+
+
 def _sig_attention_rows(lib: ctypes.CDLL) -> None:
     lib.mi_attention_rows.argtypes = [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p]
+        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
     lib.mi_attention_rows_tile_tokens.argtypes = [c_int, c_int]
     lib.mi_attention_rows_supported.argtypes = [c_int, c_int, c_int, c_int, c_int]
 
@@ -346,6 +353,7 @@ def _sig_attention_rows(lib: ctypes.CDLL) -> None:
 _SIGNATURES = {
     "attention_rows": _sig_attention_rows,
     "depth": _sig_depth,
+    "latent_decode": _sig_latent_decode,
     "stream": _sig_stream,
     "qk_prepare": _sig_qk_prepare,
     "layernorm": _sig_layernorm,
@@ -2357,7 +2365,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), _ptr(vc), _ptr(bt), bt.stride(0),
             _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len),
             _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), tt, rows, nq, nkv, d, dv, float(scale), _ptr(sinks),
-            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, int(window), _stream())
+            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, int(window), 1, _stream())
         _finish(lib, rc, "attention")
         if splits > 1:
             launch_count += 1        # the merge of the runs
@@ -2397,10 +2405,101 @@ def attention_latent_singles(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq:
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), None, _ptr(bt), bt.stride(0), _ptr(ctx.single_rows),
         int(group.page_size), _ptr(ctx.single_q_start), None, _ptr(ctx.single_kv_len), None, None, int(ctx.n_single),
         rows_attention_tile_tokens(nq, 16), 16, nq, 1, d, dv, float(scale), _ptr(sinks), None, 1, splits, _ptr(part_o),
-        _ptr(part_ml), 1, int(window), _stream())
+        _ptr(part_ml), 1, int(window), 1, _stream())
     _finish(lib, rc, "attention")
     if splits > 1:
         launch_count += 1
+
+
+# --------------------------------------------------------------------------------------- single tokens in the latent's space
+
+
+LATENT_DECODE_TOKENS = 16      # steps of up to this many single tokens run the fused small products
+
+
+def latent_decode_fusable(dtype: torch.dtype, ctx, n: int, d: int, rd: int, dv: int, rank: int, q: torch.Tensor) -> bool:
+    """Whether this step's single tokens run ``latent_query``, ``attention_latent_runs`` and ``latent_value``."""
+    return (dtype == torch.bfloat16 and ctx.decode_only and ctx.n_tokens <= LATENT_DECODE_TOKENS
+            and d % 8 == 0 and d <= 128 and (d + rd) % 8 == 0 and rank % 8 == 0 and rank <= 512
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+            and rows_attention_supported(n, 1, rank + rd, rank, True)
+            and rows_attention_tile_tokens(n, 16) in ctx.tiles)
+
+
+def latent_query(q: torch.Tensor, uk_t: torch.Tensor, n: int, d: int, rd: int, rot: int, *, positions: torch.Tensor,
+                 freq: torch.Tensor, interleaved: bool) -> torch.Tensor:
+    """``[uk_t[h] q_un, rotate(q_rot)]`` of every head as ``[M, n, rank + rd]`` for up to 16 bfloat16 rows ``q [M, n (d +
+    rd)]`` (``uk_t [n, rank, d]``): the mapping into the latent's space and the rotation in one kernel."""
+    _cuda(q, uk_t, positions, freq)
+    _cols(q, "latent_query")
+    M, rank = q.shape[0], uk_t.shape[1]
+    if (q.shape[1] != n * (d + rd) or tuple(uk_t.shape) != (n, rank, d) or not uk_t.is_contiguous()
+            or q.dtype != torch.bfloat16 or uk_t.dtype != q.dtype):
+        raise KernelError("latent_query: q must be bfloat16 [M, n * (d + rd)] and uk_t contiguous [n, rank, d]")
+    if positions.dtype != torch.int32 or positions.shape != (M,) or (rot and (freq.dtype != torch.float64 or
+                                                                             freq.shape != (rot // 2,))):
+        raise KernelError("latent_query: positions int32 [M], freq float64 [rot / 2]")
+    out = torch.empty((M, n, rank + rd), dtype=q.dtype, device=q.device)
+    lib = _lib("latent_decode")
+    rc = lib.mi_latent_query(_ptr(q), q.stride(0), _ptr(uk_t), M, n, d, rank, rd, int(rot), 1 if interleaved else 0,
+                             _ptr(positions), _ptr(freq), _ptr(out), _stream())
+    _finish(lib, rc, "latent_query")
+    return out
+
+
+def attention_latent_runs(q: torch.Tensor, cache, ctx, n: int, d: int, rank: int, scale: float, *, window: int = 0,
+                          sinks: torch.Tensor | None = None):
+    """``attention_ext`` with ``values_in_keys`` in a step of single tokens, stopped before the runs of keys are merged:
+    returns ``(sums, maxima and denominators, runs, finished rows or None)`` for ``latent_value``."""
+    group = ctx.groups[cache.group]
+    kc, bt = cache.k, group.block_table
+    _cuda(q, kc, sinks)
+    M = ctx.n_tokens
+    if kc.dtype != q.dtype or kc.shape[1:] != (1, group.page_size, d) or not kc.is_contiguous():
+        raise KernelError("attention: the key cache must be contiguous [pages, 1, page_size, d] in q's dtype")
+    _opt_f32(sinks, n, "attention (sinks)")
+    units = M * max(1, -(-n // 16))
+    splits = _rows_attention_runs(ctx, units, int(window), q.device)
+    part_o = part_ml = latent = None
+    if splits > 1:
+        part_o = torch.empty(units * splits * 16 * rank, dtype=torch.float32, device=q.device)
+        part_ml = torch.empty(units * splits * 16 * 2, dtype=torch.float32, device=q.device)
+    else:
+        latent = torch.empty((M, n * rank), dtype=q.dtype, device=q.device)
+    lib = _lib("attention_rows")
+    rc = lib.mi_attention_rows(
+        _ptr(q), q.stride(0), _ptr(latent if latent is not None else q), n * rank, _ptr(kc), None, _ptr(bt), bt.stride(0),
+        _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), None, _ptr(ctx.kv_len), None, None, M,
+        rows_attention_tile_tokens(n, 16), 16, n, 1, d, rank, float(scale), _ptr(sinks), None, 1, splits, _ptr(part_o),
+        _ptr(part_ml), 1, int(window), 0, _stream())
+    _finish(lib, rc, "attention")
+    return part_o, part_ml, splits, latent
+
+
+def latent_value(runs, sinks: torch.Tensor | None, uv: torch.Tensor, out: torch.Tensor, n: int, *,
+                 gate: torch.Tensor | None = None, act: str | None = None, scale: float = 1.0) -> None:
+    """The heads' values ``uv[h] latent`` (``uv [n, dv, rank]``) from what ``attention_latent_runs`` returned: the merge
+    of the runs with the heads' sinks, the expansion, the gate (``[M, n]`` or ``[M, n dv]``) and ``scale`` in one kernel."""
+    part_o, part_ml, splits, latent = runs
+    _cuda(part_o, part_ml, latent, sinks, uv, out, gate)
+    _cols(out, "latent_value")
+    M = out.shape[0]
+    dv, rank = uv.shape[1], uv.shape[2]
+    if uv.shape[0] != n or not uv.is_contiguous() or out.shape[1] != n * dv or out.dtype != torch.bfloat16 or uv.dtype != out.dtype:
+        raise KernelError("latent_value: uv must be contiguous bfloat16 [n, dv, rank] and out [M, n * dv]")
+    if (gate is None) != (act is None):
+        raise KernelError("latent_value: a gate and its activation come together")
+    per_head = 0
+    if gate is not None:
+        _cols(gate, "latent_value")
+        per_head = 1 if gate.shape[1] == n else 0
+        if gate.shape[0] != M or gate.shape[1] not in (n, n * dv) or gate.dtype != out.dtype:
+            raise KernelError("latent_value: the gate must be [M, n] or [M, n * dv]")
+    lib = _lib("latent_decode")
+    rc = lib.mi_latent_value(_ptr(part_o), _ptr(part_ml), splits, _ptr(latent), _ptr(sinks) if splits > 1 else None, _ptr(uv),
+                             M, n, rank, dv, _ptr(gate), gate.stride(0) if gate is not None else 0, per_head, _ACT[act],
+                             float(scale), _ptr(out), out.stride(0), _stream())
+    _finish(lib, rc, "latent_value")
 
 
 # --------------------------------------------------------------------------------------- prompt portions over expanded latents

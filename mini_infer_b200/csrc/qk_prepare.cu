@@ -134,6 +134,8 @@ extern "C" int mi_qk_bias_norm_store(void* packed, int stride, int q_off, int k_
 }
 
 #define LATENT_MAX_ROT 512
+#define LATENT_THREADS 128
+#define LATENT_HELD 8
 
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -150,6 +152,15 @@ latent_prepare_kernel(const T* packed, int stride, int q_off, int nq, int q_head
   const T* row = packed + (size_t)t * stride;
   const int half = rot >> 1;
   const double pos = (double)positions[t];
+  // both latents' elements are asked for first (up to LATENT_HELD per thread stay in registers), then the
+  // angles are worked out while they arrive
+  float qv[LATENT_HELD], cv[LATENT_HELD];
+#pragma unroll
+  for (int j = 0; j < LATENT_HELD; ++j) {
+    const int k = tid + j * LATENT_THREADS;
+    qv[j] = k < cq_rank ? mi_to_float(row[cq_off + k]) : 0.f;
+    cv[j] = c_gain && k < rank ? mi_to_float(row[c_off + k]) : 0.f;
+  }
   for (int i = tid; i < half; i += blockDim.x) {
     // the angle in double precision, brought into [-pi, pi] there; its sine and cosine in fp32
     double a = pos * freq[i];
@@ -159,15 +170,44 @@ latent_prepare_kernel(const T* packed, int stride, int q_off, int nq, int q_head
     sn[i] = s;
     cs[i] = c;
   }
-  if (cq_rank > 0) {                   // the queries' own latent: an RMS norm, the next product's input
-    float sq = 0.f;
-    for (int k = tid; k < cq_rank; k += blockDim.x) {
-      const float v = mi_to_float(row[cq_off + k]);
-      sq += v * v;
+  // sums of squares (fixed order: by thread, then by warp), the queries' latent and the keys' in one reduction
+  float sq = 0.f, ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < LATENT_HELD; ++j) {
+    sq += qv[j] * qv[j];
+    ss += cv[j] * cv[j];
+  }
+  for (int k = tid + LATENT_HELD * LATENT_THREADS; k < cq_rank; k += LATENT_THREADS) {
+    const float v = mi_to_float(row[cq_off + k]);
+    sq += v * v;
+  }
+  if (c_gain)
+    for (int k = tid + LATENT_HELD * LATENT_THREADS; k < rank; k += LATENT_THREADS) {
+      const float v = mi_to_float(row[c_off + k]);
+      ss += v * v;
     }
-    const float m = 1.f / sqrtf(mi_block_sum(sq, red) / (float)cq_rank + eps);
-    for (int k = tid; k < cq_rank; k += blockDim.x)
-      cq_out[(size_t)t * cq_rank + k] = mi_from_float<T>(mi_to_float(row[cq_off + k]) * m * cq_gain[k]);
+  sq = mi_warp_sum(sq);
+  ss = mi_warp_sum(ss);
+  if ((tid & 31) == 0) {
+    red[tid >> 5] = sq;
+    red[16 + (tid >> 5)] = ss;
+  }
+  __syncthreads();                     // the sums, sn and cs are there
+  sq = ss = 0.f;
+#pragma unroll
+  for (int w = 0; w < LATENT_THREADS / 32; ++w) {
+    sq += red[w];
+    ss += red[16 + w];
+  }
+  const float q_mult = 1.f / sqrtf(sq / (float)max(cq_rank, 1) + eps), mult = 1.f / sqrtf(ss / (float)rank + eps);
+  if (cq_rank > 0) {                   // the queries' own latent: the next product's input
+#pragma unroll
+    for (int j = 0; j < LATENT_HELD; ++j) {
+      const int k = tid + j * LATENT_THREADS;
+      if (k < cq_rank) cq_out[(size_t)t * cq_rank + k] = mi_from_float<T>(qv[j] * q_mult * cq_gain[k]);
+    }
+    for (int k = tid + LATENT_HELD * LATENT_THREADS; k < cq_rank; k += LATENT_THREADS)
+      cq_out[(size_t)t * cq_rank + k] = mi_from_float<T>(mi_to_float(row[cq_off + k]) * q_mult * cq_gain[k]);
   }
   // element k of a rotated part: half layout (k with k + half) or interleaved pairs (2i with 2i + 1)
   auto rotated = [&](const T* src, int k) {
@@ -179,17 +219,6 @@ latent_prepare_kernel(const T* packed, int stride, int q_off, int nq, int q_head
     mi_rotate(u, v, sn[i], cs[i], y1, y2);
     return upper ? y2 : y1;
   };
-  // the latent's sum of squares (fixed order: by thread, then by warp)
-  float mult = 0.f;
-  if (c_gain) {
-    float ss = 0.f;
-    for (int k = tid; k < rank; k += blockDim.x) {
-      const float v = mi_to_float(row[c_off + k]);
-      ss += v * v;
-    }
-    mult = 1.f / sqrtf(mi_block_sum(ss, red) / (float)rank + eps);
-  }
-  __syncthreads();                     // sn and cs are there
   constexpr int EPC = 16 / (int)sizeof(T);
   const int dk = rank + rot_dim;
   if (writes) {
@@ -197,7 +226,12 @@ latent_prepare_kernel(const T* packed, int stride, int q_off, int nq, int q_head
     const int page = slot / page_size, offset = slot - page * page_size;
     const int mk = mi_swizzle_mask_rows(dk, (int)sizeof(T));
     T* kdst = kcache + ((size_t)page * page_size + offset) * dk;
-    for (int k = tid; k < rank; k += blockDim.x)
+#pragma unroll
+    for (int j = 0; j < LATENT_HELD; ++j) {
+      const int k = tid + j * LATENT_THREADS;
+      if (k < rank) kdst[mi_swizzled(k, offset, mk, EPC)] = mi_from_float<T>(cv[j] * mult * c_gain[k]);
+    }
+    for (int k = tid + LATENT_HELD * LATENT_THREADS; k < rank; k += LATENT_THREADS)
       kdst[mi_swizzled(k, offset, mk, EPC)] = mi_from_float<T>(mi_to_float(row[c_off + k]) * mult * c_gain[k]);
     const T* kr = row + c_off + rank;
     for (int k = tid; k < rot_dim; k += blockDim.x)

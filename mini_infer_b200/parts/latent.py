@@ -170,6 +170,16 @@ class LatentAttention(ProjectedMixer):
                                **row, **common)
             q = self.uq(cq)
             row = dict(c_gain=None)
+        if ops.latent_decode_fusable(proj.dtype, ctx, n, self.d, self.rd, self.dv, rank, q):
+            # single tokens: mapping and rotation, attention, then merge, expansion and gate, a kernel each
+            if row["c_gain"] is not None:
+                ops.latent_prepare(proj, 0, 0, self.qh, self.d, *sizes, qfull=None, **row, **common)
+            qfull = ops.latent_query(q, self.uk_t, n, self.d, self.rd, self.rot, positions=ctx.positions, freq=self.freq,
+                                     interleaved=self.interleaved)
+            runs = ops.attention_latent_runs(qfull.view(M, n * dk), cache, ctx, n, dk, rank, self.scale,
+                                             window=self.window or 0, sinks=self.sinks)
+            ops.latent_value(runs, self.sinks, self.uv, out, n, gate=gate, act=self.gate, scale=out_scale)
+            return
         heads = torch.empty((M, n * self.dv), dtype=proj.dtype, device=proj.device)
         qfull = torch.empty((M, n, dk), dtype=proj.dtype, device=proj.device) if in_latent_space else None
         if row["c_gain"] is not None or in_latent_space:
