@@ -162,7 +162,8 @@ __global__ void branch_depth_kernel(const BranchDepthArgs a) {
 // The same for rows of up to 4096 channels in whole 16-byte pieces: a thread holds four channels from the first
 // load to the last store, and everything that does not depend on the row's statistics is asked for before them.
 #define ROW_MAX_THREADS 1024
-template <typename T>
+// AVG, CONV: whether the launch averages and convolves (an instance without them needs half the registers).
+template <typename T, bool AVG, bool CONV>
 __global__ void __launch_bounds__(ROW_MAX_THREADS)
 branch_depth_row_kernel(const BranchDepthArgs a) {
   mi_pdl_launch_dependents();
@@ -179,7 +180,7 @@ branch_depth_row_kernel(const BranchDepthArgs a) {
   if (on) {
     if (a.branch) Pack<T, 4>::load(reinterpret_cast<const T*>(a.branch) + (size_t)t * a.branch_stride + k, y);
     Pack<float, 4>::load(a.stream + at, x);
-    if (a.n_prev > 0) {
+    if (AVG) {
       float f[4];
       Pack<float, 4>::load(a.first + at, f);
       const float a0 = a.avg[0];
@@ -221,14 +222,14 @@ branch_depth_row_kernel(const BranchDepthArgs a) {
   }
   if (!on) return;
   if (a.stream_out) Pack<float, 4>::store(a.stream_out + at, x);
-  if (a.n_prev > 0) {
+  if (AVG) {
     const float an = a.avg[a.n_prev];
 #pragma unroll
     for (int i = 0; i < 4; ++i) x[i] = fmaf(an, x[i], acc[i]);
     if (a.avg_out) Pack<float, 4>::store(a.avg_out + at, x);
   }
   if (a.copy) Pack<T, 4>::store(reinterpret_cast<T*>(a.copy) + at, x);
-  if (a.conv_w) {
+  if (CONV) {
     float* tail = a.taps > 1 ? a.conv_state + (size_t)a.state_slot[t] * a.conv_stride + k : nullptr;
     float s[4] = {}, w[4], in[4];
     for (int j = 0; j < a.taps - 1; ++j) {
@@ -270,9 +271,17 @@ extern "C" int mi_branch_depth(const float* stream, const void* branch, int bran
   const int per = vec ? H / 4 : H;
   if (vec && per <= ROW_MAX_THREADS) {      // (the choice depends on the width alone: a row's bits do not depend on the step)
     const int row_threads = (per + 31) / 32 * 32;
-    if (dtype == MI_DTYPE_F32) MI_LAUNCH((branch_depth_row_kernel<float>), M, row_threads, 0, cu_stream, a);
-    else if (dtype == MI_DTYPE_BF16) MI_LAUNCH((branch_depth_row_kernel<bf16>), M, row_threads, 0, cu_stream, a);
+#define MI_ROW(T)                                                                                             \
+  do {                                                                                                        \
+    if (n_prev > 0 && conv_w) MI_LAUNCH((branch_depth_row_kernel<T, true, true>), M, row_threads, 0, cu_stream, a);   \
+    else if (n_prev > 0) MI_LAUNCH((branch_depth_row_kernel<T, true, false>), M, row_threads, 0, cu_stream, a);       \
+    else if (conv_w) MI_LAUNCH((branch_depth_row_kernel<T, false, true>), M, row_threads, 0, cu_stream, a);           \
+    else MI_LAUNCH((branch_depth_row_kernel<T, false, false>), M, row_threads, 0, cu_stream, a);                      \
+  } while (0)
+    if (dtype == MI_DTYPE_F32) MI_ROW(float);
+    else if (dtype == MI_DTYPE_BF16) MI_ROW(bf16);
     else MI_REFUSE("branch_depth: unknown dtype %d", dtype);
+#undef MI_ROW
     MI_RETURN_LAUNCH_STATUS();
   }
   const int threads = per >= 1024 ? 512 : (per >= 256 ? 256 : 128);
