@@ -225,7 +225,8 @@ struct EpilogueFusion {
 // `swiglu` beyond the gated forms: an activation of every value of the product by itself
 #define ACT_XIELU 3
 
-template <typename OutT, bool kFused>
+// kAct: an instance of its own for an activation of single values, so that the others keep their code.
+template <typename OutT, bool kFused, bool kAct>
 __global__ void __launch_bounds__(GT_THREADS, 1)
 gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                 OutT* __restrict__ y, int ldy, int M, int N, int K, int n_tok, int stages, int kb, int chunked, int swiglu,
@@ -421,12 +422,11 @@ gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
           fus.stats_out[tile * FUSED_MAX_TOKENS + etid] =
               (square_sums[0][etid] + square_sums[1][etid]) + (square_sums[2][etid] + square_sums[3][etid]);
         asm volatile("bar.sync 1, 128;\n" ::: "memory");   // the sums are read before the next tile writes them
-      } else if (swiglu == ACT_XIELU) {
+      } else if (kAct) {
         if (n < N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(sizeof(OutT) == 2 ? mi_xielu_bf16(v[j], fus.act_a, fus.act_b)
-                                                                                                : mi_xielu(v[j], fus.act_a, fus.act_b));
+            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(mi_xielu_bf16(v[j], fus.act_a, fus.act_b));
         }
       } else if (swiglu) {
         // rows alternate gate, up: the even lane of a pair has the gate, its neighbour the up
@@ -654,6 +654,8 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
     if (residual && !mi_aligned(residual, 4)) MI_REFUSE("gemm_tma: misaligned residual stream");
   }
   if (swiglu < 0 || swiglu > ACT_XIELU) MI_REFUSE("gemm_tma: unknown activation %d", swiglu);
+  if (swiglu == ACT_XIELU && (stats_in || residual || out_dtype != MI_DTYPE_BF16))
+    MI_REFUSE("gemm_tma: an activation of single values goes with the plain product and a bfloat16 result");
   if (swiglu && swiglu != ACT_XIELU && (N % 2)) MI_REFUSE("gemm_tma: the gate/up epilogue needs an even number of rows of W, got %d", N);
   if (M <= 0 || N <= 0) return 0;
   if (M > MAX_TOKENS) MI_REFUSE("gemm_tma: %d rows of x; this kernel takes at most %d", M, MAX_TOKENS);
@@ -698,9 +700,9 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
   if (!maps_ok)
     MI_REFUSE("gemm_tma: the driver refused a tensor map (N %d, K %d, M %d)", N, K, M);
   cudaError_t e;
-#define GT_LAUNCH(T, FUSED)                                                                                        \
+#define GT_LAUNCH(T, FUSED, ACT)                                                                                        \
   {                                                                                                                \
-    auto kern = gemm_tma_kernel<T, FUSED>;                                                                         \
+    auto kern = gemm_tma_kernel<T, FUSED, ACT>;                                                                         \
     e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                        \
     if (e != cudaSuccess) return (int)e;                                                                           \
     MI_LAUNCH((kern), grid, GT_THREADS, smem, stream, map_w, map_x, (T*)y, (int)ldy, M, N, K, n_tok, stages, kb,   \
@@ -708,10 +710,12 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
   }
   const bool fused = stats_in || residual;
   const int w_evict_first = mi_l2_hints_enabled() ? 1 : 0;
-  if (out_dtype == MI_DTYPE_BF16) {
-    if (fused) GT_LAUNCH(bf16, true) else GT_LAUNCH(bf16, false)
+  if (swiglu == ACT_XIELU && out_dtype == MI_DTYPE_BF16) {
+    GT_LAUNCH(bf16, false, true)
+  } else if (out_dtype == MI_DTYPE_BF16) {
+    if (fused) GT_LAUNCH(bf16, true, false) else GT_LAUNCH(bf16, false, false)
   } else {
-    if (fused) GT_LAUNCH(float, true) else GT_LAUNCH(float, false)
+    if (fused) GT_LAUNCH(float, true, false) else GT_LAUNCH(float, false, false)
   }
 #undef GT_LAUNCH
   MI_RETURN_LAUNCH_STATUS();

@@ -1065,7 +1065,7 @@ def gemm_tma(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bf
     partial, count = _tma_workspace(x.device, int(floats.value), int(counters.value))
     if swiglu and N % 2:
         raise KernelError("gemm_tma: the gate/up epilogue needs an even number of rows")
-    if act is not None and (swiglu or residual is not None):
+    if act is not None and (swiglu or residual is not None or row_stats is not None or out_dtype != torch.bfloat16):
         raise KernelError("gemm_tma: an activation of single values goes with the plain product")
     n_out = N // 2 if swiglu else N
     out = torch.empty((M, n_out), dtype=out_dtype, device=x.device)
