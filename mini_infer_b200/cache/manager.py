@@ -11,7 +11,8 @@ its free list is LIFO as well, ``:570,735-757``).  Groups with a window give pag
 soon as every position in them has fallen out of every future query's window; the table
 keeps ``-1`` there, and kernels never look below the window.  Groups whose queries read their
 own chunk of positions only (``chunk``) give back the pages that lie wholly before the chunk of
-the next position in the same way.
+the next position in the same way.  A window may keep the first positions of a sequence visible
+(``keep_first``): the pages that hold them stay with the request.
 
 *Requests.*  ``add_request`` hands out a stable slot (requests never move when another one
 ends, unlike the reference's ``remove_request`` which shifts indices,
@@ -92,6 +93,7 @@ class GroupSpec:
     window: int | None
     value_dim: int | None = None   # size of a value per head where it differs from head_dim (0: keys only)
     chunk: int | None = None       # queries read the keys of their own chunk of this many positions only
+    keep_first: int = 0            # beside the window, the first positions of the sequence are always read
 
 
 @dataclass
@@ -123,12 +125,12 @@ def group_needs(needs: Sequence) -> list[GroupSpec]:
             continue
         vdim = getattr(n.kv, "value_dim", None)
         key = (n.kv.kv_heads, n.kv.head_dim, n.kv.window, None if vdim in (None, n.kv.head_dim) else vdim,
-               getattr(n.kv, "chunk", None))
+               getattr(n.kv, "chunk", None), getattr(n.kv, "keep_first", 0))
         if key not in members:
             members[key] = []
             order.append(key)
         members[key].append(n.index)
-    return [GroupSpec(tuple(members[k]), k[0], k[1], k[2], k[3], k[4]) for k in order]
+    return [GroupSpec(tuple(members[k]), k[0], k[1], k[2], k[3], k[4], k[5]) for k in order]
 
 
 class CacheManager:
@@ -278,7 +280,8 @@ class CacheManager:
     # ------------------------------------------------------------------ pages
 
     def _window_release_count(self, gi: int, length: int) -> int:
-        """Leading pages of a request holding ``length`` tokens that no future query reads."""
+        """The page up to which (exclusive) no future query of a request holding ``length`` tokens reads, the
+        pages of the first ``keep_first`` positions aside (``_kept_pages``)."""
         g = self.groups[gi]
         first_needed = 0                   # the next query sits at position >= length
         if g.window is not None:
@@ -286,6 +289,10 @@ class CacheManager:
         if g.chunk is not None:            # it reads from the start of its own chunk on
             first_needed = max(first_needed, (length // g.chunk) * g.chunk)
         return first_needed // self.page_size
+
+    def _kept_pages(self, gi: int) -> int:
+        """Leading pages that are never given back before the request ends."""
+        return -(-self.groups[gi].keep_first // self.page_size)
 
     def pages_needed(self, entries: Iterable[tuple[Hashable, int]]) -> list[int]:
         """Pages each group must still hand out for these ``(request, new tokens)``,
@@ -297,7 +304,8 @@ class CacheManager:
             for gi, g in enumerate(self.groups):
                 need[gi] += max(0, want - len(req.tables[gi]))
                 if g.window is not None or g.chunk is not None:
-                    need[gi] -= max(0, self._window_release_count(gi, req.length) - req.released[gi])
+                    need[gi] -= max(0, self._window_release_count(gi, req.length) -
+                                    max(req.released[gi], self._kept_pages(gi)))
         return need
 
     def can_append(self, entries: Iterable[tuple[Hashable, int]]) -> bool:
@@ -337,7 +345,7 @@ class CacheManager:
                 pool = self.pools[gi]
                 table = req.tables[gi]
                 upto = min(self._window_release_count(gi, req.length), len(table))
-                for idx in range(req.released[gi], upto):
+                for idx in range(max(req.released[gi], self._kept_pages(gi)), upto):
                     if table[idx] >= 0:
                         pool.free(table[idx])
                         table[idx] = -1

@@ -11,6 +11,9 @@
 // queries and keys, dv for values and the output); keys of any size that fits in shared memory
 // and values up to 512 are taken, sizes that are no multiple of 4 element by element.
 //
+// `keep` > 0: beside its window a query also sees the first `keep` keys of the sequence; chunks between the two
+// are not walked.  `softcap` > 0: a scaled score s becomes softcap tanh(s / softcap).
+//
 // Three optional extras.  `sinks` [nq]: the softmax's denominator also holds exp(sinks[h]), a
 // score without a key or a value that is not scaled and counts once.  `slopes` [nq]: the scaled
 // score of query i and key j is lowered by slopes[h] * (i - j).  `v_prefix`: there is no value
@@ -44,7 +47,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                          const int* __restrict__ tile_tok0, int nq, int nkv, int d, int dv, float scale,
                          int window, int chunk, const float* __restrict__ sinks, const float* __restrict__ slopes,
-                         int v_prefix) {
+                         int v_prefix, int keep, float softcap) {
   mi_pdl_enter();   // inputs come from the kernels before this one
   extern __shared__ __align__(16) float smem[];
   float* Vs = smem;                       // [BK][dvp], dvp = dv rounded up to 4 (nothing with v_prefix)
@@ -89,12 +92,15 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
   for (int e = 0; e < DMAX / 8; ++e) acc[e] = 0.f;
   const int ne = (dv + 7) >> 3;
 
-  for (int j0 = (j_lo / BK) * BK; j0 < j_end; j0 += BK) {
+  const MiKeyWalk walk(j_lo, keep, BK);
+  const int n_chunks = walk.count(j_end, BK);
+  for (int ci = 0; ci < n_chunks; ++ci) {
+    const int j0 = walk.chunk(ci) * BK;
     __syncthreads();  // previous chunk fully consumed (and Qs written, first time)
     if (tid < BK) {
       const int j = j0 + tid;
       int base = -1;
-      if (j >= j_lo && j < j_end) {
+      if ((j >= j_lo || j < keep) && j < j_end) {
         const int page = block_table[(size_t)trow * bt_stride + j / page_size];
         base = (page * nkv + kvh) * page_size + j % page_size;
       }
@@ -160,8 +166,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
 #pragma unroll
     for (int jj = 0; jj < 4; ++jj) {
       const int j = j0 + c + 8 * jj;
-      const bool ok = (r < rows) && (j <= prow) && (j >= lo_r);
-      s[jj] = ok ? s[jj] * scale - slope * (float)(prow - j) : -INFINITY;
+      const bool ok = (r < rows) && (j <= prow) && (j >= lo_r || j < keep);
+      const float raw = s[jj] * scale;
+      s[jj] = ok ? (softcap > 0.f ? softcap * tanhf(raw / softcap) : raw) - slope * (float)(prow - j) : -INFINITY;
       mx = fmaxf(mx, s[jj]);
     }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -219,7 +226,8 @@ static int launch(const void* q, int q_stride, void* out, int out_stride, const 
                   const void* vcache, const int* block_table, int bt_stride, const int* table_rows, int page_size,
                   const int* q_start, const int* q_len, const int* kv_len, const int* tile_req,
                   const int* tile_tok0, int n_tiles, int nq, int nkv, int d, int dv, float scale, int window,
-                  int chunk, const float* sinks, const float* slopes, int v_prefix, cudaStream_t stream) {
+                  int chunk, const float* sinks, const float* slopes, int v_prefix, int keep, float softcap,
+                  cudaStream_t stream) {
   const size_t smem = ((v_prefix ? 0 : (size_t)BK * ((dv + 3) & ~3)) + (size_t)BQ * d + (size_t)BK * (d + 1) + BQ * BK) *
                           sizeof(float) + 2 * BK * sizeof(int);
   auto kern = attention_generic_kernel<T, DMAX>;
@@ -232,21 +240,23 @@ static int launch(const void* q, int q_stride, void* out, int out_stride, const 
   MI_LAUNCH((kern), grid, NTHREADS, smem, stream, (const T*)q, q_stride, (T*)out, out_stride, (const T*)kcache,
                                          (const T*)vcache, block_table, bt_stride, table_rows, page_size, q_start,
                                          q_len, kv_len, tile_req, tile_tok0, nq, nkv, d, dv, scale, window, chunk, sinks,
-                                         slopes, v_prefix);
+                                         slopes, v_prefix, keep, softcap);
   return 0;
 }
 
 extern "C" int mi_attention_generic_tile_tokens() { return BQ; }
 
-extern "C" int mi_attention_generic_masked(const void* q, int q_stride, void* out, int out_stride,
+extern "C" int mi_attention_generic_capped(const void* q, int q_stride, void* out, int out_stride,
                                            const void* kcache, const void* vcache, const int* block_table,
                                            int bt_stride, const int* table_rows, int page_size, const int* q_start,
                                            const int* q_len, const int* kv_len, const int* tile_req,
                                            const int* tile_tok0, int n_tiles, int nq, int nkv, int d, int dv,
-                                           float scale, int window, int chunk, const float* sinks,
-                                           const float* slopes, int v_prefix, int dtype, cudaStream_t stream) {
+                                           float scale, int window, int chunk, int keep, float softcap,
+                                           const float* sinks, const float* slopes, int v_prefix, int dtype,
+                                           cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (chunk < 0) MI_REFUSE("attention: bad chunk size %d", chunk);
+  if (keep < 0 || (keep && chunk) || !(softcap >= 0.f)) MI_REFUSE("attention: bad kept keys %d or cap %f", keep, softcap);
   if (d <= 0 || d > 1024 || dv <= 0 || dv > 512)
     MI_REFUSE("attention: head sizes %d (keys, up to 1024) and %d (values, up to 512) are not taken", d, dv);
   if (v_prefix && dv > d) MI_REFUSE("attention: values of %d cannot be the first columns of keys of %d", dv, d);
@@ -260,7 +270,7 @@ extern "C" int mi_attention_generic_masked(const void* q, int q_stride, void* ou
 #define MI_GO(T, DMAX)                                                                              \
   rc = launch<T, DMAX>(q, q_stride, out, out_stride, kcache, vcache, block_table, bt_stride,        \
                        table_rows, page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles, nq, nkv, d, dv, \
-                       scale, window, chunk, sinks, slopes, v_prefix, stream)
+                       scale, window, chunk, sinks, slopes, v_prefix, keep, softcap, stream)
   if (dtype == MI_DTYPE_F32) {
     if (dv <= 64) MI_GO(float, 64);
     else if (dv <= 128) MI_GO(float, 128);
@@ -278,6 +288,18 @@ extern "C" int mi_attention_generic_masked(const void* q, int q_stride, void* ou
   if (rc == MI_REFUSED - 1) MI_REFUSE("attention: keys of %d and values of %d do not fit in shared memory", d, dv);
   if (rc) return rc;
   MI_RETURN_LAUNCH_STATUS();
+}
+
+extern "C" int mi_attention_generic_masked(const void* q, int q_stride, void* out, int out_stride,
+                                           const void* kcache, const void* vcache, const int* block_table,
+                                           int bt_stride, const int* table_rows, int page_size, const int* q_start,
+                                           const int* q_len, const int* kv_len, const int* tile_req,
+                                           const int* tile_tok0, int n_tiles, int nq, int nkv, int d, int dv,
+                                           float scale, int window, int chunk, const float* sinks,
+                                           const float* slopes, int v_prefix, int dtype, cudaStream_t stream) {
+  return mi_attention_generic_capped(q, q_stride, out, out_stride, kcache, vcache, block_table, bt_stride, table_rows,
+                                     page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles, nq, nkv, d, dv,
+                                     scale, window, chunk, 0, 0.f, sinks, slopes, v_prefix, dtype, stream);
 }
 
 extern "C" int mi_attention_generic_ext(const void* q, int q_stride, void* out, int out_stride,

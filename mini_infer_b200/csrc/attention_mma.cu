@@ -17,7 +17,9 @@
 //
 // A query at absolute position p sees keys j with first_visible(p, window) <= j <= p: with window > 0 the
 // last `window` positions, with window < 0 its own chunk of -window positions (chunks counted from
-// position 0), with window = 0 all of them.
+// position 0), with window = 0 all of them.  With `keep` > 0 (the balanced decode and the prefill kernel) the
+// first `keep` keys of the sequence are seen as well; with cap_k > 0 a raw score s counts as cap_h tanh(s cap_k)
+// (cap_k = scale / cap, cap_h = cap log2 e: exponents to base two) instead of s scale log2 e.
 // Layouts are those of attention_generic.cu (cache pages are [nkv, page_size, d], so the keys of a
 // page lie together per key/value head and a 64-key chunk is read as a few long runs).
 #include "common.cuh"
@@ -219,14 +221,14 @@ __device__ __forceinline__ void consumer_barrier(int count) {
 }
 
 template <int THREADS, bool NAMED = false>
-__device__ __forceinline__ void zero_masked_values(bf16* vtile, int chunk, int lo, int hi, int d) {
+__device__ __forceinline__ void zero_masked_values(bf16* vtile, int chunk, int lo, int hi, int d, int keep = 0) {
   const int cb = chunk * KCHUNK;
-  if (cb >= lo && cb + KCHUNK <= hi) return;   // uniform over the calling threads
+  if ((cb >= lo || cb + KCHUNK <= keep) && cb + KCHUNK <= hi) return;   // uniform over the calling threads
   const int units = d >> 3;
   for (int idx = threadIdx.x; idx < KCHUNK * units; idx += THREADS) {
     const int r = idx / units, u = idx - r * units;
     const int j = cb + r;
-    if (j < lo || j >= hi) *reinterpret_cast<uint4*>(vtile + r * d + u * 8) = make_uint4(0u, 0u, 0u, 0u);
+    if ((j < lo && j >= keep) || j >= hi) *reinterpret_cast<uint4*>(vtile + r * d + u * 8) = make_uint4(0u, 0u, 0u, 0u);
   }
   fence_proxy_async();   // these writes come before the copy engine's next writes to the tile
   if (NAMED) consumer_barrier(THREADS);
@@ -761,7 +763,7 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
                                  int nkv, int d, float scale, int window, int min_chunks, int unit_cost,
                                  float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                                  int* __restrict__ status, const float* __restrict__ rope_cs, int store_kv,
-                                 const float* __restrict__ sinks) {
+                                 const float* __restrict__ sinks, int keep, float cap_k, float cap_h) {
   // sinks [nq] (optional): per head a score that joins the softmax's denominator with neither key nor value.
   // ROPE (the head size is then DMAX exactly): rope_cs holds per query token [d / 2] sines then
   // [d / 2] cosines of its rotary angles; q arrives un-rotated and is rotated here, in registers; and with store_kv
@@ -791,7 +793,7 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
   for (int b = tid; b < B; b += (ROPE ? BAL_THREADS : DEC_THREADS)) {
     const int kl = kv_len[b];
     const int lo = first_visible(kl - 1, window);   // (a window skips the chunks below it)
-    cum[b + 1] = (kl + KCHUNK - 1) / KCHUNK - lo / KCHUNK;
+    cum[b + 1] = MiKeyWalk(lo, keep, KCHUNK).count(kl, KCHUNK);
   }
   __syncthreads();
   if (warp == 0) {
@@ -855,10 +857,12 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
       const int len = balanced_part(i, i1, cum, B, U, ov, b, u, c_rel, seg, n_b);
       const int kvh = u / hblocks;
       const int kl = kv_len[b];
-      const int lo = first_visible(kl - 1, window);
+      const int lo_w = first_visible(kl - 1, window);
+      const MiKeyWalk walk(lo_w, keep, KCHUNK);
       const int* table = block_table + (size_t)(table_rows ? table_rows[b] : b) * bt_stride;
       for (int s = 0; s < seg && ok; ++s, ++it) {
-        const int c = lo / KCHUNK + c_rel + s, st = it % DEC_STAGES;
+        const int c = walk.chunk(c_rel + s), st = it % DEC_STAGES;
+        const int lo = c * KCHUNK < keep ? 0 : lo_w;     // a chunk with kept keys is copied from its beginning
         if (it >= DEC_STAGES)
           ok = __all_sync(0xffffffffu, mbar_wait_bounded(&empty[st], ((it / DEC_STAGES) - 1) & 1, status));
         if (!ok) break;
@@ -958,6 +962,7 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
     const int head0 = kvh * g + hb * DEC_HEADS;
     const int kl = kv_len[b], tok = q_start[b];
     const int lo = first_visible(kl - 1, window);
+    const MiKeyWalk walk(lo, keep, KCHUNK);
 
     // Q as the B operand: lane (qd, t4) holds head qd, dims ks*16 + 2*t4 + {0,1} and + 8
     uint32_t qb[DMAX / 16][2];
@@ -990,21 +995,21 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
     for (int k = 0; k < DMAX / 16; ++k) o[k][0] = o[k][1] = o[k][2] = o[k][3] = 0.f;
 
     for (int s = 0; s < seg; ++s, ++it) {
-      const int c = lo / KCHUNK + c_rel + s, buf = it % DEC_STAGES;
+      const int c = walk.chunk(c_rel + s), buf = it % DEC_STAGES;
       const bool arrived =
           !warp_dead && __all_sync(0xffffffffu, mbar_wait_bounded(&bars[buf], (it / DEC_STAGES) & 1, status));
       if (!arrived && !warp_dead) {
         warp_dead = true;
         if (lane == 0) dead = 1;
       }
-      zero_masked_values<NTHREADS, true>(Vs + buf * KCHUNK * d, c, lo, kl, d);
+      zero_masked_values<NTHREADS, true>(Vs + buf * KCHUNK * d, c, lo, kl, d, keep);
       const int key0 = c * KCHUNK + warp * 16;
       const int kr = lane & 15, vr = (lane & 7) + (lane >> 4) * 8;
       const int ksw = inpage_of(key0 + kr, page_size, page_shift) & swz_mask;
       const int vsw = inpage_of(key0 + vr, page_size, page_shift) & swz_mask;
       const bf16* Kb = Ks + buf * KCHUNK * d + (warp * 16 + kr) * d;
       const bf16* Vb = Vs + buf * KCHUNK * d + (warp * 16 + vr) * d;
-      if (arrived && key0 < kl && key0 + 16 > lo) {   // (the arithmetic of attention_decode_kernel)
+      if (arrived && key0 < kl && (key0 + 16 > lo || key0 < keep)) {   // (the arithmetic of attention_decode_kernel)
         constexpr int GROUP = (DMAX / 16) < 8 ? (DMAX / 16) : 8;
         float sa[4] = {0.f, 0.f, 0.f, 0.f}, s_odd[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -1027,11 +1032,18 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
         for (int k = 0; k < GROUP; ++k)
           if (k < ksteps) ldmatrix_x4_trans(vf[k], Vb + (((k * 2 + ((lane >> 3) & 1)) ^ vsw) << 3));
         const int j0 = key0 + qd, j1 = j0 + 8;
-        const bool ok0 = j0 < kl && j0 >= lo, ok1 = j1 < kl && j1 >= lo;
-        sa[0] = ok0 ? sa[0] * sc : -INFINITY;
-        sa[1] = ok0 ? sa[1] * sc : -INFINITY;
-        sa[2] = ok1 ? sa[2] * sc : -INFINITY;
-        sa[3] = ok1 ? sa[3] * sc : -INFINITY;
+        const bool ok0 = j0 < kl && (j0 >= lo || j0 < keep), ok1 = j1 < kl && (j1 >= lo || j1 < keep);
+        if (cap_k > 0.f) {   // (the same for the whole launch)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sa[e] = mi_softcap(sa[e], cap_k, cap_h);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) sa[e] *= sc;
+        }
+        sa[0] = ok0 ? sa[0] : -INFINITY;
+        sa[1] = ok0 ? sa[1] : -INFINITY;
+        sa[2] = ok1 ? sa[2] : -INFINITY;
+        sa[3] = ok1 ? sa[3] : -INFINITY;
         float alpha[2], p[4];
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
@@ -1198,7 +1210,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                          const int* __restrict__ q_start, const int* __restrict__ q_len,
                          const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                          const int* __restrict__ tile_tok0, int nq, int nkv, int d, float scale, int window,
-                         int gb, int tt, int* __restrict__ status) {
+                         int gb, int tt, int* __restrict__ status, int keep, float cap_k, float cap_h) {
   constexpr int MT = PrefillShape<DMAX>::MT;
   constexpr int THREADS = PrefillShape<DMAX>::THREADS;
   mi_pdl_enter();   // inputs come from the kernels before this one
@@ -1270,9 +1282,12 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
 #pragma unroll
     for (int i = 0; i < DMAX / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
   }
-  const float sc = scale * LOG2E;
+  const float sc = cap_k > 0.f ? 1.f : scale * LOG2E;   // capped scores are exponents already
   const int ksteps = d >> 4;
-  const int c0 = lo / KCHUNK, c1 = (hi + KCHUNK - 1) / KCHUNK;
+  const MiKeyWalk walk(lo, keep, KCHUNK);
+  const int n_chunks = walk.count(hi, KCHUNK);
+  const int c0 = walk.chunk(0);
+  auto load_lo = [&](int c) { return c * KCHUNK < keep ? 0 : lo; };   // a chunk with kept keys is copied from its beginning
   const uint32_t q_addr = smem_u32(Qs) + (uint32_t)((row0 + (lane & 15)) * sd + (lane >> 4) * 8) * 2u;
 
   __shared__ __align__(8) uint64_t bars[2];
@@ -1283,23 +1298,24 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
   }
   __syncthreads();
   PageLoader loader;
-  loader.fetch(table, page_size, page_shift, c0, lo, hi);
-  if (tid == 0) mbar_expect_tx(&bars[0], PageLoader::chunk_bytes(c0, lo, hi, d, page_size, page_shift));
+  loader.fetch(table, page_size, page_shift, c0, load_lo(c0), hi);
+  if (tid == 0) mbar_expect_tx(&bars[0], PageLoader::chunk_bytes(c0, load_lo(c0), hi, d, page_size, page_shift));
   loader.issue(Ks, Vs, kcache, vcache, page_size, page_shift, c0, nkv, kvh, d, &bars[0]);
-  if (c0 + 1 < c1) loader.fetch(table, page_size, page_shift, c0 + 1, lo, hi);
+  if (n_chunks > 1) loader.fetch(table, page_size, page_shift, walk.chunk(1), load_lo(walk.chunk(1)), hi);
   __syncthreads();   // the query tile is visible to every warp
 
-  for (int c = c0; c < c1; ++c) {
-    const int buf = (c - c0) & 1;
-    if (c + 1 < c1) {
+  for (int it = 0; it < n_chunks; ++it) {
+    const int c = walk.chunk(it), buf = it & 1;
+    if (it + 1 < n_chunks) {
+      const int cn = walk.chunk(it + 1);
       if (tid == 0)
-        mbar_expect_tx(&bars[buf ^ 1], PageLoader::chunk_bytes(c + 1, lo, hi, d, page_size, page_shift));
+        mbar_expect_tx(&bars[buf ^ 1], PageLoader::chunk_bytes(cn, load_lo(cn), hi, d, page_size, page_shift));
       loader.issue(Ks + (buf ^ 1) * KCHUNK * d, Vs + (buf ^ 1) * KCHUNK * d, kcache, vcache, page_size, page_shift,
-                   c + 1, nkv, kvh, d, &bars[buf ^ 1]);
-      if (c + 2 < c1) loader.fetch(table, page_size, page_shift, c + 2, lo, hi);
+                   cn, nkv, kvh, d, &bars[buf ^ 1]);
+      if (it + 2 < n_chunks) loader.fetch(table, page_size, page_shift, walk.chunk(it + 2), load_lo(walk.chunk(it + 2)), hi);
     }
-    const bool arrived = __all_sync(0xffffffffu, mbar_wait_bounded(&bars[buf], ((c - c0) >> 1) & 1, status));
-    zero_masked_values<THREADS>(Vs + buf * KCHUNK * d, c, lo, hi, d);
+    const bool arrived = __all_sync(0xffffffffu, mbar_wait_bounded(&bars[buf], (it >> 1) & 1, status));
+    zero_masked_values<THREADS>(Vs + buf * KCHUNK * d, c, lo, hi, d, keep);
     const bf16* Kb = Ks + buf * KCHUNK * d;
     const bf16* Vb = Vs + buf * KCHUNK * d;
     const int key0 = c * KCHUNK;
@@ -1322,7 +1338,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         vxor[i] = (uint32_t)((vsw & ~1) << 4);
       }
     }
-    if (arrived && warp_active && key0 < warp_hi && key0 + KCHUNK > warp_lo) {
+    if (arrived && warp_active && key0 < warp_hi && (key0 + KCHUNK > warp_lo || key0 < keep)) {
       float s[MT][8][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
@@ -1352,9 +1368,15 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       // few on the diagonal and at a window's edge) needs no mask.  Scores stay unscaled; the
       // scale is folded into the exponent's multiply-add: p = 2^(s * sc - m), m = sc * max(s).
       const bool interior = key0 + KCHUNK - 1 <= p_first + wt0 &&
-                            key0 >= first_visible(p_first + wt1, window);
+                            (key0 >= first_visible(p_first + wt1, window) || key0 + KCHUNK <= keep);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
+        if (cap_k > 0.f) {   // (the same for the whole launch)
+#pragma unroll
+          for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[mt][nt][e] = mi_softcap(s[mt][nt][e], cap_k, cap_h);
+        }
         if (!interior) {
 #pragma unroll
           for (int nt = 0; nt < 8; ++nt)
@@ -1362,7 +1384,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
             for (int e = 0; e < 4; ++e) {
               const int hr = e >> 1;
               const int j = key0 + nt * 8 + 2 * t4 + (e & 1);
-              if (!(rvalid[mt][hr] && j <= prow[mt][hr] && j >= lorow[mt][hr])) s[mt][nt][e] = -INFINITY;
+              if (!(rvalid[mt][hr] && j <= prow[mt][hr] && (j >= lorow[mt][hr] || j < keep))) s[mt][nt][e] = -INFINITY;
             }
         }
         // both rows of the lane side by side and sums in four strands: short dependency chains
@@ -1629,9 +1651,11 @@ extern "C" int mi_attention_decode_balanced(const void* q, int q_stride, void* o
                                             const int* table_rows, int page_size, const int* q_start,
                                             const int* kv_len, int B, int nq, int nkv, int d, float scale, int window,
                                             int grid, float* part_o, float* part_ml, int* counters,
-                                            const float* rope_cs, int store_kv, const float* sinks,
-                                            cudaStream_t stream) {
+                                            const float* rope_cs, int store_kv, const float* sinks, int keep,
+                                            float softcap, cudaStream_t stream) {
   if (B <= 0) return 0;
+  if (keep < 0 || (keep && window < 0) || !(softcap >= 0.f)) MI_REFUSE("attention: bad kept keys %d or cap %f", keep, softcap);
+  const float cap_k = softcap > 0.f ? scale / softcap : 0.f, cap_h = softcap * LOG2E;
   if (rope_cs && ((d != 64 && d != 128 && d != 256) || !mi_aligned(rope_cs, 4)))
     MI_REFUSE("attention: rotating inside the decode kernel needs a head size of 64, 128 or 256, got %d", d);
   if (int rc = check_common(q, q_stride, out, out_stride, kcache, vcache, nq, nkv, d, page_size, window)) return rc;
@@ -1651,7 +1675,8 @@ extern "C" int mi_attention_decode_balanced(const void* q, int q_stride, void* o
     MI_LAUNCH((kern), grid, ROPE ? BAL_THREADS : DEC_THREADS, smem, stream, (const bf16*)q, q_stride,     \
               (bf16*)out, out_stride, (const bf16*)kcache, (const bf16*)vcache, block_table, bt_stride,   \
               table_rows, page_size, page_shift, q_start, kv_len, B, nq, nkv, d, scale, window, 4,        \
-              g_unit_cost, part_o, part_ml, counters, wait_status_ptr(), rope_cs, store_kv, sinks);       \
+              g_unit_cost, part_o, part_ml, counters, wait_status_ptr(), rope_cs, store_kv, sinks, keep,  \
+              cap_k, cap_h);                                                                              \
   } while (0)
   if (rope_cs) {
     if (d == 64) MI_DECODE_BAL(64, true);
@@ -1670,12 +1695,15 @@ extern "C" int mi_attention_prefill_tile_tokens(int g) {
   return PROWS / gb;
 }
 
-extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
+extern "C" int mi_attention_prefill_capped(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
                                     const void* vcache, const int* block_table, int bt_stride, const int* table_rows,
                                     int page_size, const int* q_start, const int* q_len, const int* kv_len,
                                     const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens,
-                                    int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
+                                    int nq, int nkv, int d, float scale, int window, int keep, float softcap,
+                                    cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
+  if (keep < 0 || (keep && window < 0) || !(softcap >= 0.f)) MI_REFUSE("attention: bad kept keys %d or cap %f", keep, softcap);
+  const float cap_k = softcap > 0.f ? scale / softcap : 0.f, cap_h = softcap * LOG2E;
   if (int rc = check_common(q, q_stride, out, out_stride, kcache, vcache, nq, nkv, d, page_size, window)) return rc;
   if (!(scale > 0.f)) MI_REFUSE("attention: the score scale must be positive (the row maximum is taken before scaling)");
   const int g = nq / nkv;
@@ -1697,13 +1725,23 @@ extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int 
                                            (const bf16*)kcache, (const bf16*)vcache, block_table,       \
                                            bt_stride, table_rows, page_size, page_shift, q_start, q_len, kv_len,    \
                                            tile_req, tile_tok0, nq, nkv, d, scale, window, gb,          \
-                                           PROWS / gb, wait_status_ptr());                              \
+                                           PROWS / gb, wait_status_ptr(), keep, cap_k, cap_h);          \
   } while (0)
   if (d <= 64) MI_PREFILL(64);
   else if (d <= 128) MI_PREFILL(128);
   else MI_PREFILL(256);
 #undef MI_PREFILL
   MI_RETURN_LAUNCH_STATUS();
+}
+
+extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
+                                    const void* vcache, const int* block_table, int bt_stride, const int* table_rows,
+                                    int page_size, const int* q_start, const int* q_len, const int* kv_len,
+                                    const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens,
+                                    int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
+  return mi_attention_prefill_capped(q, q_stride, out, out_stride, kcache, vcache, block_table, bt_stride, table_rows,
+                                     page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles, tile_tokens, nq,
+                                     nkv, d, scale, window, 0, 0.f, stream);
 }
 
 // ------------------------------------------------------------------------------- no allocation

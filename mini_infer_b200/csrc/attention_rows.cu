@@ -5,7 +5,8 @@
 // head.  Prompt portions and single decoded tokens alike.
 //
 // With `window` > 0 a query at position p sees the keys j > p - window only; chunks wholly before the
-// tile's first window are not walked.
+// tile's first window are not walked.  With `keep` > 0 the first `keep` keys of the sequence are seen as well
+// (their chunks come first in the walk).  `softcap` > 0: a scaled score s becomes softcap tanh(s / softcap).
 //
 // A block takes R = 16 MT query rows that share one key/value head (MT = 1: four warps, for steps of
 // single tokens; MT = 2 or 4: eight or sixteen warps, for prompt portions, with two buffers for the
@@ -127,7 +128,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
                       const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                       const int* __restrict__ tile_tok0, int tile_tokens, int nq, int nkv, int d, int dv, float scale,
                       const float* __restrict__ sinks, const float* __restrict__ slopes, int v_prefix,
-                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window) {
+                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep,
+                      float softcap) {
   mi_pdl_enter();
   constexpr int R = ROWS * MT, NW = QUARTERS * MT, NT = NW * 32;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -166,9 +168,10 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   auto row_head = [&](int r) { return rows.head(r); };
   // this block's run of keys: whole chunks, the same cut for every row of the tile
   const int j_lo = window > 0 ? max(0, p0 - window + 1) : 0;    // the first key that any row sees
-  const int chunk0 = j_lo / CHUNK;
-  const int chunks_all = (j_end + CHUNK - 1) / CHUNK - chunk0, chunks_mine = (chunks_all + n_splits - 1) / n_splits;
-  const int j_begin = (chunk0 + split * chunks_mine) * CHUNK, j_stop = min(j_end, (chunk0 + (split + 1) * chunks_mine) * CHUNK);
+  const MiKeyWalk walk(j_lo, keep, CHUNK);
+  const int chunks_all = walk.count(j_end, CHUNK), chunks_mine = (chunks_all + n_splits - 1) / n_splits;
+  const int i_begin = split * chunks_mine, i_stop = min(chunks_all, (split + 1) * chunks_mine);
+  const float cap_k = softcap > 0.f ? scale / softcap : 0.f;
 
   // ---- the queries: 16-byte pieces, zero for rows without a token
   const int pieces = d >> 3;
@@ -195,12 +198,12 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   const int ntiles_v = (dv / QUARTERS) >> 3;
   const int mk = mi_swizzle_mask_rows(d, 2), mv = mi_swizzle_mask_rows(dv, 2);
   const int vpitch = v_prefix ? dp : dvp;
-  // where the 64 keys from j0 on lie in the cache (threads 0..63), into list `which`
-  auto list_rows = [&](int j0, int which) {
+  // where the 64 keys of the walk's chunk i lie in the cache (threads 0..63), into list `which`
+  auto list_rows = [&](int i, int which) {
     if (tid < CHUNK) {
-      const int j = j0 + tid;
+      const int j = walk.chunk(i) * CHUNK + tid;
       int base = -1;
-      if (j >= j_lo && j < j_stop) {
+      if (i < i_stop && j < j_end && (j >= j_lo || j < keep)) {
         const int page = block_table[(size_t)trow * bt_stride + j / page_size];
         base = (page * nkv + kvh) * page_size + j % page_size;
       }
@@ -215,26 +218,27 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
       gather_rows_async<NT>(kdst + CHUNK * dp, dvp, vcache, dv, mv, rowbase_all + which * CHUNK, rowoff_all + which * CHUNK, tid);
     cp_async_commit();
   };
-  if (DB && j_begin < j_stop) {
-    list_rows(j_begin, 0);
+  if (DB && i_begin < i_stop) {
+    list_rows(i_begin, 0);
     __syncthreads();
     copy_chunk(0);
-    list_rows(j_begin + CHUNK, 1);
+    list_rows(i_begin + 1, 1);
   }
 
   int it = 0;
-  for (int j0 = j_begin; j0 < j_stop; j0 += CHUNK, ++it) {
+  for (int i = i_begin; i < i_stop; ++i, ++it) {
+    const int j0 = walk.chunk(i) * CHUNK;
     const int cur = DB ? (it & 1) : 0;
     const bf16* Ks = KV + cur * stage_elems;
     const bf16* Vrows = v_prefix ? Ks : Ks + CHUNK * dp;
     if (DB) {
       cp_async_wait_all();
       __syncthreads();          // this chunk has landed, the next one's rows are listed, the chunk before is consumed
-      if (j0 + CHUNK < j_stop) copy_chunk(cur ^ 1);
-      list_rows(j0 + 2 * CHUNK, cur);      // read after the next iteration's barrier (this chunk's list has done its work)
+      if (i + 1 < i_stop) copy_chunk(cur ^ 1);
+      list_rows(i + 2, cur);      // read after the next iteration's barrier (this chunk's list has done its work)
     } else {
       __syncthreads();                                          // the chunk before is consumed (first time: Qs written)
-      list_rows(j0, 0);
+      list_rows(i, 0);
       __syncthreads();
       bf16* kdst = KV;
       if (MT == 1) {     // few warps: every piece of the chunk is asked for at once (cp.async)
@@ -276,8 +280,10 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
         const int j = j0 + warp * 16 + n * 8 + 2 * t4 + (e & 1);
         const bool hi = e >= 2;
         const int pos = hi ? pos_hi : pos_lo;
-        const bool ok = (hi ? ok_hi : ok_lo) && (unsigned)(pos - j) < span;      // not behind the query, not before its window
-        const float v = ok ? (s[n][e] * scale - (hi ? slope_hi : slope_lo) * (float)(pos - j)) * LOG2E : -INFINITY;
+        // not behind the query; not before its window, unless it is one of the kept first keys
+        const bool ok = (hi ? ok_hi : ok_lo) && ((unsigned)(pos - j) < span || (j < keep && j <= pos));
+        const float raw = softcap > 0.f ? mi_softcap(s[n][e], cap_k, softcap) : s[n][e] * scale;
+        const float v = ok ? (raw - (hi ? slope_hi : slope_lo) * (float)(pos - j)) * LOG2E : -INFINITY;
         s[n][e] = v;
         if (hi) mx_hi = fmaxf(mx_hi, v); else mx_lo = fmaxf(mx_lo, v);
       }
@@ -509,7 +515,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
                                  const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens, int rows,
                                  int nq, int nkv, int d, int dv, float scale, const float* sinks, const float* slopes,
                                  int v_prefix, int n_splits, float* part_o, float* part_ml, int stages,
-                                 int window, int merge, cudaStream_t stream) {
+                                 int window, int merge, int keep, float softcap, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   if (stages != 1 && stages != 2) MI_REFUSE("attention_rows: one or two buffers for a chunk, not %d", stages);
   if ((rows == 2 * ROWS && stages != 2) || (rows == ROWS && stages != 1))
@@ -520,6 +526,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
   if (!mi_attention_rows_tile_tokens(G, rows) || tile_tokens != mi_attention_rows_tile_tokens(G, rows))
     MI_REFUSE("attention_rows: tiles of %d tokens and %d rows do not fit a group of %d heads", tile_tokens, rows, G);
   if (page_size <= 0 || window < 0) MI_REFUSE("attention_rows: bad page size %d or window %d", page_size, window);
+  if (keep < 0 || !(softcap >= 0.f)) MI_REFUSE("attention_rows: bad kept keys %d or cap %f", keep, softcap);
   if (!v_prefix && !vcache) MI_REFUSE("attention_rows: no value cache");
   if (n_splits < 1 || n_splits > MERGE_MAX_SPLITS || (n_splits > 1 && (!part_o || !part_ml)))
     MI_REFUSE("attention_rows: 1 to %d runs of keys, and scratch for more than one", MERGE_MAX_SPLITS);
@@ -544,7 +551,7 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
     MI_LAUNCH(kern, (unsigned)blocks, QUARTERS * MT * 32, smem, stream, (const bf16*)q, q_stride, (bf16*)out,    \
               out_stride, (const bf16*)kcache, (const bf16*)vcache, block_table, bt_stride, table_rows, page_size, \
               q_start, q_len, kv_len, tile_req, tile_tok0, tile_tokens, nq, nkv, d, dv, scale, sinks, slopes,    \
-              v_prefix, n_splits, part_o, part_ml, window);                                                     \
+              v_prefix, n_splits, part_o, part_ml, window, keep, softcap);                                                     \
   } while (0)
   if (rows == ROWS) {
     if (dv <= 128) MI_GO(32, 1, false);

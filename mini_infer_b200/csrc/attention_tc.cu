@@ -228,6 +228,35 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// A row of 64 raw scores s to cap_h tanh(s cap_k).  Scores far below the cap (the whole warp's) take the
+// polynomial in the two-wide instructions, six per pair; others the exponential form.
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ void cap_scores(float (&s)[64], float cap_k, float cap_h) {
+  float m4[4];
+#pragma unroll
+  for (int j = 0; j < 64; j += 2) m4[j >> 4] = (j & 15) ? max3(m4[j >> 4], fabsf(s[j]), fabsf(s[j + 1])) : fmaxf(fabsf(s[j]), fabsf(s[j + 1]));
+  const float largest = fmaxf(max3(m4[0], m4[1], m4[2]), m4[3]) * cap_k;
+  if (__all_sync(0xffffffffu, largest <= MI_TANH_POLY)) {
+    // the factors ride in the coefficients: y = s (c0 + z (c1 + z (c2 + z (c3 + z c4)))), z = s^2
+    const float k1 = cap_h * cap_k, k2 = cap_k * cap_k;
+    const float c0 = MI_TANH_C0 * k1, c1 = MI_TANH_C1 * k1 * k2, c2 = MI_TANH_C2 * k1 * k2 * k2,
+                c3 = MI_TANH_C3 * k1 * k2 * k2 * k2, c4 = MI_TANH_C4 * k1 * k2 * k2 * k2 * k2;
+    const uint64_t p0 = pair_of(c0, c0), p1 = pair_of(c1, c1), p2 = pair_of(c2, c2), p3 = pair_of(c3, c3), p4 = pair_of(c4, c4);
+#pragma unroll
+    for (int j = 0; j < 64; j += 2) {
+      const uint64_t x = pair_of(s[j], s[j + 1]), z = mul2(x, x);
+      unpair(mul2(x, fma2(fma2(fma2(fma2(p4, z, p3), z, p2), z, p1), z, p0)), s[j], s[j + 1]);
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 64; ++j) s[j] = mi_softcap(s[j], cap_k, cap_h);
+  }
+}
+
 // barriers of the block, in one array
 #ifndef NTILE
 #define NTILE 1    // query tiles of 128 rows per block
@@ -253,6 +282,9 @@ enum {
   B_COUNT = 4 * NSTAGE + 12
 };
 
+// CAPPED (with cap_k > 0): a raw score s counts as cap_h tanh(s cap_k), in the exponents' units, before the mask.
+// keep > 0: beside its window a row also sees the first `keep` keys of the sequence.
+template <bool CAPPED>
 __global__ void __launch_bounds__(TC_THREADS, 2 / NTILE)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
@@ -261,7 +293,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             const int* __restrict__ q_start, const int* __restrict__ q_len,
                             const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                             const int* __restrict__ tile_tok0, int nq, int nkv, int d, float scale, int window,
-                            int chunk, int gb, int tt, const float* __restrict__ sinks, const float* __restrict__ slopes) {
+                            int chunk, int gb, int tt, const float* __restrict__ sinks, const float* __restrict__ slopes,
+                            int keep, float cap_k, float cap_h) {
   mi_pdl_enter();   // inputs come from the kernels before this one
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -293,8 +326,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   int lo = window > 0 ? max(0, p_first - window + 1) : 0;
   if (chunk > 0) lo = max(lo, (p_first / chunk) * chunk);
   const int heads_here = min(gb, g - hb * gb);
-  const int c0 = lo / KC, c1 = (hi + KC - 1) / KC;
-  const int n_chunks = c1 - c0;
+  const MiKeyWalk walk(lo, keep, KC);
+  const int n_chunks = walk.count(hi, KC);
   volatile int* gu = &give_up;
 
   if (tid == 0) {
@@ -365,7 +398,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     unsigned char* ring = is_v ? Vs : Ks;
     const int full0 = is_v ? B_VFULL : B_KFULL, empty0 = is_v ? B_VEMPTY : B_KEMPTY;
     auto page_of = [&](int it) -> int {
-      const int key = (c0 + it) * KC + (lane << page_shift);
+      const int key = walk.chunk(it) * KC + (lane << page_shift);
       return (it < n_chunks && lane < ppc && key < hi) ? table[key >> page_shift] : -1;
     };
     int page = page_of(0);
@@ -375,7 +408,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       if (round > 0 && !warp_wait(&bars[empty0 + st], (round - 1) & 1, gu)) break;
       // pages of the chunk that hold a key below hi (the others are never touched: their
       // scores are masked and their value rows are cleared by the softmax warps)
-      const int key0 = (c0 + it) * KC;
+      const int key0 = walk.chunk(it) * KC;
       const int n_pages = min(ppc, (hi - key0 + page_size - 1) >> page_shift);
       if (lane == 0) mbar_expect_tx(&bars[full0 + st], (uint32_t)n_pages * page_size * 128u * halves);
       __syncwarp();
@@ -454,7 +487,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     const int t_first = p_first + (t * ROWS) / gb, t_last = min(hi - 1, p_first + (t * ROWS + ROWS - 1) / gb);
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t tmem_o = tmem + TM_O + t * 128;
-    const float sc = scale * LOG2E;
+    const float sc = CAPPED ? 1.f : scale * LOG2E;      // capped scores are exponents already
     // optional extras, per head: a distance bias (the scaled score of a key `dist` positions back is
     // lowered by slope * dist: taken off the raw scores, in their units) and a sink (a score without a
     // key that joins the denominator once)
@@ -464,8 +497,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int it = 0; it < n_chunks; ++it) {
-      const int c = c0 + it, sb = it & 1, sround = it >> 1, st = it % NSTAGE, round = it / NSTAGE;
-      const int key0 = c * KC;
+      const int sb = it & 1, sround = it >> 1, st = it % NSTAGE, round = it / NSTAGE;
+      const int key0 = walk.chunk(it) * KC;
       if (!warp_wait(&bars[B_SFULL + 2 * t + sb], sround & 1, gu)) { ok = false; break; }
       tc_fence_after();
       float s[64];
@@ -480,17 +513,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           s[32 + i] = __uint_as_float(rb[i]);
         }
       }
+      if (CAPPED) cap_scores(s, cap_k, cap_h);
       if (slopes) {   // (the same for the whole block)
         const float back = (float)(prow - key0);
 #pragma unroll
         for (int j = 0; j < 64; ++j) s[j] = fmaf(bias_per_step, (float)j - back, s[j]);
       }
-      const bool interior = key0 + KC - 1 <= t_first && key0 >= (window > 0 ? max(0, t_last - window + 1) : 0) &&
-                            key0 >= (chunk > 0 ? (t_last / chunk) * chunk : 0) && key0 >= lo;
+      const bool interior = key0 + KC - 1 <= t_first &&
+                            ((key0 >= (window > 0 ? max(0, t_last - window + 1) : 0) &&
+                              key0 >= (chunk > 0 ? (t_last / chunk) * chunk : 0) && key0 >= lo) || key0 + KC <= keep);
       if (!interior || !rvalid) {
 #pragma unroll
         for (int j = 0; j < 64; ++j)
-          if (!(rvalid && key0 + j <= prow && key0 + j >= lorow)) s[j] = -INFINITY;
+          if (!(rvalid && key0 + j <= prow && (key0 + j >= lorow || key0 + j < keep))) s[j] = -INFINITY;
       }
       // The exponents are taken relative to m_run, which follows the true running maximum
       // lazily: it moves (and O and l are rescaled) only when some row of the warp found a
@@ -574,12 +609,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       // clear them, 0 * NaN is NaN.  Only a request's first and last chunks have such rows.  Each
       // tile does it before it publishes its probabilities (the tiles' second products are
       // issued independently; both write the same zeros).
-      if (key0 < lo || key0 + KC > hi) {
+      if ((key0 < lo && key0 + KC > keep) || key0 + KC > hi) {
         if (!warp_wait(&bars[B_VFULL + st], round & 1, gu)) { ok = false; break; }
         unsigned char* vt = Vs + st * tile_bytes;
         for (int idx = r; idx < KC * halves * 8; idx += ROWS) {
           const int j = idx / (halves * 8), rest = idx - j * (halves * 8);
-          if (key0 + j < lo || key0 + j >= hi)
+          if ((key0 + j < lo && key0 + j >= keep) || key0 + j >= hi)
             *reinterpret_cast<uint4*>(vt + (rest >> 3) * (KC * 128) + j * 128 + ((rest & 7) << 4)) = make_uint4(0u, 0u, 0u, 0u);
         }
         fence_async_smem();   // plain stores that the tensor core reads
@@ -992,14 +1027,16 @@ extern "C" int mi_attention_prefill_tc_tile_tokens(int g) {
 // denominator without a key or a value, and a distance bias (the scaled score of a key `dist`
 // positions back is lowered by slopes[h] * dist).
 // `chunk` > 0: a query at position p sees only the keys of its own chunk of positions, j >= (p / chunk) * chunk.
-extern "C" int mi_attention_prefill_tc_masked(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
+extern "C" int mi_attention_prefill_tc_capped(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
                                               const void* vcache, long long n_pages, const int* block_table,
                                               int bt_stride, const int* table_rows, int page_size, const int* q_start,
                                               const int* q_len, const int* kv_len, const int* tile_req,
                                               const int* tile_tok0, int n_tiles, int tile_tokens, int nq, int nkv, int d,
-                                              float scale, int window, int chunk, const float* sinks,
-                                              const float* slopes, cudaStream_t stream) {
+                                              float scale, int window, int chunk, int keep, float softcap,
+                                              const float* sinks, const float* slopes, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
+  if (keep < 0 || (keep && chunk) || !(softcap >= 0.f)) MI_REFUSE("attention_tc: bad kept keys %d or cap %f", keep, softcap);
+  if (softcap > 0.f && slopes) MI_REFUSE("attention_tc: a distance bias is not taken beside a cap");
   if (chunk < 0) MI_REFUSE("attention_tc: bad chunk size %d", chunk);
   if (!mi_attention_prefill_tc_supported(nq, nkv, d, page_size))
     MI_REFUSE("attention_tc: sizes not taken (heads %d/%d, head size %d, pages of %d)", nq, nkv, d, page_size);
@@ -1021,7 +1058,7 @@ extern "C" int mi_attention_prefill_tc_masked(const void* q, int q_stride, void*
     MI_REFUSE("attention_tc: the driver refused a tensor map");
   const int halves = d / 64;
   const size_t smem = (size_t)NTILE * ROWS * 128 * halves + 2 * NSTAGE * (size_t)KC * 128 * halves + 1024;
-  auto kern = attention_prefill_tc_kernel;
+  auto kern = softcap > 0.f ? attention_prefill_tc_kernel<true> : attention_prefill_tc_kernel<false>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const long long n_blocks = (long long)n_tiles * nkv * hblocks;
@@ -1029,8 +1066,21 @@ extern "C" int mi_attention_prefill_tc_masked(const void* q, int q_stride, void*
   dim3 grid((unsigned)n_blocks);
   MI_LAUNCH((kern), grid, TC_THREADS, smem, stream, map_k, map_v, (const bf16*)q, q_stride, (bf16*)out, out_stride,
             block_table, bt_stride, table_rows, page_size, page_shift, q_start, q_len, kv_len, tile_req, tile_tok0, nq, nkv, d, scale,
-            window, chunk, gb, NTILE * ROWS / gb, sinks, slopes);
+            window, chunk, gb, NTILE * ROWS / gb, sinks, slopes, keep, softcap > 0.f ? scale / softcap : 0.f,
+            softcap * LOG2E);
   MI_RETURN_LAUNCH_STATUS();
+}
+
+extern "C" int mi_attention_prefill_tc_masked(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
+                                              const void* vcache, long long n_pages, const int* block_table,
+                                              int bt_stride, const int* table_rows, int page_size, const int* q_start,
+                                              const int* q_len, const int* kv_len, const int* tile_req,
+                                              const int* tile_tok0, int n_tiles, int tile_tokens, int nq, int nkv, int d,
+                                              float scale, int window, int chunk, const float* sinks,
+                                              const float* slopes, cudaStream_t stream) {
+  return mi_attention_prefill_tc_capped(q, q_stride, out, out_stride, kcache, vcache, n_pages, block_table, bt_stride,
+                                        table_rows, page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles,
+                                        tile_tokens, nq, nkv, d, scale, window, chunk, 0, 0.f, sinks, slopes, stream);
 }
 
 extern "C" int mi_attention_prefill_tc_ext(const void* q, int q_stride, void* out, int out_stride, const void* kcache,

@@ -47,6 +47,7 @@ LIBRARIES: dict[str, tuple[list[str], list[str], list[str]]] = {
     "attention_rows": (["attention_rows.cu"], ["common.cuh"], []),
     "depth": (["depth.cu"], ["common.cuh"], []),
     "latent_decode": (["latent_decode.cu"], ["common.cuh"], []),
+    "attention_stage": (["attention_stage.cu"], ["common.cuh"], []),
 }
 
 

@@ -194,12 +194,53 @@ __device__ __forceinline__ void mi_rotate(float x1, float x2, float s, float c, 
   y2 = __fadd_rn(__fmul_rn(x2, c), __fmul_rn(x1, s));
 }
 
+// The walk over a row of keys cut into chunks of `size`, for queries that see the keys from `lo` on and, with
+// keep > 0, the first `keep` keys of the sequence as well: the chunks that hold kept keys below lo's chunk, then
+// the chunks from lo's on.
+struct MiKeyWalk {
+  int pre, c0;
+  __host__ __device__ __forceinline__ MiKeyWalk(int lo, int keep, int size) {
+    c0 = lo / size;
+    pre = keep > 0 ? (keep + size - 1) / size : 0;
+    if (pre > c0) pre = c0;
+  }
+  __host__ __device__ __forceinline__ int chunk(int i) const { return i < pre ? i : c0 + i - pre; }
+  // chunks of the walk when the keys end at `hi` (exclusive)
+  __host__ __device__ __forceinline__ int count(int hi, int size) const { return pre + (hi + size - 1) / size - c0; }
+};
+
+// tanh(t) for |t| <= MI_TANH_POLY as t P(t^2): the coefficients are a minimax fit (iteratively reweighted least
+// squares on a dense grid) with an error of 2e-8.
+#define MI_TANH_POLY 0.6f
+#define MI_TANH_C0 0.999999627f
+#define MI_TANH_C1 -0.333312086f
+#define MI_TANH_C2 0.132992106f
+#define MI_TANH_C3 -0.0516967532f
+#define MI_TANH_C4 0.0149769696f
+__device__ __forceinline__ float mi_tanh_wide(float t) {      // 1 - 2 / (e^(2t) + 1), an absolute error near 1e-7
+  return 1.f - __fdividef(2.f, __expf(2.f * t) + 1.f);
+}
+// A capped score for scores whose weights are rounded to bfloat16: height * tanh(s * k), with k = scale / cap and
+// height = cap (or cap log2 e, for exponents to base two).
+__device__ __forceinline__ float mi_softcap(float s, float k, float height) {
+  const float t = s * k, z = t * t;
+  const float p = fmaf(fmaf(fmaf(fmaf(MI_TANH_C4, z, MI_TANH_C3), z, MI_TANH_C2), z, MI_TANH_C1), z, MI_TANH_C0);
+  const float a = fminf(fabsf(t), 40.f);
+  return height * (a <= MI_TANH_POLY ? t * p : copysignf(mi_tanh_wide(a), t));
+}
+
 // An activation of one value: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0.
 __device__ __forceinline__ float mi_xielu(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
 
-// The same for a result that is rounded to bfloat16: the exponential is the hardware's, and close to zero,
+// The square of max(z, 0).
+__device__ __forceinline__ float mi_relu2(float z) {
+  const float p = fmaxf(z, 0.f);
+  return p * p;
+}
+
+// mi_xielu for a result that is rounded to bfloat16: the exponential is the hardware's, and close to zero,
 // where e^z - 1 - z would cancel, its power series z^2 / 2 + z^3 / 6 + z^4 / 24 takes its place.
 __device__ __forceinline__ float mi_xielu_bf16(float z, float a, float b) {
   const float series = z * z * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f);

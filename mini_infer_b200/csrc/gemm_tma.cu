@@ -224,9 +224,10 @@ struct EpilogueFusion {
 #define FUSED_MAX_TOKENS 16
 // `swiglu` beyond the gated forms: an activation of every value of the product by itself
 #define ACT_XIELU 3
+#define ACT_RELU2 4      // the square of max(z, 0)
 
 // kAct: an instance of its own for an activation of single values, so that the others keep their code.
-template <typename OutT, bool kFused, bool kAct>
+template <typename OutT, bool kFused, int kAct>
 __global__ void __launch_bounds__(GT_THREADS, 1)
 gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                 OutT* __restrict__ y, int ldy, int M, int N, int K, int n_tok, int stages, int kb, int chunked, int swiglu,
@@ -426,7 +427,7 @@ gemm_tma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
         if (n < N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(mi_xielu_bf16(v[j], fus.act_a, fus.act_b));
+            if (c0 + j < M) y[(size_t)(c0 + j) * ldy + n] = mi_from_float<OutT>(kAct == ACT_RELU2 ? mi_relu2(v[j]) : mi_xielu_bf16(v[j], fus.act_a, fus.act_b));
         }
       } else if (swiglu) {
         // rows alternate gate, up: the even lane of a pair has the gate, its neighbour the up
@@ -629,8 +630,8 @@ extern "C" int mi_gemm_tma_workspace(int M, int N, int blocks, long long* partia
 
 // x [M, K] bf16 (row stride ldx), w [N, K] bf16 contiguous, y [M, N] (row stride ldy) bf16 or
 // fp32.  With `swiglu` (1: SiLU, 2: the tanh form of GELU) the rows of w alternate gate, up and y is [M, N / 2]:
-// y[m, i] = act(x w[2i]) * (x w[2i+1]), computed on the fp32 accumulators; with `swiglu` 3 y is [M, N] and every value
-// passes mi_xielu with act_a and act_b.  `blocks` is the number of persistent blocks (the number of SMs); `partials` and
+// y[m, i] = act(x w[2i]) * (x w[2i+1]), computed on the fp32 accumulators; with `swiglu` 3 or 4 y is [M, N] and
+// every value passes mi_xielu with act_a and act_b, or mi_relu2.  `blocks` is the number of persistent blocks (the number of SMs); `partials` and
 // `counters` (zero before the first call; the kernel leaves them zero) as mi_gemm_tma_workspace
 // says.
 //
@@ -653,10 +654,11 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
       MI_REFUSE("gemm_tma: the residual epilogue needs a gain and room for its statistics, and no gate/up pairs");
     if (residual && !mi_aligned(residual, 4)) MI_REFUSE("gemm_tma: misaligned residual stream");
   }
-  if (swiglu < 0 || swiglu > ACT_XIELU) MI_REFUSE("gemm_tma: unknown activation %d", swiglu);
-  if (swiglu == ACT_XIELU && (stats_in || residual || out_dtype != MI_DTYPE_BF16))
+  const bool single = swiglu == ACT_XIELU || swiglu == ACT_RELU2;     // an activation of single values
+  if (swiglu < 0 || swiglu > ACT_RELU2) MI_REFUSE("gemm_tma: unknown activation %d", swiglu);
+  if (single && (stats_in || residual || out_dtype != MI_DTYPE_BF16))
     MI_REFUSE("gemm_tma: an activation of single values goes with the plain product and a bfloat16 result");
-  if (swiglu && swiglu != ACT_XIELU && (N % 2)) MI_REFUSE("gemm_tma: the gate/up epilogue needs an even number of rows of W, got %d", N);
+  if (swiglu && !single && (N % 2)) MI_REFUSE("gemm_tma: the gate/up epilogue needs an even number of rows of W, got %d", N);
   if (M <= 0 || N <= 0) return 0;
   if (M > MAX_TOKENS) MI_REFUSE("gemm_tma: %d rows of x; this kernel takes at most %d", M, MAX_TOKENS);
   if (K <= 0 || K % 8 != 0 || ldx % 8 != 0)
@@ -711,11 +713,13 @@ extern "C" int mi_gemm_tma_fused(const void* x, long long ldx, const void* w, vo
   const bool fused = stats_in || residual;
   const int w_evict_first = mi_l2_hints_enabled() ? 1 : 0;
   if (swiglu == ACT_XIELU && out_dtype == MI_DTYPE_BF16) {
-    GT_LAUNCH(bf16, false, true)
+    GT_LAUNCH(bf16, false, ACT_XIELU)
+  } else if (swiglu == ACT_RELU2 && out_dtype == MI_DTYPE_BF16) {
+    GT_LAUNCH(bf16, false, ACT_RELU2)
   } else if (out_dtype == MI_DTYPE_BF16) {
-    if (fused) GT_LAUNCH(bf16, true, false) else GT_LAUNCH(bf16, false, false)
+    if (fused) GT_LAUNCH(bf16, true, 0) else GT_LAUNCH(bf16, false, 0)
   } else {
-    if (fused) GT_LAUNCH(float, true, false) else GT_LAUNCH(float, false, false)
+    if (fused) GT_LAUNCH(float, true, 0) else GT_LAUNCH(float, false, 0)
   }
 #undef GT_LAUNCH
   MI_RETURN_LAUNCH_STATUS();

@@ -156,6 +156,10 @@ def _sig_attention_generic(lib: ctypes.CDLL) -> None:
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
         c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p]
+    lib.mi_attention_generic_capped.argtypes = [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+        c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p]
 
 
 def _sig_sampling(lib: ctypes.CDLL) -> None:
@@ -179,7 +183,7 @@ def _sig_attention_mma(lib: ctypes.CDLL) -> None:
     lib.mi_attention_decode_balanced.argtypes = [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
         c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-        c_void_p]
+        c_int, c_float, c_void_p]
     lib.mi_attention_decode_balanced_unit_cost.argtypes = [c_int]
     lib.mi_attention_wait_status.argtypes = [c_int]
     lib.mi_set_status_word.argtypes = [c_void_p]
@@ -187,6 +191,10 @@ def _sig_attention_mma(lib: ctypes.CDLL) -> None:
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
         c_float, c_int, c_void_p]
+    lib.mi_attention_prefill_capped.argtypes = [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+        c_float, c_int, c_int, c_float, c_void_p]
     lib.mi_attention_prefill_tile_tokens.argtypes = [c_int]
     lib.mi_attention_prefill_tile_tokens.restype = c_int
 
@@ -216,6 +224,10 @@ def _sig_attention_tc(lib: ctypes.CDLL) -> None:
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
         c_void_p, c_void_p, c_void_p]
+    lib.mi_attention_prefill_tc_capped.argtypes = [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+        c_int, c_float, c_void_p, c_void_p, c_void_p]
     lib.mi_attention_prefill_tc_supported.argtypes = [c_int, c_int, c_int, c_int]
     lib.mi_attention_tc_status.argtypes = [c_int]
     lib.mi_set_status_word.argtypes = [c_void_p]
@@ -304,6 +316,9 @@ def _sig_stream(lib: ctypes.CDLL) -> None:
                                   c_int, c_int, c_void_p]
     lib.mi_scale_f32.argtypes = [c_void_p, ll, c_float, c_void_p]
     lib.mi_xielu_map.argtypes = [c_void_p, c_void_p, ll, c_float, c_float, c_int, c_void_p]
+    lib.mi_relu2_map.argtypes = [c_void_p, c_void_p, ll, c_int, c_void_p]
+    lib.mi_branch_norm_then_norm.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_float, c_float, c_void_p, c_float,
+                                             c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
 
 
 def _sig_depth(lib: ctypes.CDLL) -> None:
@@ -345,12 +360,25 @@ def _sig_attention_rows(lib: ctypes.CDLL) -> None:
     lib.mi_attention_rows.argtypes = [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
+        c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]
     lib.mi_attention_rows_tile_tokens.argtypes = [c_int, c_int]
     lib.mi_attention_rows_supported.argtypes = [c_int, c_int, c_int, c_int, c_int]
 
 
+def _sig_attention_stage(lib: ctypes.CDLL) -> None:
+    lib.mi_rope_angles.argtypes = [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p]
+    lib.mi_conv_rope_store.argtypes = [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+        c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
+    lib.mi_split_maps_store.argtypes = [
+        c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p,
+        c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
+    lib.mi_combine_maps.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                    c_float, c_int, c_void_p]
+
+
 _SIGNATURES = {
+    "attention_stage": _sig_attention_stage,
     "attention_rows": _sig_attention_rows,
     "depth": _sig_depth,
     "latent_decode": _sig_latent_decode,
@@ -657,7 +685,7 @@ def decode_rope_fusable(q_dtype: torch.dtype, head_dim: int, decode_only: bool, 
 
 def attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, ctx, nq: int, nkv: int,
               head_dim: int, scale: float, window: int = 0, rope_table: torch.Tensor | None = None,
-              chunk: int = 0) -> None:
+              chunk: int = 0, keep_first: int = 0, softcap: float = 0.0) -> None:
     """Attention of this step's queries over one cache layer.
 
     ``cache`` is a ``LayerCache`` (its ``k``/``v`` pages and group index), ``ctx`` the
@@ -668,8 +696,12 @@ def attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, ctx, nq:
     un-rotated and not yet stored; the decode kernel does both.  ``window`` > 0: a query sees the last
     ``window`` positions only; ``chunk`` > 0: only the keys of its own chunk of positions,
     ``j >= (p // chunk) * chunk`` (one of the two; the mma.sync kernels take a chunk as a negative window).
+    ``keep_first`` > 0: beside its window a query sees the first ``keep_first`` positions of its sequence;
+    ``softcap`` > 0: a scaled score ``s`` becomes ``softcap tanh(s / softcap)`` (bfloat16 only, as ``chunk``).
     """
     group = ctx.groups[cache.group]
+    if keep_first and chunk:
+        raise KernelError("attention: first positions are kept beside a window, not beside chunks")
     if window and chunk:
         raise KernelError("attention: a window or chunks, not both")
     if chunk < 0 or window < 0:
@@ -680,7 +712,7 @@ def attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, ctx, nq:
             attention_decode_balanced(q, q_stride, out, cache.k, cache.v, group.block_table, group.page_size,
                                       ctx.q_start, ctx.kv_len, ctx.n_requests, nq, nkv, head_dim, scale, mask,
                                       table_rows=group.table_rows, rope_table=rope_table,
-                                      store_kv=bool(cache.writes))
+                                      store_kv=bool(cache.writes), keep_first=keep_first, softcap=softcap)
         else:
             if rope_table is not None:
                 raise KernelError("attention: only the decode kernel rotates and stores by itself")
@@ -692,19 +724,22 @@ def attention(q: torch.Tensor, q_stride: int, out: torch.Tensor, cache, ctx, nq:
                 # all blocks), the prompt portions through the prefill kernel; disjoint rows of `out`
                 attention_decode_balanced(q, q_stride, out, cache.k, cache.v, group.block_table, group.page_size,
                                           ctx.single_q_start, ctx.single_kv_len, ctx.n_single, nq, nkv, head_dim,
-                                          scale, mask, table_rows=ctx.single_rows)
+                                          scale, mask, table_rows=ctx.single_rows, keep_first=keep_first,
+                                          softcap=softcap)
                 tile_req, tile_tok0, n_tiles = ctx.tiles_multi[tt]
             if tc:
                 attention_prefill_tc(q, q_stride, out, cache.k, cache.v, group.block_table, group.page_size,
                                      ctx.q_start, ctx.q_len, ctx.kv_len, tile_req, tile_tok0, n_tiles, tt,
-                                     nq, nkv, head_dim, scale, window, table_rows=group.table_rows, chunk=chunk)
+                                     nq, nkv, head_dim, scale, window, table_rows=group.table_rows, chunk=chunk,
+                                     keep_first=keep_first, softcap=softcap)
             else:
                 attention_prefill(q, q_stride, out, cache.k, cache.v, group.block_table, group.page_size,
                                   ctx.q_start, ctx.q_len, ctx.kv_len, tile_req, tile_tok0, n_tiles, tt,
-                                  nq, nkv, head_dim, scale, mask, table_rows=group.table_rows)
+                                  nq, nkv, head_dim, scale, mask, table_rows=group.table_rows,
+                                  keep_first=keep_first, softcap=softcap)
         return
-    if chunk:
-        raise KernelError("attention: float32 chunks go through attention_ext")
+    if chunk or keep_first or softcap:
+        raise KernelError("attention: float32 chunks, kept first positions and capped scores go through attention_ext")
     tile_req, tile_tok0, n_tiles = ctx.q_tiles(ATTENTION_TILE_TOKENS)
     attention_generic(q, q_stride, out, cache.k, cache.v, group.block_table, group.page_size,
                       ctx.q_start, ctx.q_len, ctx.kv_len, tile_req, tile_tok0, n_tiles,
@@ -789,14 +824,15 @@ def _balanced_workspace(device: torch.device, o_floats: int, ml_floats: int, cou
 def attention_decode_balanced(q, q_stride, out, kcache, vcache, block_table, page_size, q_start, kv_len,
                               n_requests, nq, nkv, head_dim, scale, window=0, table_rows=None,
                               rope_table: torch.Tensor | None = None, store_kv: bool = True,
-                              sinks: torch.Tensor | None = None) -> None:
+                              sinks: torch.Tensor | None = None, keep_first: int = 0, softcap: float = 0.0) -> None:
     """bfloat16 decode attention with the keys of all requests spread evenly over persistent
     blocks, whatever the requests' lengths (attention_decode_balanced_kernel): no plan from the
     host, the blocks read the lengths themselves.  With ``rope_table`` (``rope_table()`` of the
     step's positions) q, k and v come as the projection left them (one row per token: q heads, k
     heads, v heads): the kernel rotates q itself and, with ``store_kv``, rotates the new key and
     writes it and the new value into their page before it reads them.  ``sinks`` (fp32 ``[nq]``): a score per
-    head that joins the softmax's denominator without a key or a value."""
+    head that joins the softmax's denominator without a key or a value.  ``keep_first``, ``softcap``: see
+    ``attention``."""
     _cuda(q, out, kcache, vcache, block_table, q_start, kv_len, table_rows, rope_table, sinks)
     _opt_f32(sinks, nq, "attention_decode (sinks)")
     if rope_table is not None and (rope_table.dtype != torch.float32 or not rope_table.is_contiguous()
@@ -818,7 +854,7 @@ def attention_decode_balanced(q, q_stride, out, kcache, vcache, block_table, pag
         _ptr(q), int(q_stride), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(block_table),
         block_table.stride(0), _ptr(table_rows), int(page_size), _ptr(q_start), _ptr(kv_len), int(n_requests), nq, nkv,
         head_dim, float(scale), int(window), int(grid.value), _ptr(part_o), _ptr(part_ml), _ptr(count),
-        _ptr(rope_table), 1 if store_kv else 0, _ptr(sinks), _stream())
+        _ptr(rope_table), 1 if store_kv else 0, _ptr(sinks), int(keep_first), float(softcap), _stream())
     _finish(lib, rc, "attention_decode")
 
 
@@ -838,7 +874,7 @@ def attention_wait_status(reset: bool = True) -> int:
 
 def attention_prefill(q, q_stride, out, kcache, vcache, block_table, page_size, q_start, q_len, kv_len,
                       tile_req, tile_tok0, n_tiles, tile_tokens, nq, nkv, head_dim, scale, window=0,
-                      table_rows=None) -> None:
+                      table_rows=None, keep_first: int = 0, softcap: float = 0.0) -> None:
     """bfloat16 attention of query portions of any length over the paged cache (attention_mma.cu)."""
     _cuda(q, out, kcache, vcache, block_table, q_start, q_len, kv_len, tile_req, tile_tok0, table_rows)
     if q.dtype != torch.bfloat16:
@@ -848,11 +884,11 @@ def attention_prefill(q, q_stride, out, kcache, vcache, block_table, page_size, 
                            ("kv_len", kv_len), ("tile_req", tile_req), ("tile_tok0", tile_tok0),
                            ("table_rows", table_rows)))
     lib = _waiting_lib("attention_mma", q.device)
-    rc = lib.mi_attention_prefill(
+    rc = lib.mi_attention_prefill_capped(
         _ptr(q), int(q_stride), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(block_table),
         block_table.stride(0), _ptr(table_rows), int(page_size), _ptr(q_start), _ptr(q_len), _ptr(kv_len), _ptr(tile_req),
         _ptr(tile_tok0), int(n_tiles), int(tile_tokens), nq, nkv, head_dim, float(scale), int(window),
-        _stream())
+        int(keep_first), float(softcap), _stream())
     _finish(lib, rc, "attention_prefill")
 
 
@@ -874,12 +910,13 @@ def prefill_tc_supported(nq: int, nkv: int, head_dim: int, page_size: int) -> bo
 def attention_prefill_tc(q, q_stride, out, kcache, vcache, block_table, page_size, q_start, q_len, kv_len,
                          tile_req, tile_tok0, n_tiles, tile_tokens, nq, nkv, head_dim, scale, window=0,
                          table_rows=None, sinks: torch.Tensor | None = None,
-                         slopes: torch.Tensor | None = None, chunk: int = 0) -> None:
+                         slopes: torch.Tensor | None = None, chunk: int = 0, keep_first: int = 0,
+                         softcap: float = 0.0) -> None:
     """bfloat16 attention of query portions over the paged cache on tcgen05 (attention_tc.cu);
     same arguments as ``attention_prefill``, and optionally ``sinks`` / ``slopes`` (fp32 ``[nq]``: a
     score per head in the softmax's denominator without a key; a distance bias ``slope * (i - j)``
     taken off the scaled scores) and ``chunk`` (> 0: a query at position ``p`` sees only the keys of its
-    own chunk of positions, ``j >= (p // chunk) * chunk``)."""
+    own chunk of positions, ``j >= (p // chunk) * chunk``); ``keep_first``, ``softcap``: see ``attention``."""
     _cuda(q, out, kcache, vcache, block_table, q_start, q_len, kv_len, tile_req, tile_tok0, table_rows, sinks, slopes)
     for name, t in (("sinks", sinks), ("slopes", slopes)):
         if t is not None and (t.dtype != torch.float32 or t.numel() != nq or not t.is_contiguous()):
@@ -891,11 +928,11 @@ def attention_prefill_tc(q, q_stride, out, kcache, vcache, block_table, page_siz
                            ("kv_len", kv_len), ("tile_req", tile_req), ("tile_tok0", tile_tok0),
                            ("table_rows", table_rows)))
     lib = _waiting_lib("attention_tc", q.device)
-    rc = lib.mi_attention_prefill_tc_masked(
+    rc = lib.mi_attention_prefill_tc_capped(
         _ptr(q), int(q_stride), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), int(kcache.shape[0]),
         _ptr(block_table), block_table.stride(0), _ptr(table_rows), int(page_size), _ptr(q_start), _ptr(q_len), _ptr(kv_len),
         _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), int(tile_tokens), nq, nkv, head_dim, float(scale),
-        int(window), int(chunk), _ptr(sinks), _ptr(slopes), _stream())
+        int(window), int(chunk), int(keep_first), float(softcap), _ptr(sinks), _ptr(slopes), _stream())
     _finish(lib, rc, "attention_prefill_tc")
 
 
@@ -1146,12 +1183,12 @@ def linear_swiglu(x: torch.Tensor, w_pairs: torch.Tensor, row_stats: "RowStats |
     return glu_mul_pairs(linear(x, w_pairs), act)
 
 
-UNARY_ACT = {"xielu": 3}      # the streaming product's epilogue numbers
+UNARY_ACT = {"xielu": 3, "relu2": 4}      # the streaming product's epilogue numbers
 
 
 def linear_activated(x: torch.Tensor, w: torch.Tensor, act: str, numbers: tuple[float, float]) -> torch.Tensor:
     """``act(x w^T)`` value by value in fp32; ``"xielu"`` with ``numbers = (a, b)``: ``a z^2 + z / 2`` for ``z > 0``,
-    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``.  Decode-sized bfloat16 inputs run the activation in the streaming
+    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``; ``"relu2"``: the square of ``max(z, 0)``.  Decode-sized bfloat16 inputs run the activation in the streaming
     product's epilogue, everything else runs ``linear`` and the activation in place."""
     if act not in UNARY_ACT:
         raise KernelError(f"linear_activated: unknown activation {act!r}")
@@ -1160,8 +1197,11 @@ def linear_activated(x: torch.Tensor, w: torch.Tensor, act: str, numbers: tuple[
         return gemm_tma(x, w, torch.bfloat16, act=(act, numbers))
     y = linear(x, w)
     lib = _lib("stream")
-    rc = lib.mi_xielu_map(_ptr(y), _ptr(y), y.numel(), float(numbers[0]), float(numbers[1]), _code(y.dtype), _stream())
-    _finish(lib, rc, "xielu")
+    if act == "relu2":
+        rc = lib.mi_relu2_map(_ptr(y), _ptr(y), y.numel(), _code(y.dtype), _stream())
+    else:
+        rc = lib.mi_xielu_map(_ptr(y), _ptr(y), y.numel(), float(numbers[0]), float(numbers[1]), _code(y.dtype), _stream())
+    _finish(lib, rc, act)
     return y
 
 
@@ -2281,7 +2321,7 @@ def _rows_attention_smem(rows: int, d: int, dv: int, values_in_keys: bool, stage
 
 
 def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys: bool, device,
-                         window: int = 0) -> tuple[int, int, int, int]:
+                         window: int = 0, keep_first: int = 0) -> tuple[int, int, int, int]:
     """``(rows per block, tokens per tile, runs of keys per tile, buffers per chunk)`` for this step:
     steps of single tokens take 16 rows and cut every request's keys into runs, so that the blocks
     fill the GPU; prompt portions take 64 rows with two buffers for the chunk's rows (the next chunk
@@ -2298,26 +2338,27 @@ def _rows_attention_plan(ctx, nq: int, nkv: int, d: int, dv: int, values_in_keys
         return 16, rows_attention_tile_tokens(group, 16), 1, 1
     tt = rows_attention_tile_tokens(group, 16)
     units = ctx.tiles[tt][2] * nkv * max(1, -(-group // 16))
-    return 16, tt, _rows_attention_runs(ctx, units, window, device), 1
+    return 16, tt, _rows_attention_runs(ctx, units, window, device, keep_first), 1
 
 
-def _rows_attention_runs(ctx, units: int, window: int, device) -> int:
+def _rows_attention_runs(ctx, units: int, window: int, device, keep_first: int = 0) -> int:
     """Runs of keys per tile in a step of ``units`` tiles of single tokens, so that the blocks fill the GPU."""
     chunks = max(1, -(-int(getattr(ctx, "max_kv_len", 0) or 64) // 64))
     if window:                       # the keys of one window touch at most this many chunks
-        chunks = min(chunks, -(-(window - 1) // 64) + 1)
+        chunks = min(chunks, -(-(window - 1) // 64) + 1 + -(-keep_first // 64))
     return max(1, min(-(-4 * _sms(device) // units), chunks, 64))
 
 
 def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: int, d: int, dv: int, scale: float, *,
                   window: int = 0, sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
-                  values_in_keys: bool = False, chunk: int = 0) -> None:
+                  values_in_keys: bool = False, chunk: int = 0, keep_first: int = 0, softcap: float = 0.0) -> None:
     """``attention_kv`` with the extras of the CUDA-core kernel: ``sinks`` (fp32 ``[nq]``: a score per
     head that joins the softmax's denominator without a key or a value), ``slopes`` (fp32 ``[nq]``:
     the scaled score of a key ``dist`` positions back is lowered by ``slope * dist``) and
     ``values_in_keys`` (the cache layer has keys only; a key's value is the first ``dv`` numbers of its
     own row); ``chunk`` > 0: a query at position ``p`` sees only the keys of its own chunk of positions,
-    ``j >= (p // chunk) * chunk``.  fp32 scores, weights and sums for float32 and bfloat16 alike.  bfloat16 prompt portions
+    ``j >= (p // chunk) * chunk``; ``keep_first`` > 0: beside its window a query sees the first ``keep_first`` positions
+    of its sequence; ``softcap`` > 0: a scaled score ``s`` becomes ``softcap tanh(s / softcap)``.  fp32 scores, weights and sums for float32 and bfloat16 alike.  bfloat16 prompt portions
     with keys and values of one size that attention_tc.cu takes run on tcgen05; other bfloat16 steps with sizes that
     attention_rows.cu takes (``rows_attention_supported``) and tiles planned for it runs on tensor
     cores (weights rounded to bfloat16 for the second product); everything else on CUDA cores."""
@@ -2339,7 +2380,7 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
     bt = group.block_table
     # prompt portions of heads that the tcgen05 prefill kernel takes (keys and values of 64 or 128) go there
     if (q.dtype == torch.bfloat16 and not values_in_keys and d == dv and not getattr(ctx, "decode_only", False)
-            and not chunk and USE_TC_PREFILL and scale > 0 and prefill_tc_supported(nq, nkv, d, group.page_size)
+            and not chunk and not (softcap and slopes is not None) and USE_TC_PREFILL and scale > 0 and prefill_tc_supported(nq, nkv, d, group.page_size)
             and prefill_tc_tile_tokens(nq // nkv) in ctx.tiles and out.is_contiguous()
             and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
             and kc.data_ptr() % 128 == 0 and vc.data_ptr() % 128 == 0):
@@ -2347,13 +2388,15 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
         tile_req, tile_tok0, n_tiles = ctx.q_tiles(tt)
         attention_prefill_tc(q, q.stride(0), out, kc, vc, bt, group.page_size, ctx.q_start, ctx.q_len, ctx.kv_len,
                              tile_req, tile_tok0, n_tiles, tt, nq, nkv, d, scale, int(window),
-                             table_rows=group.table_rows, sinks=sinks, slopes=slopes)
+                             table_rows=group.table_rows, sinks=sinks, slopes=slopes, keep_first=keep_first,
+                             softcap=softcap)
         return
     if (q.dtype == torch.bfloat16 and not chunk
             and rows_attention_supported(nq, nkv, d, dv, values_in_keys)
             and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0 and out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0
             and rows_attention_tile_tokens(nq // nkv, 16) in ctx.tiles):
-        rows, tt, splits, stages = _rows_attention_plan(ctx, nq, nkv, d, dv, values_in_keys, q.device, int(window))
+        rows, tt, splits, stages = _rows_attention_plan(ctx, nq, nkv, d, dv, values_in_keys, q.device, int(window),
+                                                        int(keep_first))
         tile_req, tile_tok0, n_tiles = ctx.q_tiles(tt)
         part_o = part_ml = None
         if splits > 1:
@@ -2365,7 +2408,8 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), _ptr(vc), _ptr(bt), bt.stride(0),
             _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len),
             _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), tt, rows, nq, nkv, d, dv, float(scale), _ptr(sinks),
-            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, int(window), 1, _stream())
+            _ptr(slopes), 1 if values_in_keys else 0, splits, _ptr(part_o), _ptr(part_ml), stages, int(window), 1,
+            int(keep_first), float(softcap), _stream())
         _finish(lib, rc, "attention")
         if splits > 1:
             launch_count += 1        # the merge of the runs
@@ -2374,11 +2418,11 @@ def attention_ext(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq: int, nkv: 
     lib = _lib("attention_generic")
     if lib.mi_attention_generic_tile_tokens() != ATTENTION_TILE_TOKENS:
         raise KernelError("attention: the kernel's tile size differs from ATTENTION_TILE_TOKENS")
-    rc = lib.mi_attention_generic_masked(
+    rc = lib.mi_attention_generic_capped(
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), _ptr(vc), _ptr(bt), bt.stride(0),
         _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), _ptr(ctx.q_len), _ptr(ctx.kv_len),
         _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), nq, nkv, d, dv, float(scale), int(window), int(chunk),
-        _ptr(sinks), _ptr(slopes), 1 if values_in_keys else 0, _code(q.dtype), _stream())
+        int(keep_first), float(softcap), _ptr(sinks), _ptr(slopes), 1 if values_in_keys else 0, _code(q.dtype), _stream())
     _finish(lib, rc, "attention")
 
 
@@ -2405,7 +2449,7 @@ def attention_latent_singles(q: torch.Tensor, out: torch.Tensor, cache, ctx, nq:
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kc), None, _ptr(bt), bt.stride(0), _ptr(ctx.single_rows),
         int(group.page_size), _ptr(ctx.single_q_start), None, _ptr(ctx.single_kv_len), None, None, int(ctx.n_single),
         rows_attention_tile_tokens(nq, 16), 16, nq, 1, d, dv, float(scale), _ptr(sinks), None, 1, splits, _ptr(part_o),
-        _ptr(part_ml), 1, int(window), 1, _stream())
+        _ptr(part_ml), 1, int(window), 1, 0, 0.0, _stream())
     _finish(lib, rc, "attention")
     if splits > 1:
         launch_count += 1
@@ -2471,7 +2515,7 @@ def attention_latent_runs(q: torch.Tensor, cache, ctx, n: int, d: int, rank: int
         _ptr(q), q.stride(0), _ptr(latent if latent is not None else q), n * rank, _ptr(kc), None, _ptr(bt), bt.stride(0),
         _ptr(group.table_rows), int(group.page_size), _ptr(ctx.q_start), None, _ptr(ctx.kv_len), None, None, M,
         rows_attention_tile_tokens(n, 16), 16, n, 1, d, rank, float(scale), _ptr(sinks), None, 1, splits, _ptr(part_o),
-        _ptr(part_ml), 1, int(window), 0, _stream())
+        _ptr(part_ml), 1, int(window), 0, 0, 0.0, _stream())
     _finish(lib, rc, "attention")
     return part_o, part_ml, splits, latent
 
@@ -2603,4 +2647,143 @@ def batched_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch
         raise KernelError("batched_linear: operands must share float32 or bfloat16")
     launch_count += 1
     torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
+    return out
+
+
+# --------------------------------------------------------------------------------------- around a paged attention
+
+
+CONV_STORE_MAX_TAPS = 16
+
+
+def rope_angles(positions: torch.Tensor, freq: torch.Tensor, mult: float = 1.0) -> torch.Tensor:
+    """fp32 ``[M, 2 n]``: per token the sines, then the cosines of ``position * freq`` (float64 ``[n]``; the angle in
+    double precision), both times ``mult``."""
+    _cuda(positions, freq)
+    if positions.dtype != torch.int32 or positions.dim() != 1 or not positions.is_contiguous():
+        raise KernelError("rope_angles: positions must be a contiguous int32 vector")
+    if freq.dtype != torch.float64 or freq.dim() != 1 or not freq.is_contiguous():
+        raise KernelError("rope_angles: frequencies must be a contiguous float64 vector")
+    M, n = positions.shape[0], freq.shape[0]
+    out = torch.empty((M, 2 * n), dtype=torch.float32, device=positions.device)
+    lib = _lib("attention_stage")
+    rc = lib.mi_rope_angles(_ptr(positions), _ptr(freq), float(mult), _ptr(out), M, n, _stream())
+    _finish(lib, rc, "rope_angles")
+    return out
+
+
+def _stage_caches(slots, kcache, vcache, M: int, nkv: int, d: int, dv: int, dtype, what: str) -> int:
+    if slots is None or slots.dtype != torch.int32 or slots.shape != (M,):
+        raise KernelError(f"{what}: slots must be int32 [M]")
+    for c, size in ((kcache, d), (vcache, dv)):
+        if c is None or c.dtype != dtype or c.dim() != 4 or c.shape[1] != nkv or c.shape[3] != size or not c.is_contiguous():
+            raise KernelError(f"{what}: caches must be contiguous [pages, nkv, page_size, size] in the packed dtype")
+    return int(kcache.shape[2])
+
+
+def conv_rope_store(packed: torch.Tensor, q_out: torch.Tensor, weight: torch.Tensor, state: torch.Tensor | None, ctx,
+                    nq: int, nkv: int, d: int, dv: int, *, rot: int, angles: torch.Tensor | None, slots: torch.Tensor,
+                    kcache: torch.Tensor, vcache: torch.Tensor) -> None:
+    """The packed projection ``[M, >= (nq + nkv) d + nkv dv]`` (q, k, v side by side) through a causal convolution per
+    channel (``weight`` fp32 ``[channels, taps]``, the last tap meets the current token), then the rotation of q and
+    k in the half layout on their first ``rot`` dimensions (``angles`` of ``rope_angles``).  Queries go to ``q_out [M, nq
+    d]``, keys and values to their pages.  ``state`` (fp32 ``[slots, (taps - 1) * channels]``): each request's last
+    projected rows, oldest first, read for a portion's first tokens and moved on.  Needs query tiles of
+    ``ATTENTION_TILE_TOKENS``."""
+    _cuda(packed, q_out, weight, state, angles, slots, kcache, vcache)
+    _cols(packed, "conv_rope_store")
+    M, C = packed.shape[0], (nq + nkv) * d + nkv * dv
+    if packed.shape[1] < C or M != ctx.n_tokens:
+        raise KernelError(f"conv_rope_store: the projection must be [tokens, {C} or more]")
+    if q_out.dtype != packed.dtype or q_out.shape != (M, nq * d) or not q_out.is_contiguous():
+        raise KernelError("conv_rope_store: queries go to a contiguous [M, nq * d] in the packed dtype")
+    if weight.dtype != torch.float32 or weight.dim() != 2 or weight.shape[0] != C or not weight.is_contiguous():
+        raise KernelError(f"conv_rope_store: the taps must be contiguous fp32 [{C}, taps]")
+    taps = weight.shape[1]
+    if rot and (angles is None or angles.dtype != torch.float32 or angles.shape != (M, rot) or not angles.is_contiguous()):
+        raise KernelError("conv_rope_store: angles must be contiguous fp32 [M, rot]")
+    stride = 0
+    if taps > 1:
+        if state is None:
+            raise KernelError("conv_rope_store: more than one tap needs a state")
+        stride = _state_rows(state, "conv_rope_store")
+    page_size = _stage_caches(slots, kcache, vcache, M, nkv, d, dv, packed.dtype, "conv_rope_store")
+    lib = _lib("attention_stage")
+    if lib.mi_conv_rope_store_tile_tokens() != ATTENTION_TILE_TOKENS:
+        raise KernelError("conv_rope_store: the kernel's tile size differs from ATTENTION_TILE_TOKENS")
+    tile_req, tile_tok0, n_tiles = ctx.q_tiles(ATTENTION_TILE_TOKENS)
+    rc = lib.mi_conv_rope_store(
+        _ptr(packed), packed.stride(0), _ptr(weight), taps, _ptr(state), stride, _ptr(ctx.state_slot), _ptr(ctx.q_start),
+        _ptr(ctx.q_len), _ptr(tile_req), _ptr(tile_tok0), int(n_tiles), nq, nkv, d, dv, int(rot), _ptr(angles),
+        _ptr(slots), _ptr(q_out), _ptr(kcache), _ptr(vcache), page_size, _code(packed.dtype), _stream())
+    _finish(lib, rc, "conv_rope_store")
+
+
+def split_maps_store(packed: torch.Tensor, q_out: torch.Tensor, k_off: int, v_off: int, nq: int, nkv: int, d: int,
+                     row: int, dv: int, *, positions: torch.Tensor, temp_coef: float = 0.0, temp_every: int = 1,
+                     slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor) -> None:
+    """Queries (``nq * 2 * d`` columns from 0) and keys (``nkv * 2 * d`` from ``k_off``) that come as two maps per head
+    side by side, values (``nkv * dv`` from ``v_off``).  A key's cache row is ``[map 1, map 2, zeros]`` of ``row``
+    numbers; ``q_out [M, 2 nq * row]`` gets a row per head and map with that map in its place and zeros elsewhere,
+    times ``1 + temp_coef ln(floor((p + 1) / temp_every) + 1)`` at position ``p``."""
+    _cuda(packed, q_out, positions, slots, kcache, vcache)
+    _cols(packed, "split_maps_store")
+    M = packed.shape[0]
+    if max(2 * nq * d, k_off + 2 * nkv * d, v_off + nkv * dv) > packed.shape[1]:
+        raise KernelError("split_maps_store: a column range lies outside the packed projection")
+    if q_out.dtype != packed.dtype or q_out.shape != (M, 2 * nq * row) or not q_out.is_contiguous():
+        raise KernelError("split_maps_store: queries go to a contiguous [M, 2 nq * row] in the packed dtype")
+    if positions.dtype != torch.int32 or positions.shape != (M,):
+        raise KernelError("split_maps_store: positions must be int32 [M]")
+    page_size = _stage_caches(slots, kcache, vcache, M, nkv, row, dv, packed.dtype, "split_maps_store")
+    lib = _lib("attention_stage")
+    rc = lib.mi_split_maps_store(_ptr(packed), packed.stride(0), int(k_off), int(v_off), M, nq, nkv, d, row, dv,
+                                 _ptr(positions), float(temp_coef), int(temp_every), _ptr(slots), _ptr(q_out),
+                                 _ptr(kcache), _ptr(vcache), page_size, _code(packed.dtype), _stream())
+    _finish(lib, rc, "split_maps_store")
+
+
+def combine_maps(heads: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor, nq: int, dv: int, lam: float,
+                 eps: float, mult: float) -> None:
+    """Per head, from its two maps' outputs ``a1, a2`` (``heads [M, nq * 2 * dv]``): ``o = a1 - lam a2``, and ``out [M, nq
+    * dv]`` gets ``o * mult / sqrt(mean(o^2) + eps)``, times ``sigmoid(gate[t, h])`` with a gate ``[M, nq]``."""
+    _cuda(heads, gate, out)
+    _cols(out, "combine_maps")
+    M = heads.shape[0]
+    if heads.shape != (M, 2 * nq * dv) or not heads.is_contiguous() or out.shape != (M, nq * dv) or out.dtype != heads.dtype:
+        raise KernelError("combine_maps: heads must be contiguous [M, 2 nq * dv] and out [M, nq * dv] in one dtype")
+    if gate is not None:
+        _cols(gate, "combine_maps")
+        if gate.shape != (M, nq) or gate.dtype != heads.dtype:
+            raise KernelError("combine_maps: the gate must be [M, nq] in the heads' dtype")
+    lib = _lib("attention_stage")
+    rc = lib.mi_combine_maps(_ptr(heads), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0),
+                             M, nq, dv, float(lam), float(eps), float(mult), _code(heads.dtype), _stream())
+    _finish(lib, rc, "combine_maps")
+
+
+def branch_norm_then_norm(stream: torch.Tensor, branch: torch.Tensor, gain_y: torch.Tensor, eps_y: float, mult: float,
+                          gain_r: torch.Tensor, eps_r: float, dtype: torch.dtype, *,
+                          rows: torch.Tensor | None = None) -> torch.Tensor:
+    """``r = stream + mult * y * rsqrt(mean(y^2) + eps_y) * gain_y`` (``y`` a branch's rows in ``dtype``), then ``r *
+    rsqrt(mean(r^2) + eps_r) * gain_r`` in ``dtype``, one pass, everything between in fp32.  The fp32 ``stream`` takes
+    ``r`` in place; with ``rows`` (int32) only those rows run and the stream stays as it is."""
+    _cuda(stream, branch, gain_y, gain_r, rows)
+    if stream is None or stream.dtype != torch.float32 or stream.dim() != 2 or not stream.is_contiguous():
+        raise KernelError("norms: the stream must be contiguous fp32 [M, H]")
+    M, H = stream.shape
+    _cols(branch, "norms")
+    if branch.shape != (M, H) or branch.dtype != dtype:
+        raise KernelError("norms: the branch must be [M, H] in the compute dtype")
+    _f32vec(gain_y, H, "norms")
+    _f32vec(gain_r, H, "norms")
+    if rows is not None and (rows.dtype != torch.int32 or rows.dim() != 1 or not rows.is_contiguous()):
+        raise KernelError("norms: rows must be a contiguous int32 vector")
+    n = M if rows is None else rows.shape[0]
+    out = torch.empty((n, H), dtype=dtype, device=stream.device)
+    lib = _lib("stream")
+    rc = lib.mi_branch_norm_then_norm(_ptr(stream), _ptr(branch), branch.stride(0) if M > 1 else H, _ptr(gain_y),
+                                      float(eps_y), float(mult), _ptr(gain_r), float(eps_r), _ptr(rows), _ptr(out), n, H,
+                                      _code(dtype), _stream())
+    _finish(lib, rc, "norms")
     return out

@@ -20,6 +20,8 @@
 //                            what the next branch's products read.  Without a branch: the copy alone.
 //   mi_token_gate            out[t, c] = T(gelu_tanh(z[t, c]) * float(table[id_t, col0 + c])): a gate times the
 //                            columns [col0, col0 + n) of a token's row of a table.
+//   mi_branch_norm_then_norm the norm behind a branch, the sum and the norm in front of the next branch in one pass.
+//   mi_xielu_map, mi_relu2_map  one activation, value by value.
 //   mi_scale_f32             x *= s in place (fp32).
 #include "common.cuh"
 
@@ -381,8 +383,15 @@ extern "C" int mi_token_gate(const void* z, int z_stride, int z_dtype, const voi
   MI_RETURN_LAUNCH_STATUS();
 }
 
-template <typename T, int V>
-__global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n, float a, float b) {
+// one activation of single values: ACT 0 mi_xielu with a and b, 1 mi_relu2
+template <typename T, int ACT>
+__device__ __forceinline__ float activated(float z, float a, float b) {
+  if (ACT == 1) return mi_relu2(z);
+  return sizeof(T) == 2 ? mi_xielu_bf16(z, a, b) : mi_xielu(z, a, b);
+}
+
+template <typename T, int V, int ACT>
+__global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n, float a, float b) {
   mi_pdl_enter();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
     if (V == 8) {                    // bfloat16, eight values per access
@@ -391,31 +400,154 @@ __global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, size_
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
-        const __nv_bfloat162 o = __floats2bfloat162_rn(mi_xielu_bf16(f.x, a, b), mi_xielu_bf16(f.y, a, b));
+        const __nv_bfloat162 o = __floats2bfloat162_rn(activated<T, ACT>(f.x, a, b), activated<T, ACT>(f.y, a, b));
         w[j] = *reinterpret_cast<const uint32_t*>(&o);
       }
       reinterpret_cast<uint4*>(out)[idx] = v;
     } else {
       const float z = mi_to_float(x[idx]);
-      out[idx] = mi_from_float<T>(sizeof(T) == 2 ? mi_xielu_bf16(z, a, b) : mi_xielu(z, a, b));
+      out[idx] = mi_from_float<T>(activated<T, ACT>(z, a, b));
     }
   }
 }
 
-// out = xielu(x) value by value (mi_xielu); out may be x
-extern "C" int mi_xielu_map(const void* x, void* out, long long n, float a, float b, int dtype, cudaStream_t stream) {
+template <int ACT>
+static int activation_map(const void* x, void* out, long long n, float a, float b, int dtype, cudaStream_t stream) {
   if (n <= 0) return 0;
   const bool eight = dtype == MI_DTYPE_BF16 && n % 8 == 0 && mi_aligned(x, 16) && mi_aligned(out, 16);
   const size_t items = eight ? (size_t)n / 8 : (size_t)n;
   const int blocks = (int)((items + 255) / 256 < 8192 ? (items + 255) / 256 : 8192);
   if (dtype == MI_DTYPE_F32)
-    MI_LAUNCH((xielu_kernel<float, 1>), blocks, 256, 0, stream, (const float*)x, (float*)out, items, a, b);
+    MI_LAUNCH((activation_kernel<float, 1, ACT>), blocks, 256, 0, stream, (const float*)x, (float*)out, items, a, b);
   else if (dtype == MI_DTYPE_BF16 && eight)
-    MI_LAUNCH((xielu_kernel<bf16, 8>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
+    MI_LAUNCH((activation_kernel<bf16, 8, ACT>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
   else if (dtype == MI_DTYPE_BF16)
-    MI_LAUNCH((xielu_kernel<bf16, 1>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
+    MI_LAUNCH((activation_kernel<bf16, 1, ACT>), blocks, 256, 0, stream, (const bf16*)x, (bf16*)out, items, a, b);
   else
-    MI_REFUSE("xielu: unknown dtype %d", dtype);
+    MI_REFUSE("activation: unknown dtype %d", dtype);
+  MI_RETURN_LAUNCH_STATUS();
+}
+
+// value by value, out may be x: mi_xielu with a and b; mi_relu2
+extern "C" int mi_xielu_map(const void* x, void* out, long long n, float a, float b, int dtype, cudaStream_t stream) {
+  return activation_map<0>(x, out, n, a, b, dtype, stream);
+}
+extern "C" int mi_relu2_map(const void* x, void* out, long long n, int dtype, cudaStream_t stream) {
+  return activation_map<1>(x, out, n, 0.f, 0.f, dtype, stream);
+}
+
+// Two norms with the sum between them, a block per row: r = stream + mult * y * rsqrt(mean(y^2) + eps_y) * gain_y
+// (y the branch whose norm stands behind it), out = r * rsqrt(mean(r^2) + eps_r) * gain_r.  The stream takes r in
+// place; with `rows` only the listed rows run, their results side by side in `out`, and the stream stays as it is.
+// HELD > 0: a thread keeps HELD pieces of four values in registers between the passes; 0: any width, values one by
+// one, r kept in shared memory.
+template <typename T, int HELD>
+__global__ void __launch_bounds__(512)
+branch_norm_then_norm_kernel(float* __restrict__ stream, const T* __restrict__ branch, int branch_stride,
+                             const float* __restrict__ gain_y, float eps_y, float mult,
+                             const float* __restrict__ gain_r, float eps_r, const int* __restrict__ rows,
+                             T* __restrict__ out, int H) {
+  mi_pdl_enter();
+  __shared__ float red[32];
+  extern __shared__ float kept[];
+  const int t = rows ? rows[blockIdx.x] : (int)blockIdx.x;
+  float* sr = stream + (size_t)t * H;
+  const T* yr = branch + (size_t)t * branch_stride;
+  T* dst = out + (size_t)blockIdx.x * H;
+  if constexpr (HELD == 0) {
+    float sq = 0.f;
+    for (int k = threadIdx.x; k < H; k += blockDim.x) {
+      const float v = mi_to_float(yr[k]);
+      sq += v * v;
+    }
+    const float ry = mult / sqrtf(mi_block_sum(sq, red) / (float)H + eps_y);
+    sq = 0.f;
+    for (int k = threadIdx.x; k < H; k += blockDim.x) {
+      const float r = sr[k] + mi_to_float(yr[k]) * ry * gain_y[k];
+      if (!rows) sr[k] = r;
+      kept[k] = r;
+      sq += r * r;
+    }
+    const float rr = 1.f / sqrtf(mi_block_sum(sq, red) / (float)H + eps_r);
+    for (int k = threadIdx.x; k < H; k += blockDim.x) dst[k] = mi_from_float<T>(kept[k] * rr * gain_r[k]);
+  } else {
+    float y[HELD > 0 ? HELD : 1][4], r[HELD > 0 ? HELD : 1][4];
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < HELD; ++i) {
+      const int k = 4 * (threadIdx.x + i * blockDim.x);
+      if (k < H) {
+        Vec4<T> a;
+        a.load(yr + k);
+        a.get(y[i]);
+        Vec4<float> b;
+        b.load(sr + k);
+        b.get(r[i]);
+        sq += y[i][0] * y[i][0] + y[i][1] * y[i][1] + y[i][2] * y[i][2] + y[i][3] * y[i][3];
+      }
+    }
+    const float ry = mult / sqrtf(mi_block_sum(sq, red) / (float)H + eps_y);
+    sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < HELD; ++i) {
+      const int k = 4 * (threadIdx.x + i * blockDim.x);
+      if (k < H) {
+        float g[4];
+        Vec4<float> b;
+        b.load(gain_y + k);
+        b.get(g);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          r[i][e] += y[i][e] * ry * g[e];
+          sq += r[i][e] * r[i][e];
+        }
+        if (!rows) {
+          b.set(r[i]);
+          b.store(sr + k);
+        }
+      }
+    }
+    const float rr = 1.f / sqrtf(mi_block_sum(sq, red) / (float)H + eps_r);
+#pragma unroll
+    for (int i = 0; i < HELD; ++i) {
+      const int k = 4 * (threadIdx.x + i * blockDim.x);
+      if (k < H) {
+        float g[4];
+        Vec4<float> b;
+        b.load(gain_r + k);
+        b.get(g);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) g[e] *= r[i][e] * rr;
+        Vec4<T> o;
+        o.set(g);
+        o.store(dst + k);
+      }
+    }
+  }
+}
+
+extern "C" int mi_branch_norm_then_norm(float* stream, const void* branch, int branch_stride, const float* gain_y,
+                                        float eps_y, float mult, const float* gain_r, float eps_r, const int* rows,
+                                        void* out, int M, int H, int dtype, cudaStream_t stream_) {
+  if (M <= 0) return 0;
+  if (H <= 0 || branch_stride < H) MI_REFUSE("norms: bad width %d or row stride %d", H, branch_stride);
+  if (!stream || !branch || !gain_y || !gain_r || !out) MI_REFUSE("norms: a stream, a branch, two gains and an output");
+  if (dtype != MI_DTYPE_F32 && dtype != MI_DTYPE_BF16) MI_REFUSE("norms: unknown dtype %d", dtype);
+  const bool four = H % 4 == 0 && branch_stride % 4 == 0 && mi_aligned(stream, 16) && mi_aligned(branch, 16) &&
+                    mi_aligned(gain_y, 16) && mi_aligned(gain_r, 16) && mi_aligned(out, 16);
+  const int quads = H / 4;
+#define MI_NORMS(HELD, THREADS, SMEM)                                                                                      do {                                                                                                                       if (dtype == MI_DTYPE_F32)                                                                                                 MI_LAUNCH((branch_norm_then_norm_kernel<float, HELD>), M, THREADS, SMEM, stream_, stream, (const float*)branch,                    branch_stride, gain_y, eps_y, mult, gain_r, eps_r, rows, (float*)out, H);                                    else                                                                                                                       MI_LAUNCH((branch_norm_then_norm_kernel<bf16, HELD>), M, THREADS, SMEM, stream_, stream, (const bf16*)branch,                      branch_stride, gain_y, eps_y, mult, gain_r, eps_r, rows, (bf16*)out, H);                                   } while (0)
+  if (four && quads <= 512) {            // threads: the row's pieces, rounded up to whole warps
+    MI_NORMS(1, ((quads + 31) / 32) * 32, 0);
+  } else if (four && quads <= 1024) {
+    MI_NORMS(2, 512, 0);
+  } else if (four && quads <= 2048) {
+    MI_NORMS(4, 512, 0);
+  } else {
+    if (H > 12000) MI_REFUSE("norms: rows of %d values are not taken", H);
+    MI_NORMS(0, 256, (size_t)H * sizeof(float));
+  }
+#undef MI_NORMS
   MI_RETURN_LAUNCH_STATUS();
 }
 

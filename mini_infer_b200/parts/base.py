@@ -55,13 +55,16 @@ class KVNeed:
     ``value_dim``: size of a value per head where it is not ``head_dim`` (keys keep ``head_dim``);
     0: nothing is kept beside the keys (the mixer finds its values in them).
     ``chunk``: a query reads only the keys of its own chunk of ``chunk`` positions (counted from
-    position 0), so whole chunks behind the sequence's end are never read again (None: no chunks)."""
+    position 0), so whole chunks behind the sequence's end are never read again (None: no chunks).
+    ``keep_first``: beside its window a query also reads the first ``keep_first`` positions of its sequence, so
+    the pages that hold them are never given back."""
 
     kv_heads: int
     head_dim: int
     window: int | None = None
     value_dim: int | None = None
     chunk: int | None = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -303,7 +306,8 @@ class StreamCopy(BranchSum):
 class PendingBranch(BranchSum):
     """What a layer hands on when its last branch has run but not what stands behind it: ``norm`` (a norm
     with ``add_branch``) is still to take the branch's output ``branch`` and add it to the stream.  Handed
-    only to a stream part that asks for it (``StreamPart.finishes_branch``)."""
+    to a stream part that asks for it (``StreamPart.finishes_branch``), or to a norm in front of the next
+    branch that runs both norms as one (``RMSNorm``)."""
 
     norm: "Norm | None" = None
     branch: torch.Tensor | None = None
@@ -427,6 +431,10 @@ class Arrangement:
     # whether the arrangement runs an input part in front of its mixer (``mixer_input``)
     takes_mixer_input: ClassVar[bool] = False
     mixer_input: "InputPart | None" = None
+    # whether the arrangement has norms behind its branches beside the ones in front of them
+    takes_branch_norms: ClassVar[bool] = False
+    mixer_branch_norm: "Norm | None" = None
+    feed_forward_branch_norm: "Norm | None" = None
 
     def __init__(self, mixer: Mixer, feed_forward: FeedForward, mixer_norm: Norm,
                  feed_forward_norm: Norm, position: Position | None) -> None:
@@ -440,6 +448,7 @@ class Arrangement:
         ps: list[Part] = [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
         if self.mixer_input is not None:
             ps.append(self.mixer_input)
+        ps.extend(n for n in (self.mixer_branch_norm, self.feed_forward_branch_norm) if n is not None)
         if self.position is not None:
             ps.append(self.position)
         return ps
@@ -514,7 +523,7 @@ def register_input_part(kind: str, cls, *, replace: bool = False) -> None:
 
 
 def lookup(family: str, kind: str):
-    from . import builtin, depth, experts, latent, mixers  # noqa: F401  (register the parts that ship with the package)
+    from . import attention, builtin, depth, experts, latent, mixers  # noqa: F401  (register the parts that ship with the package)
 
     try:
         return _REGISTRIES[family][kind]

@@ -113,6 +113,8 @@ class RMSNorm(Norm):
             if x.norm is not self or rows is not None:
                 raise ValueError("a deferred norm was handed to another norm than the one it was made for")
             return x, x.residual
+        if isinstance(x, PendingBranch):
+            return self._forward_pending(x, residual, rows)
         if isinstance(x, BranchSum) or (residual is None and x.dtype == torch.float32 and self.dtype != torch.float32):
             return self._forward_sum(x, residual, rows)
         if rows is not None:
@@ -121,6 +123,17 @@ class RMSNorm(Norm):
         out = ops.add_rmsnorm(x, self.weight, self.eps, residual_in=residual,
                               residual_out=new_residual)
         return out, new_residual
+
+    def _forward_pending(self, x, residual, rows):
+        """The norm that stands behind the branch before (a ``BranchRMSNorm``), the sum and this norm as one
+        kernel; the stream is updated in place.  With ``rows`` only those rows run, and no stream is left."""
+        if not isinstance(x.norm, BranchRMSNorm):
+            raise ValueError("this norm finishes branches whose norm is a BranchRMSNorm")
+        if getattr(self, "_gain32", None) is None:
+            self._gain32 = self.weight.to(torch.float32).contiguous()
+        out = ops.branch_norm_then_norm(residual, x.branch, x.norm.weight, x.norm.eps, x.norm.mult, self._gain32,
+                                        self.eps, self.dtype, rows=rows)
+        return out, (None if rows is not None else residual)
 
     def _forward_sum(self, x, residual, rows):
         """Several addends at once, none of them rounded on the way: the outputs of parallel
@@ -320,10 +333,33 @@ def rotary_inv_freq(head_dim: int, theta: float, rotary_dim: int | None = None,
     return torch.where(in_between, blended, slowed)
 
 
+def yarn_freq64(over: int, theta: float, rotary_dim: int, scaling: dict) -> list[float]:
+    """Frequencies (float64) of the YaRN rescale: with ``t(n) = over ln(L / (2 pi n)) / (2 ln theta)`` the pair that
+    makes ``n`` turns over the original length ``L``, pairs up to ``floor(t(beta_fast))`` keep ``theta^(-2i / over)``,
+    pairs from ``ceil(t(beta_slow))`` on turn ``factor`` times slower, and the share of the slow frequency grows
+    linearly with the pair's index between them."""
+    factor, L = float(scaling["factor"]), float(scaling["original_max_position_embeddings"])
+
+    def pair_of(turns: float) -> float:
+        return over * math.log(L / (turns * 2.0 * math.pi)) / (2.0 * math.log(theta))
+
+    first = max(math.floor(pair_of(float(scaling["beta_fast"]))), 0)
+    last = min(math.ceil(pair_of(float(scaling["beta_slow"]))), over - 1)
+    span = max(last - first, 0.001)
+    out = []
+    for i in range(rotary_dim // 2):
+        f = float(theta) ** (-2.0 * i / over)
+        slow = min(max((i - first) / span, 0.0), 1.0)
+        out.append(f / factor * slow + f * (1.0 - slow))
+    return out
+
+
 def rotary_freq64(over: int, theta: float, rotary_dim: int, scaling: dict | None) -> torch.Tensor:
     """The same frequencies in float64 from end to end (``theta^(-2i / over)`` for ``i < rotary_dim / 2``, with
     the three bands of the rescale where ``scaling`` is given), for kernels that form the angle in double
     precision."""
+    if scaling is not None and scaling.get("type") == "yarn":
+        return torch.tensor(yarn_freq64(over, theta, rotary_dim, scaling), dtype=torch.float64)
     out = []
     for i in range(rotary_dim // 2):
         f = float(theta) ** (-2.0 * i / over)
@@ -347,7 +383,9 @@ class RotaryPosition(Position):
     and cosine are fp32 and computed in the kernel; each rotated value is rounded once.
 
     params: ``head_dim``, ``theta``, optional ``rotary_dim`` (default ``head_dim``),
-    optional ``scaling`` (the llama3 mapping), optional ``span`` (``"head"``, the default: dimension
+    optional ``scaling`` (the llama3 mapping, or with ``type`` ``"yarn"``: ``factor``,
+    ``original_max_position_embeddings``, ``beta_fast``, ``beta_slow``; sines and cosines are then multiplied by
+    ``0.1 ln(factor) + 1``, ``multiplier``, and only a mixer whose own kernel rotates takes it), optional ``span`` (``"head"``, the default: dimension
     ``i`` turns with ``theta^(-2i / head_dim)``; ``"rotated"``: with ``theta^(-2i / rotary_dim)``).
 
     A mixer whose own kernel rotates reads ``rotary_dim`` and ``freq64`` (the frequencies in float64:
@@ -363,23 +401,40 @@ class RotaryPosition(Position):
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= d:
             raise ValueError(f"{self.rotary_dim} rotated dimensions of a head of {d}")
         over = d if span == "head" else self.rotary_dim
-        self.inv_freq = rotary_inv_freq(
-            over, float(self.param("theta")), self.rotary_dim, self.spec.params.get("scaling")
-        ).to(device)
+        scaling = self.spec.params.get("scaling")
+        self.multiplier, self.inv_freq = 1.0, None
+        if scaling is not None and scaling.get("type") == "yarn":
+            self.multiplier = 0.1 * math.log(float(scaling["factor"])) + 1.0
+        else:
+            self.inv_freq = rotary_inv_freq(over, float(self.param("theta")), self.rotary_dim, scaling).to(device)
         self.freq64 = rotary_freq64(over, float(self.param("theta")), self.rotary_dim,
                                     self.spec.params.get("scaling")).to(device)
         # layers with the same frequencies share one table per step
         self._table_key = (d, self.rotary_dim, float(self.param("theta")), repr(self.spec.params.get("scaling")), span)
 
+    def _plain(self) -> torch.Tensor:
+        if self.inv_freq is None:
+            raise ValueError("this rescale of the rotation needs a mixer whose own kernel rotates")
+        return self.inv_freq
+
     def encode(self, qkv, nq, nkv, head_dim, ctx):
-        ops.rope_write(qkv, nq, nkv, head_dim, positions=ctx.positions, inv_freq=self.inv_freq,
+        ops.rope_write(qkv, nq, nkv, head_dim, positions=ctx.positions, inv_freq=self._plain(),
                        rotary_dim=self.rotary_dim)
+
+    def step_angles(self, ctx):
+        """Sines and cosines of this step's positions, ``[tokens, rotary_dim]`` fp32 (per token the sines, then the
+        cosines, each times ``multiplier``), from angles in double precision.  Layers share one table per step."""
+        key = ("rope_angles", self._table_key)
+        table = ctx.scratch.get(key)
+        if table is None:
+            table = ctx.scratch[key] = ops.rope_angles(ctx.positions, self.freq64, self.multiplier)
+        return table
 
     def step_table(self, ctx, head_dim):
         """Sines and cosines of this step's positions for a mixer that rotates by itself, or
         None where that is not possible (a rotary width below the head size).  Layers share one
         table per step: it depends on the positions and the frequencies only."""
-        if self.rotary_dim != head_dim:
+        if self.rotary_dim != head_dim or self.inv_freq is None:
             return None
         key = ("rope_table", self._table_key)
         table = ctx.scratch.get(key)
@@ -390,7 +445,7 @@ class RotaryPosition(Position):
     def rotate_and_store(self, qkv, nq, nkv, head_dim, ctx, cache):
         if cache.writes and cache.k is not None:
             ops.rope_write(qkv, nq, nkv, head_dim, positions=ctx.positions,
-                           inv_freq=self.inv_freq, rotary_dim=self.rotary_dim,
+                           inv_freq=self._plain(), rotary_dim=self.rotary_dim,
                            slots=ctx.groups[cache.group].slots, kcache=cache.k, vcache=cache.v)
         else:
             self.encode(qkv, nq, nkv, head_dim, ctx)
@@ -578,9 +633,10 @@ class ClampedGLU(FeedForward):
 
 
 class ActivatedMLP(FeedForward):
-    """``down(act(up(x)))`` without gate and biases.  ``activation`` ``"xielu"``: with ``a = softplus(p)`` and ``b =
+    """``down(act(up(x)))`` without gate and biases, ``act`` in fp32.  ``activation`` ``"relu2"``: the square of
+    ``max(z, 0)``.  ``"xielu"``: with ``a = softplus(p)`` and ``b =
     1/2 + softplus(q)`` of the two numbers in the tensor ``act``, ``act(z) = a z^2 + z / 2`` for ``z > 0`` and
-    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``, in fp32.
+    ``b (e^z - 1 - z) + z / 2`` for ``z <= 0``.
 
     params: ``hidden_size``, ``intermediate_size``, ``activation``.  tensors: ``up``, ``down`` and, for
     ``"xielu"``, ``act [2]``.
@@ -594,13 +650,18 @@ class ActivatedMLP(FeedForward):
 
     def param_decls(self):
         H, I = int(self.param("hidden_size")), int(self.param("intermediate_size"))
-        return {"up": ParamDecl((I, H)), "down": ParamDecl((H, I)), "act": ParamDecl((2,), "table")}
+        decls = {"up": ParamDecl((I, H)), "down": ParamDecl((H, I))}
+        if self.activation == "xielu":
+            decls["act"] = ParamDecl((2,), "table")
+        return decls
 
     def bind(self, tensors, dtype, device):
         self.up = _as_compute(tensors["up"], dtype).contiguous()
         self.down = Linear(_as_compute(tensors["down"], dtype).contiguous())
-        p, q = (float(v) for v in torch.nn.functional.softplus(tensors["act"].to(torch.float64).cpu()))
-        self.act_params = (p, 0.5 + q)
+        self.act_params = (0.0, 0.0)
+        if self.activation == "xielu":
+            p, q = (float(v) for v in torch.nn.functional.softplus(tensors["act"].to(torch.float64).cpu()))
+            self.act_params = (p, 0.5 + q)
 
     def forward(self, x, ctx):
         return self.down(ops.linear_activated(x, self.up, self.activation, self.act_params))
@@ -786,6 +847,23 @@ class BranchNormBlock(Arrangement):
         return StreamCopy.of(h), stream
 
 
+class SandwichNormBlock(Arrangement):
+    """``h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h)))``: an RMS norm in front of every branch and a
+    ``BranchRMSNorm`` (the residual factor in it) behind it.  The norm behind a branch, the sum and the norm in
+    front of the next branch, be it this layer's or the next one's, run as one kernel: the block hands on its
+    last branch as a ``PendingBranch``.  A layer without a feed-forward (``no_feed_forward``) is the mixer's half."""
+
+    takes_branch_norms = True
+
+    def forward(self, x, residual, ctx, cache):
+        a, stream = self.mixer_norm.forward(x, residual)
+        last = PendingBranch.of(self.mixer_branch_norm, self.mixer.forward(a, ctx, cache, self.position))
+        if not isinstance(self.feed_forward, NoFeedForward):
+            b, stream = self.feed_forward_norm.forward(last, stream)
+            last = PendingBranch.of(self.feed_forward_branch_norm, self.feed_forward.forward(b, ctx))
+        return last, stream
+
+
 class TokenSideInput(StreamPart):
     """What a layer takes from the token itself, behind its branches: with ``e`` the columns ``[index *
     dim, (index + 1) * dim)`` of the token's row of a table shared by all layers, ``g = gelu_tanh(W_gate h)
@@ -841,6 +919,7 @@ register_norm("branch_rmsnorm", BranchRMSNorm, replace=True)
 register_norm("branch_layernorm", BranchLayerNorm, replace=True)
 register_feed_forward("activated_mlp", ActivatedMLP, replace=True)
 register_arrangement("branch_norm", BranchNormBlock, replace=True)
+register_arrangement("sandwich_norm", SandwichNormBlock, replace=True)
 register_stream_part("token_side_input", TokenSideInput, replace=True)
 register_norm("same_norm", SameNorm, replace=True)
 register_position("rotary_interleaved", InterleavedRotary, replace=True)

@@ -63,6 +63,13 @@ class DecoderModel:
                 if not block.takes_mixer_input:
                     raise ValueError(f"arrangement {layer.arrangement!r} runs no input part in front of its mixer")
                 block.mixer_input = build_part("input", layer.mixer_input)
+            for name in ("mixer_branch_norm", "feed_forward_branch_norm"):
+                norm = getattr(layer, name)
+                if (norm is not None) != block.takes_branch_norms:
+                    raise ValueError(f"arrangement {layer.arrangement!r} "
+                                     f"{'needs' if norm is None else 'has no place for'} {name}")
+                if norm is not None:
+                    setattr(block, name, build_part("norm", norm))
             self.blocks.append(block)
         self.schedule = spec.schedule
         # stream parts that run before a schedule entry (None where an entry has none)

@@ -45,6 +45,8 @@ class LayerSpec:
     the residual additions stand).  ``position`` is the position encoding the
     mixer applies (``None``: the mixer uses none).  ``mixer_input``: a registered input part that
     works on what the mixer reads, right before it (``None``: the mixer reads it as it is).
+    ``mixer_branch_norm`` and ``feed_forward_branch_norm``: norms behind the branches of a layer that also has
+    norms in front of them (``None``: nothing behind a branch, or the arrangement puts the only norm there).
     """
 
     mixer: PartSpec
@@ -54,6 +56,8 @@ class LayerSpec:
     position: PartSpec | None = None
     arrangement: str = "prenorm"
     mixer_input: PartSpec | None = None
+    mixer_branch_norm: PartSpec | None = None
+    feed_forward_branch_norm: PartSpec | None = None
 
 
 @dataclass(frozen=True)
