@@ -656,6 +656,92 @@ def run_zinesun_designs(args) -> int:
     return 0
 
 
+# The Gotivik architecture at the same widths: layers alternate differential attention over the whole past (heads of
+# two maps of 64 over values of 128: rows of Llama's sizes) and windowed attention behind short convolutions, each with
+# a squared-ReLU unit of the same number of weights as Llama's gated one.
+GOTIVIK_SIZES = {"2k": dict(window=1024, ff=8448), "4k": dict(window=2048, ff=16512)}
+
+
+def gotivik_design(s: dict, g: dict, layers: int) -> tuple[dict, dict]:
+    """(Gotivik, Llama) configurations of equal width, heads, cached numbers per token and feed-forward weights."""
+    H, n, kv, d = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    mlp = {"kind": "dense", "ff": g["ff"]}
+    diff = {"type": "attention_2", "mlp": mlp,
+            "mixer": {"heads": n, "kv_heads": kv, "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5, "softcap": 50.0,
+                      "q_temp": {"coef": 0.1, "every": 4096}, "diff": 0.2}}
+    window = {"type": "attention", "mlp": mlp,
+              "mixer": {"heads": n, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "conv": 4,
+                        "mask": {"size": g["window"], "keep_first": 4},
+                        "rot": {"base": 10000.0, "dims": d // 2,
+                                "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    raw = {"architecture": "Gotivik", "vocab": s["vocab"], "width": H, "norm": {"eps": 1e-6}, "residual_mult": 0.25,
+           "layers": [window if i % 2 else diff for i in range(layers)]}
+    llama = dict(LLAMA_8B, hidden_size=H, num_attention_heads=n, num_key_value_heads=kv, head_dim=d,
+                 intermediate_size=s["ff"], vocab_size=s["vocab"], num_hidden_layers=layers)
+    return raw, llama
+
+
+def gotivik_numbers(s: dict, g: dict, layers: int, batch: int, context: float, tokens: int) -> tuple[float, float]:
+    """(bytes a decode step must move, floating-point operations of a prefill of ``tokens``): weights once, the cached
+    rows a token sees; products per token, both maps' scores (of ``dim / 2`` each) and sums."""
+    H, n, kv, d = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    n_win = layers // 2
+    n_diff = layers - n_win
+    weights = layers * (H * d * (2 * n + 2 * kv) + 2 * H * g["ff"]) + n_diff * n * H
+    w = min(g["window"] + 4, tokens)
+    causal, windowed = tokens * (tokens + 1) / 2.0, tokens * w - w * (w - 1) / 2.0
+    nbytes = 2.0 * (weights + s["vocab"] * H) + \
+        4.0 * batch * kv * d * (n_diff * context + n_win * min(g["window"] + 4, context))
+    flops = 2.0 * tokens * weights + 2.0 * s["vocab"] * H + n_diff * 2.0 * causal * n * 2 * (d // 2 + d) \
+        + n_win * 2.0 * windowed * n * 2 * d
+    return nbytes, flops
+
+
+def run_gotivik_designs(args) -> int:
+    import torch
+
+    from mini_infer_b200.engine import ModelRunner
+
+    peaks = load_peaks()
+    warmup = max(3, args.warmup)
+    out = {"scenario": "designs", "design": "gotivik", "dtype": "bf16", "data": "synthetic", "batch": args.batch,
+           "context": args.context, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks, "sizes": {}}
+    clocks = ClockSampler()
+    clocks.start()
+    for name in args.design_sizes.split(","):
+        s, g = LILULIX_SIZES[name], GOTIVIK_SIZES[name]
+        layers = args.layers or 4
+        raw, llama = gotivik_design(s, g, layers)
+        cap = args.batch * (args.context + args.steps + warmup + 64) + 2 * PREFILL_TOKENS
+        row = {"layers": layers}
+        for label, cfg in (("gotivik", raw), ("llama", llama)):
+            runner = ModelRunner.from_random(cfg, seed=0, gain_std=0.0, device="cuda:0", dtype="bfloat16",
+                                             num_blocks=cap // PAGE + 8, block_size=PAGE, max_requests=args.batch,
+                                             cuda_graph=True)
+            ms, launches = time_decode(runner, args.batch, args.context, args.steps, warmup)
+            pms = time_prefill(runner, PREFILL_TOKENS, repeats=3, warmup=2)
+            mid = args.context + warmup + args.steps / 2.0
+            if label == "gotivik":
+                nbytes, flops = gotivik_numbers(s, g, layers, args.batch, mid, PREFILL_TOKENS)
+            else:
+                flops = prefill_flops(cfg, layers, PREFILL_TOKENS)
+                nbytes = decode_bytes(cfg, layers, args.batch, mid)
+            row[label] = {
+                "decode_tok_s": round(args.batch * 1000.0 / ms, 1), "decode_ms": round(ms, 4),
+                "decode_gbs": round(nbytes / (ms * 1e-3) / 1e9, 1),
+                "decode_frac_of_hbm": round(nbytes / (ms * 1e-3) / 1e9 / peaks["hbm_gbs"], 4),
+                "prefill_tok_s": round(PREFILL_TOKENS * 1000.0 / pms, 1), "prefill_ms": round(pms, 3),
+                "prefill_frac_of_bf16": round(flops / (pms * 1e-3) / (peaks["bf16_tflops"] * 1e12), 4),
+                "launches_per_decode_step": launches // max(1, args.steps),
+            }
+            del runner
+            torch.cuda.empty_cache()
+        out["sizes"][name] = row
+    out["clocks"] = clocks.stop()
+    print(json.dumps(out))
+    return 0
+
+
 def run_vepevik_designs(args) -> int:
     import torch
 
@@ -1222,9 +1308,9 @@ def main() -> int:
                     help="decode: the contract line; long-mixed: many requests of very different lengths "
                          "through the scheduler (a line of its own); serving: the reference's published "
                          "workload, 1024 tokens in and 128 out, single requests and 16 together (a line of its own); "
-                         "designs: the Ruvurax (or, with --design, the Lilulix, the Vepevik, the Ruburax or the Zinesun) architecture beside Llama at equal sizes, prefill and decode "
+                         "designs: the Ruvurax (or, with --design, the Lilulix, the Vepevik, the Ruburax, the Zinesun or the Gotivik) architecture beside Llama at equal sizes, prefill and decode "
                          "(a line of its own)")
-    ap.add_argument("--design", default="ruvurax", choices=["ruvurax", "lilulix", "vepevik", "ruburax", "zinesun"],
+    ap.add_argument("--design", default="ruvurax", choices=["ruvurax", "lilulix", "vepevik", "ruburax", "zinesun", "gotivik"],
                     help="designs: which architecture stands beside Llama")
     ap.add_argument("--design-sizes", default="2k,4k", help="designs: which of the sizes " + ",".join(DESIGN_SIZES))
     ap.add_argument("--requests", type=int, default=64, help="long-mixed: requests started together")
@@ -1260,6 +1346,8 @@ def main() -> int:
             return run_ruburax_designs(args)
         if args.design == "zinesun":
             return run_zinesun_designs(args)
+        if args.design == "gotivik":
+            return run_gotivik_designs(args)
         return run_lilulix_designs(args) if args.design == "lilulix" else run_designs(args)
     warmup = max(3, args.warmup)
 

@@ -23,7 +23,7 @@
 MI_DEFINE_ERROR_API()
 
 #define STAGE_TILE 16      // tokens per tile of mi_conv_rope_store
-#define STAGE_THREADS 128
+#define STAGE_THREADS 64
 #define STAGE_MAX_TAPS 16  // taps - 1 rows of state: only a portion's first tile reads them
 
 __global__ void rope_angles_kernel(const int* __restrict__ positions, const double* __restrict__ freq, float mult,
@@ -48,12 +48,22 @@ extern "C" int mi_rope_angles(const int* positions, const double* freq, float mu
   MI_RETURN_LAUNCH_STATUS();
 }
 
-// V consecutive values as one access (4) or one by one (1).
+// V consecutive values as one access (8 of bfloat16, or 4) or one by one (1).
 template <typename T, int V>
 struct Piece {
   float f[V];
   __device__ __forceinline__ void load(const T* p) {
-    if constexpr (V == 4) {
+    if constexpr (V == 8) {
+      static_assert(V != 8 || sizeof(T) == 2, "eight values of bfloat16 are one access");
+      const uint4 v = *reinterpret_cast<const uint4*>(p);
+      const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
+        f[2 * j] = g.x;
+        f[2 * j + 1] = g.y;
+      }
+    } else if constexpr (V == 4) {
       Vec4<T> v;
       v.load(p);
       v.get(f);
@@ -62,7 +72,15 @@ struct Piece {
     }
   }
   __device__ __forceinline__ void store(T* p) const {
-    if constexpr (V == 4) {
+    if constexpr (V == 8) {
+      uint32_t w[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const __nv_bfloat162 g = __floats2bfloat162_rn(f[2 * j], f[2 * j + 1]);
+        w[j] = *reinterpret_cast<const uint32_t*>(&g);
+      }
+      *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+    } else if constexpr (V == 4) {
       Vec4<T> v;
       v.set(f);
       v.store(p);
@@ -72,7 +90,10 @@ struct Piece {
   }
 };
 
-// TAPS > 0: that many taps, the weights of a thread's channels in registers; 0: `taps` of them, read as they are used.
+// A thread takes V channels and the V channels that are turned against them (half the rotated span further on; among
+// the dimensions that pass, half of those), and walks a run of the tile's tokens.  TAPS > 0: that many taps; the
+// weights and the last TAPS - 1 inputs of the thread's channels stay in registers, so every projected value is read
+// once per run.  0: `taps` of them, weights and inputs read as they are used.
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(STAGE_THREADS)
 conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __restrict__ weight, int taps_any,
@@ -83,6 +104,7 @@ conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __
                        T* __restrict__ kcache, T* __restrict__ vcache, int page_size) {
   mi_pdl_enter();
   constexpr int EPC = 16 / (int)sizeof(T);
+  constexpr int NW = TAPS > 0 ? TAPS : 1, NH = TAPS > 1 ? TAPS - 1 : 1;
   const int taps = TAPS > 0 ? TAPS : taps_any, C = (nq + nkv) * d + nkv * dv;
   const int tile = blockIdx.x, head = blockIdx.y;
   const int b = tile_req[tile], tok0 = tile_tok0[tile];
@@ -93,59 +115,98 @@ conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __
   const int base = is_v ? (nq + nkv) * d + (head - nq - nkv) * dv : head * d;      // the head's first channel
   const int kvh = is_v ? head - nq - nkv : head - nq;
   float* past = state ? state + (long long)state_slot[b] * state_stride : nullptr;
-  const int n_pair = half / V, n_items = n_pair + (width - turn) / V;
+  // items: pairs of pieces; with V = 1 an odd number of passing dimensions leaves the last item without a partner
+  const int rest = width - turn, rest_half = (rest / V + 1) / 2 * V;
+  const int n_turn = half / V, n_items = n_turn + rest_half / V;
   const int lanes = min(n_items, STAGE_THREADS), groups = STAGE_THREADS / lanes;
   const int group = threadIdx.x / lanes, lane = threadIdx.x - group * lanes;
   const int each = (ntok + groups - 1) / groups;
   const int t_begin = group * each, t_end = group < groups ? min(ntok, t_begin + each) : 0;
   const int mask = mi_swizzle_mask_rows(width, (int)sizeof(T));
 
-  // the convolution of V channels from c on at the portion's token t
-  auto convolve = [&](const float (&w)[TAPS > 0 ? TAPS : 1][V], int c, int t, float (&y)[V]) {
+  // the projected values of V channels from c on at the portion's token src (negative: before the portion)
+  auto input = [&](int src, int c, Piece<T, V>& u) {
+    if (src >= 0) {
+      u.load(packed + (size_t)(qs + src) * stride + c);
+    } else {
+      const float* p = past + (size_t)(taps - 1 + src) * C + c;
 #pragma unroll
-    for (int e = 0; e < V; ++e) y[e] = 0.f;
-#pragma unroll
-    for (int j = 0; j < taps; ++j) {
-      const int src = t - taps + 1 + j;
-      Piece<T, V> u;
-      if (src >= 0) {
-        u.load(packed + (size_t)(qs + src) * stride + c);
-      } else {
-        const float* p = past + (size_t)(taps - 1 + src) * C + c;
-#pragma unroll
-        for (int e = 0; e < V; ++e) u.f[e] = p[e];
-      }
-#pragma unroll
-      for (int e = 0; e < V; ++e)
-        y[e] = fmaf(TAPS > 0 ? w[TAPS > 0 ? j : 0][e] : weight[(size_t)(c + e) * taps + j], u.f[e], y[e]);
+      for (int e = 0; e < V; ++e) u.f[e] = p[e];
     }
   };
-  auto taps_of = [&](float (&w)[TAPS > 0 ? TAPS : 1][V], int c) {
+  auto weights = [&](float (&w)[NW][V], int c) {
     if constexpr (TAPS > 0) {
 #pragma unroll
-      for (int e = 0; e < V; ++e)
+      for (int j = 0; j < TAPS; ++j) {
+        Piece<float, V> p;
+        p.load(weight + (size_t)j * C + c);
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) w[j][e] = weight[(size_t)(c + e) * TAPS + j];
+        for (int e = 0; e < V; ++e) w[j][e] = p.f[e];
+      }
+    }
+  };
+  auto history = [&](Piece<T, V> (&h)[NH], int c, int t) {      // h[j]: the input of token t - (TAPS - 1) + j
+    if constexpr (TAPS > 1) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) input(t - TAPS + 1 + j, c, h[j]);
+    }
+  };
+  auto convolve = [&](const float (&w)[NW][V], Piece<T, V> (&h)[NH], int c, int t, Piece<T, V>& y) {
+    Piece<T, V> u;
+    input(t, c, u);
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float acc = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(w[j][e], h[j].f[e], acc);
+        y.f[e] = fmaf(w[TAPS - 1][e], u.f[e], acc);
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS - 1; ++j) h[j].f[e] = h[j + 1].f[e];
+        if constexpr (TAPS > 1) h[TAPS - 2].f[e] = u.f[e];
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) y.f[e] = 0.f;
+      for (int j = 0; j < taps; ++j) {
+        Piece<T, V> v;
+        input(t - taps + 1 + j, c, v);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y.f[e] = fmaf(weight[(size_t)j * C + c + e], v.f[e], y.f[e]);
+      }
     }
   };
 
   for (int item = lane; item < n_items; item += lanes) {
-    const bool pair = item < n_pair;
-    const int k1 = pair ? item * V : turn + (item - n_pair) * V;      // within the head
-    float w1[TAPS > 0 ? TAPS : 1][V], w2[TAPS > 0 ? TAPS : 1][V];
-    taps_of(w1, base + k1);
-    if (pair) taps_of(w2, base + half + k1);
+    const bool turned = item < n_turn;
+    const int k1 = turned ? item * V : turn + (item - n_turn) * V;      // within the head
+    const int k2 = k1 + (turned ? half : rest_half);
+    const bool two = k2 < width;
+    float w1[NW][V], w2[NW][V];
+    Piece<T, V> h1[NH], h2[NH];
+    if (t_begin < t_end) {
+      weights(w1, base + k1);
+      history(h1, base + k1, tok0 + t_begin);
+      if (two) {
+        weights(w2, base + k2);
+        history(h2, base + k2, tok0 + t_begin);
+      }
+    }
+#pragma unroll 2
     for (int tt = t_begin; tt < t_end; ++tt) {
       const int t = tok0 + tt, row = qs + t;
       Piece<T, V> a, c;
-      convolve(w1, base + k1, t, a.f);
-      if (pair) {
-        convolve(w2, base + half + k1, t, c.f);
+      convolve(w1, h1, base + k1, t, a);
+      if (two) convolve(w2, h2, base + k2, t, c);
+      if (turned) {
         const float* sn = angles + (size_t)row * turn + k1;
+        Piece<float, V> s, o;
+        s.load(sn);
+        o.load(sn + half);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
           const float u = a.f[e], v = c.f[e];
-          mi_rotate(u, v, sn[e], sn[half + e], a.f[e], c.f[e]);
+          mi_rotate(u, v, s.f[e], o.f[e], a.f[e], c.f[e]);
         }
       }
       T* dst;
@@ -159,7 +220,7 @@ conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __
         dst = (is_v ? vcache : kcache) + ((size_t)(page * nkv + kvh) * page_size + offset) * width;
       }
       a.store(dst + (m ? mi_swizzled(k1, offset, m, EPC) : k1));
-      if (pair) c.store(dst + (m ? mi_swizzled(half + k1, offset, m, EPC) : half + k1));
+      if (two) c.store(dst + (m ? mi_swizzled(k2, offset, m, EPC) : k2));
     }
   }
   if (tok0 == 0 && past) {
@@ -192,8 +253,9 @@ extern "C" int mi_conv_rope_store(const void* packed, int stride, const float* w
   const int n_heads = nq + 2 * nkv;
   if (n_heads > 65535) MI_REFUSE("conv_rope_store: too many heads for one launch");
   const size_t piece = dtype == MI_DTYPE_F32 ? 16 : 8;
-  const bool four = d % 4 == 0 && dv % 4 == 0 && rot % 8 == 0 && stride % 4 == 0 && mi_aligned(packed, piece) &&
-                    mi_aligned(q_out, piece) && mi_aligned(kcache, 16) && mi_aligned(vcache, 16);
+  const bool four = d % 8 == 0 && dv % 8 == 0 && rot % 8 == 0 && stride % 4 == 0 && mi_aligned(packed, piece) &&
+                    mi_aligned(q_out, piece) && mi_aligned(kcache, 16) && mi_aligned(vcache, 16) && mi_aligned(weight, 16) &&
+                    mi_aligned(angles, 16);
   const dim3 grid((unsigned)n_tiles, (unsigned)n_heads);
 #define MI_CONV(T, V, TAPS)                                                                                           \
   MI_LAUNCH((conv_rope_store_kernel<T, V, TAPS>), grid, STAGE_THREADS, 0, stream, (const T*)packed, stride, weight,   \
@@ -201,7 +263,8 @@ extern "C" int mi_conv_rope_store(const void* packed, int stride, const float* w
             nq, nkv, d, dv, rot, angles, slots, (T*)q_out, (T*)kcache, (T*)vcache, page_size)
 #define MI_CONV_TAPS(T, V)                                                                                            \
   do {                                                                                                                \
-    if (taps == 2) MI_CONV(T, V, 2);                                                                                  \
+    if (taps == 1) MI_CONV(T, V, 1);                                                                                  \
+    else if (taps == 2) MI_CONV(T, V, 2);                                                                                  \
     else if (taps == 3) MI_CONV(T, V, 3);                                                                             \
     else if (taps == 4) MI_CONV(T, V, 4);                                                                             \
     else MI_CONV(T, V, 0);                                                                                            \
@@ -221,8 +284,9 @@ extern "C" int mi_conv_rope_store(const void* packed, int stride, const float* w
 }
 
 // grid = (tokens, parts): the pieces of a token's queries, key rows and values are numbered in one row
+#define SPLIT_THREADS 128
 template <typename T, int V>
-__global__ void __launch_bounds__(STAGE_THREADS)
+__global__ void __launch_bounds__(SPLIT_THREADS)
 split_maps_store_kernel(const T* __restrict__ packed, int stride, int k_off, int v_off, int nq, int nkv, int d, int rowd,
                         int dv, const int* __restrict__ positions, float coef, int every, const int* __restrict__ slots,
                         T* __restrict__ q_out, T* __restrict__ kcache, T* __restrict__ vcache, int page_size) {
@@ -266,21 +330,25 @@ extern "C" int mi_split_maps_store(const void* packed, int stride, int k_off, in
   if (!slots || !kcache || !vcache || page_size <= 0 || (coef != 0.f && !positions))
     MI_REFUSE("split_maps_store: keys and values need slots and pages, a temperature positions");
   const size_t piece = dtype == MI_DTYPE_F32 ? 16 : 8;
-  const bool four = d % 4 == 0 && rowd % 4 == 0 && dv % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 && stride % 4 == 0 &&
-                    mi_aligned(packed, piece) && mi_aligned(q_out, piece) && mi_aligned(kcache, 16) && mi_aligned(vcache, 16);
-  const int items = (2 * nq + nkv) * rowd + nkv * dv, per = (four ? 4 : 1) * STAGE_THREADS;
-  int parts = (items + per - 1) / per;                 // a pass each for few tokens, four passes a block for many
-  if (M >= 256) parts = (parts + 3) / 4;
+  auto fits = [&](int v, size_t align) {
+    return d % v == 0 && rowd % v == 0 && dv % v == 0 && k_off % v == 0 && v_off % v == 0 && stride % v == 0 &&
+           mi_aligned(packed, align) && mi_aligned(q_out, align) && mi_aligned(kcache, 16) && mi_aligned(vcache, 16);
+  };
+  const int V = dtype == MI_DTYPE_BF16 && fits(8, 16) ? 8 : (fits(4, piece) ? 4 : 1);
+  const int items = (2 * nq + nkv) * rowd + nkv * dv, per = V * SPLIT_THREADS;
+  int parts = (items + per - 1) / per;                 // a pass each for few tokens, two passes a block for many
+  if (M >= 256) parts = (parts + 1) / 2;
   if (parts > 64) parts = 64;
   const dim3 grid((unsigned)M, (unsigned)parts);
 #define MI_SPLIT(T, V)                                                                                               \
-  MI_LAUNCH((split_maps_store_kernel<T, V>), grid, STAGE_THREADS, 0, stream, (const T*)packed, stride, k_off, v_off, \
+  MI_LAUNCH((split_maps_store_kernel<T, V>), grid, SPLIT_THREADS, 0, stream, (const T*)packed, stride, k_off, v_off, \
             nq, nkv, d, rowd, dv, positions, coef, every, slots, (T*)q_out, (T*)kcache, (T*)vcache, page_size)
   if (dtype == MI_DTYPE_F32) {
-    if (four) MI_SPLIT(float, 4);
+    if (V == 4) MI_SPLIT(float, 4);
     else MI_SPLIT(float, 1);
   } else if (dtype == MI_DTYPE_BF16) {
-    if (four) MI_SPLIT(bf16, 4);
+    if (V == 8) MI_SPLIT(bf16, 8);
+    else if (V == 4) MI_SPLIT(bf16, 4);
     else MI_SPLIT(bf16, 1);
   } else {
     MI_REFUSE("split_maps_store: unknown dtype %d", dtype);
@@ -289,39 +357,47 @@ extern "C" int mi_split_maps_store(const void* packed, int stride, int k_off, in
   MI_RETURN_LAUNCH_STATUS();
 }
 
-// a warp per (token, head); HELD pieces of V values per lane
-template <typename T, int V, int HELD>
-__global__ void __launch_bounds__(STAGE_THREADS)
+// LANES lanes per (token, head), HELD pieces of V values per lane
+#define COMBINE_THREADS 128
+template <typename T, int V, int HELD, int LANES>
+__global__ void __launch_bounds__(COMBINE_THREADS)
 combine_maps_kernel(const T* __restrict__ heads, const T* __restrict__ gate, int gate_stride, T* __restrict__ out,
                     int out_stride, int M, int nq, int dv, float lam, float eps, float mult) {
   mi_pdl_enter();
-  const int unit = blockIdx.x * (STAGE_THREADS / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= M * nq) return;
-  const int t = unit / nq, h = unit - t * nq;
+  const int unit = blockIdx.x * (COMBINE_THREADS / LANES) + threadIdx.x / LANES, lane = threadIdx.x % LANES;
+  const bool live = unit < M * nq;
+  const int t = live ? unit / nq : 0, h = live ? unit - t * nq : 0;
   const T* a1 = heads + ((size_t)t * nq + h) * 2 * dv;
   const T* a2 = a1 + dv;
-  Piece<T, V> o[HELD];
-  float sq = 0.f;
+  const float g = gate ? mi_to_float(gate[(size_t)t * gate_stride + h]) : 0.f;
+  Piece<T, V> o[HELD], b[HELD];
 #pragma unroll
   for (int i = 0; i < HELD; ++i) {
-    const int k = (lane + 32 * i) * V;
+    const int k = (lane + LANES * i) * V;
     if (k < dv) {
-      Piece<T, V> b;
       o[i].load(a1 + k);
-      b.load(a2 + k);
+      b[i].load(a2 + k);
+    }
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < HELD; ++i)
+    if ((lane + LANES * i) * V < dv) {
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        o[i].f[e] = fmaf(-lam, b.f[e], o[i].f[e]);
+        o[i].f[e] = fmaf(-lam, b[i].f[e], o[i].f[e]);
         sq += o[i].f[e] * o[i].f[e];
       }
     }
-  }
-  float f = mult / sqrtf(mi_warp_sum(sq) / (float)dv + eps);
-  if (gate) f *= 1.f / (1.f + expf(-mi_to_float(gate[(size_t)t * gate_stride + h])));
+#pragma unroll
+  for (int s = LANES / 2; s > 0; s >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, s);
+  if (!live) return;
+  float f = mult / sqrtf(sq / (float)dv + eps);
+  if (gate) f *= 1.f / (1.f + expf(-g));
   T* dst = out + (size_t)t * out_stride + h * dv;
 #pragma unroll
   for (int i = 0; i < HELD; ++i) {
-    const int k = (lane + 32 * i) * V;
+    const int k = (lane + LANES * i) * V;
     if (k < dv) {
 #pragma unroll
       for (int e = 0; e < V; ++e) o[i].f[e] *= f;
@@ -336,19 +412,22 @@ extern "C" int mi_combine_maps(const void* heads, const void* gate, int gate_str
   if (nq <= 0 || dv <= 0 || dv > 512) MI_REFUSE("combine_maps: bad sizes (%d heads, values of %d)", nq, dv);
   const size_t piece = dtype == MI_DTYPE_F32 ? 16 : 8;
   const bool four = dv % 4 == 0 && out_stride % 4 == 0 && mi_aligned(heads, piece) && mi_aligned(out, piece);
+  const bool eight = dtype == MI_DTYPE_BF16 && dv % 8 == 0 && out_stride % 8 == 0 && mi_aligned(heads, 16) && mi_aligned(out, 16);
   const long long units = (long long)M * nq;
-  if (units > 0x7fffffffLL - 8) MI_REFUSE("combine_maps: too many rows for one launch");
-  const unsigned blocks = (unsigned)((units + STAGE_THREADS / 32 - 1) / (STAGE_THREADS / 32));
-#define MI_COMBINE(T, V, HELD)                                                                                        \
-  MI_LAUNCH((combine_maps_kernel<T, V, HELD>), blocks, STAGE_THREADS, 0, stream, (const T*)heads, (const T*)gate,     \
-            gate_stride, (T*)out, out_stride, M, nq, dv, lam, eps, mult)
+  if (units > 0x7fffffffLL - 64) MI_REFUSE("combine_maps: too many rows for one launch");
+#define MI_COMBINE(T, V, HELD, LANES)                                                                                 \
+  MI_LAUNCH((combine_maps_kernel<T, V, HELD, LANES>), (unsigned)((units * LANES + COMBINE_THREADS - 1) / COMBINE_THREADS), \
+            COMBINE_THREADS, 0, stream, (const T*)heads, (const T*)gate, gate_stride, (T*)out, out_stride, M, nq, dv,   \
+            lam, eps, mult)
 #define MI_COMBINE_SIZE(T)                                                                                            \
   do {                                                                                                                \
-    if (four && dv <= 128) MI_COMBINE(T, 4, 1);                                                                       \
-    else if (four) MI_COMBINE(T, 4, 4);                                                                               \
-    else MI_COMBINE(T, 1, 16);                                                                                        \
+    if (four && dv <= 128) MI_COMBINE(T, 4, 1, 32);                                                                   \
+    else if (four) MI_COMBINE(T, 4, 4, 32);                                                                           \
+    else MI_COMBINE(T, 1, 16, 32);                                                                                    \
   } while (0)
   if (dtype == MI_DTYPE_F32) MI_COMBINE_SIZE(float);
+  else if (dtype == MI_DTYPE_BF16 && eight && dv <= 64) MI_COMBINE(bf16, 8, 1, 8);
+  else if (dtype == MI_DTYPE_BF16 && eight && dv <= 128) MI_COMBINE(bf16, 8, 2, 8);
   else if (dtype == MI_DTYPE_BF16) MI_COMBINE_SIZE(bf16);
   else MI_REFUSE("combine_maps: unknown dtype %d", dtype);
 #undef MI_COMBINE_SIZE

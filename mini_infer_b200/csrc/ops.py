@@ -2685,7 +2685,7 @@ def conv_rope_store(packed: torch.Tensor, q_out: torch.Tensor, weight: torch.Ten
                     nq: int, nkv: int, d: int, dv: int, *, rot: int, angles: torch.Tensor | None, slots: torch.Tensor,
                     kcache: torch.Tensor, vcache: torch.Tensor) -> None:
     """The packed projection ``[M, >= (nq + nkv) d + nkv dv]`` (q, k, v side by side) through a causal convolution per
-    channel (``weight`` fp32 ``[channels, taps]``, the last tap meets the current token), then the rotation of q and
+    channel (``weight`` fp32 ``[taps, channels]``, the last tap meets the current token), then the rotation of q and
     k in the half layout on their first ``rot`` dimensions (``angles`` of ``rope_angles``).  Queries go to ``q_out [M, nq
     d]``, keys and values to their pages.  ``state`` (fp32 ``[slots, (taps - 1) * channels]``): each request's last
     projected rows, oldest first, read for a portion's first tokens and moved on.  Needs query tiles of
@@ -2697,9 +2697,9 @@ def conv_rope_store(packed: torch.Tensor, q_out: torch.Tensor, weight: torch.Ten
         raise KernelError(f"conv_rope_store: the projection must be [tokens, {C} or more]")
     if q_out.dtype != packed.dtype or q_out.shape != (M, nq * d) or not q_out.is_contiguous():
         raise KernelError("conv_rope_store: queries go to a contiguous [M, nq * d] in the packed dtype")
-    if weight.dtype != torch.float32 or weight.dim() != 2 or weight.shape[0] != C or not weight.is_contiguous():
-        raise KernelError(f"conv_rope_store: the taps must be contiguous fp32 [{C}, taps]")
-    taps = weight.shape[1]
+    if weight.dtype != torch.float32 or weight.dim() != 2 or weight.shape[1] != C or not weight.is_contiguous():
+        raise KernelError(f"conv_rope_store: the taps must be contiguous fp32 [taps, {C}]")
+    taps = weight.shape[0]
     if rot and (angles is None or angles.dtype != torch.float32 or angles.shape != (M, rot) or not angles.is_contiguous()):
         raise KernelError("conv_rope_store: angles must be contiguous fp32 [M, rot]")
     stride = 0

@@ -113,7 +113,7 @@ class ConvAttention(PagedSoftmax):
     def bind(self, tensors, dtype, device):
         self.w_in = self._stack_in(tensors, ("q", "k", "v"), dtype)
         self.w_out = _as_compute(tensors["o"], dtype).contiguous()
-        self.conv_w = torch.cat([_f32(tensors[n]) for n in ("q.conv", "k.conv", "v.conv")], dim=0).contiguous()
+        self.conv_w = torch.cat([_f32(tensors[n]) for n in ("q.conv", "k.conv", "v.conv")], dim=0).t().contiguous()
         self.finish_bind()
 
     def mix(self, proj, out, out_scale, ctx, cache, position):
