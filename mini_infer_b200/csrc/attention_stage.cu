@@ -23,7 +23,8 @@
 MI_DEFINE_ERROR_API()
 
 #define STAGE_TILE 16      // tokens per tile of mi_conv_rope_store
-#define STAGE_THREADS 64
+#define STAGE_THREADS 128
+#define STAGE_RUN 4        // consecutive tokens that a thread of mi_conv_rope_store takes at a time
 #define STAGE_MAX_TAPS 16  // taps - 1 rows of state: only a portion's first tile reads them
 
 __global__ void rope_angles_kernel(const int* __restrict__ positions, const double* __restrict__ freq, float mult,
@@ -90,10 +91,10 @@ struct Piece {
   }
 };
 
-// A thread takes V channels and the V channels that are turned against them (half the rotated span further on; among
-// the dimensions that pass, half of those), and walks a run of the tile's tokens.  TAPS > 0: that many taps; the
-// weights and the last TAPS - 1 inputs of the thread's channels stay in registers, so every projected value is read
-// once per run.  0: `taps` of them, weights and inputs read as they are used.
+// A block takes one head and one tile of tokens; a thread convolves V channels of it for runs of STAGE_RUN tokens.
+// Dimensions that pass go straight to their destination, those that are turned through shared memory (`turned`,
+// [STAGE_TILE][rot] fp32), where the turn finds its partner.  TAPS > 0: that many taps; weights and inputs of a run are
+// in registers, all inputs asked for before the first is used.  0: `taps` of them, read as they are used.
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(STAGE_THREADS)
 conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __restrict__ weight, int taps_any,
@@ -105,25 +106,36 @@ conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __
   mi_pdl_enter();
   constexpr int EPC = 16 / (int)sizeof(T);
   constexpr int NW = TAPS > 0 ? TAPS : 1, NH = TAPS > 1 ? TAPS - 1 : 1;
+  constexpr int NI = TAPS > 0 ? STAGE_RUN + TAPS - 1 : 1;      // inputs of a run
+  extern __shared__ __align__(16) float turned[];
+  __shared__ long long to[STAGE_TILE];                         // where a token's row begins at its destination
+  __shared__ int swz[STAGE_TILE];                              // and the permutation of its 16-byte pieces
   const int taps = TAPS > 0 ? TAPS : taps_any, C = (nq + nkv) * d + nkv * dv;
-  const int tile = blockIdx.x, head = blockIdx.y;
+  const int tile = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
   const int b = tile_req[tile], tok0 = tile_tok0[tile];
   const int ql = q_len[b], qs = q_start[b];
   const int ntok = min(STAGE_TILE, ql - tok0);
   const bool is_q = head < nq, is_v = head >= nq + nkv;
   const int width = is_v ? dv : d, turn = is_v ? 0 : rot, half = turn >> 1;
   const int base = is_v ? (nq + nkv) * d + (head - nq - nkv) * dv : head * d;      // the head's first channel
-  const int kvh = is_v ? head - nq - nkv : head - nq;
   float* past = state ? state + (long long)state_slot[b] * state_stride : nullptr;
-  // items: pairs of pieces; with V = 1 an odd number of passing dimensions leaves the last item without a partner
-  const int rest = width - turn, rest_half = (rest / V + 1) / 2 * V;
-  const int n_turn = half / V, n_items = n_turn + rest_half / V;
-  const int lanes = min(n_items, STAGE_THREADS), groups = STAGE_THREADS / lanes;
-  const int group = threadIdx.x / lanes, lane = threadIdx.x - group * lanes;
-  const int each = (ntok + groups - 1) / groups;
-  const int t_begin = group * each, t_end = group < groups ? min(ntok, t_begin + each) : 0;
-  const int mask = mi_swizzle_mask_rows(width, (int)sizeof(T));
-
+  T* dst = is_q ? q_out : (is_v ? vcache : kcache);
+  if (tid < ntok) {
+    const int row = qs + tok0 + tid;
+    if (is_q) {
+      to[tid] = ((long long)row * nq + head) * d;
+      swz[tid] = 0;
+    } else {
+      const int kvh = is_v ? head - nq - nkv : head - nq, slot = slots[row], page = slot / page_size;
+      const int offset = slot - page * page_size;
+      to[tid] = ((long long)(page * nkv + kvh) * page_size + offset) * width;
+      swz[tid] = offset & mi_swizzle_mask_rows(width, (int)sizeof(T));
+    }
+  }
+  auto put = [&](int tt, int k, const Piece<T, V>& p) {         // V values from dimension k on of the tile's token tt
+    const int s = swz[tt];
+    p.store(dst + to[tt] + (s ? (((k / EPC) ^ s) * EPC + k % EPC) : k));
+  };
   // the projected values of V channels from c on at the portion's token src (negative: before the portion)
   auto input = [&](int src, int c, Piece<T, V>& u) {
     if (src >= 0) {
@@ -134,103 +146,122 @@ conv_rope_store_kernel(const T* __restrict__ packed, int stride, const float* __
       for (int e = 0; e < V; ++e) u.f[e] = p[e];
     }
   };
-  auto weights = [&](float (&w)[NW][V], int c) {
-    if constexpr (TAPS > 0) {
+
+  const int n_items = width / V, lanes = min(n_items, STAGE_THREADS), groups = STAGE_THREADS / lanes;
+  const int group = tid / lanes, lane = tid - group * lanes;
+  // every thread takes part in every round: the first one waits for `to` and `swz` between its loads and its stores
+  bool first = true;
+  for (int item = lane; item - lane < n_items; item += lanes) {
+    const bool mine = item < n_items && group < groups;
+    const int k = item * V, c = base + k;
+    float w[NW][V];
+    if (TAPS > 0 && mine) {
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) {
+      for (int j = 0; j < NW; ++j) {
         Piece<float, V> p;
         p.load(weight + (size_t)j * C + c);
 #pragma unroll
         for (int e = 0; e < V; ++e) w[j][e] = p.f[e];
       }
     }
-  };
-  auto history = [&](Piece<T, V> (&h)[NH], int c, int t) {      // h[j]: the input of token t - (TAPS - 1) + j
-    if constexpr (TAPS > 1) {
+    for (int run0 = 0; run0 < ntok; run0 += groups * STAGE_RUN) {
+      const int run = run0 + group * STAGE_RUN, t0 = tok0 + run, n = mine ? min(STAGE_RUN, ntok - run) : 0;
+      Piece<T, V> u[NI];
+      if (TAPS > 0 && n > 0) {
+        if (t0 >= TAPS - 1 && n == STAGE_RUN) {      // the usual run: no branch between the loads
+          const T* p = packed + (size_t)(qs + t0 - (TAPS - 1)) * stride + c;
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) input(t - TAPS + 1 + j, c, h[j]);
-    }
-  };
-  auto convolve = [&](const float (&w)[NW][V], Piece<T, V> (&h)[NH], int c, int t, Piece<T, V>& y) {
-    Piece<T, V> u;
-    input(t, c, u);
-    if constexpr (TAPS > 0) {
+          for (int j = 0; j < NI; ++j) u[j].load(p + (size_t)j * stride);
+        } else {
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        float acc = 0.f;
+          for (int j = 0; j < NI; ++j)
+            if (j < n + TAPS - 1) input(t0 - (TAPS - 1) + j, c, u[j]);
+          if (TAPS > 1 && ql <= STAGE_RUN) {           // the portion is this run: its last inputs are the new state
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(w[j][e], h[j].f[e], acc);
-        y.f[e] = fmaf(w[TAPS - 1][e], u.f[e], acc);
+            for (int r = 0; r < TAPS - 1; ++r)
 #pragma unroll
-        for (int j = 0; j + 1 < TAPS - 1; ++j) h[j].f[e] = h[j + 1].f[e];
-        if constexpr (TAPS > 1) h[TAPS - 2].f[e] = u.f[e];
-      }
-    } else {
+              for (int e = 0; e < V; ++e) {
+                float v = u[1 + r].f[e];
 #pragma unroll
-      for (int e = 0; e < V; ++e) y.f[e] = 0.f;
-      for (int j = 0; j < taps; ++j) {
-        Piece<T, V> v;
-        input(t - taps + 1 + j, c, v);
-#pragma unroll
-        for (int e = 0; e < V; ++e) y.f[e] = fmaf(weight[(size_t)j * C + c + e], v.f[e], y.f[e]);
-      }
-    }
-  };
-
-  for (int item = lane; item < n_items; item += lanes) {
-    const bool turned = item < n_turn;
-    const int k1 = turned ? item * V : turn + (item - n_turn) * V;      // within the head
-    const int k2 = k1 + (turned ? half : rest_half);
-    const bool two = k2 < width;
-    float w1[NW][V], w2[NW][V];
-    Piece<T, V> h1[NH], h2[NH];
-    if (t_begin < t_end) {
-      weights(w1, base + k1);
-      history(h1, base + k1, tok0 + t_begin);
-      if (two) {
-        weights(w2, base + k2);
-        history(h2, base + k2, tok0 + t_begin);
-      }
-    }
-#pragma unroll 2
-    for (int tt = t_begin; tt < t_end; ++tt) {
-      const int t = tok0 + tt, row = qs + t;
-      Piece<T, V> a, c;
-      convolve(w1, h1, base + k1, t, a);
-      if (two) convolve(w2, h2, base + k2, t, c);
-      if (turned) {
-        const float* sn = angles + (size_t)row * turn + k1;
-        Piece<float, V> s, o;
-        s.load(sn);
-        o.load(sn + half);
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-          const float u = a.f[e], v = c.f[e];
-          mi_rotate(u, v, s.f[e], o.f[e], a.f[e], c.f[e]);
+                for (int m = 2; m <= STAGE_RUN; ++m) v = n == m && m + r < NI ? u[m + r < NI ? m + r : 0].f[e] : v;
+                past[(size_t)r * C + c + e] = v;
+              }
+          }
         }
       }
-      T* dst;
-      int offset = 0, m = 0;
-      if (is_q) {
-        dst = q_out + (size_t)row * nq * d + head * d;
-      } else {
-        const int slot = slots[row], page = slot / page_size;
-        offset = slot - page * page_size;
-        m = mask;
-        dst = (is_v ? vcache : kcache) + ((size_t)(page * nkv + kvh) * page_size + offset) * width;
+      if (first) {
+        __syncthreads();
+        first = false;
       }
-      a.store(dst + (m ? mi_swizzled(k1, offset, m, EPC) : k1));
-      if (two) c.store(dst + (m ? mi_swizzled(k2, offset, m, EPC) : k2));
+#pragma unroll
+      for (int i = 0; i < STAGE_RUN; ++i) {
+        if (i < n) {
+          Piece<T, V> y;
+#pragma unroll
+          for (int e = 0; e < V; ++e) y.f[e] = 0.f;
+          if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+              for (int e = 0; e < V; ++e) y.f[e] = fmaf(w[j][e], u[i + j].f[e], y.f[e]);
+          } else {
+            for (int j = 0; j < taps; ++j) {
+              Piece<T, V> v;
+              input(t0 + i - taps + 1 + j, c, v);
+#pragma unroll
+              for (int e = 0; e < V; ++e) y.f[e] = fmaf(weight[(size_t)j * C + c + e], v.f[e], y.f[e]);
+            }
+          }
+          if (k < turn) {
+            Piece<float, V> p;
+#pragma unroll
+            for (int e = 0; e < V; ++e) p.f[e] = y.f[e];
+            p.store(turned + (run + i) * turn + k);
+          } else {
+            put(run + i, k, y);
+          }
+        }
+      }
     }
   }
-  if (tok0 == 0 && past) {
-    __syncthreads();            // this block, the only reader of these channels' state, has read it
-    for (int k = threadIdx.x; k < width; k += STAGE_THREADS)
-      for (int r = 0; r < taps - 1; ++r) {      // ascending: a row that moves up is read before it is written over
-        const int src = ql - (taps - 1) + r;
-        past[(size_t)r * C + base + k] = src >= 0 ? mi_to_float(packed[(size_t)(qs + src) * stride + base + k])
-                                                  : past[(size_t)(r + ql) * C + base + k];
+  __syncthreads();      // the turned dimensions are in shared memory; this block, the only reader of its state, has read it
+  if (turn) {
+    const int pieces = turn / V;
+    for (int idx = tid; idx < ntok * pieces; idx += STAGE_THREADS) {
+      const int tt = idx / pieces, k = (idx - tt * pieces) * V, i = k < half ? k : k - half;
+      const float* sn = angles + (size_t)(qs + tok0 + tt) * turn + i;
+      Piece<float, V> x, z, s, o;
+      x.load(turned + tt * turn + i);
+      z.load(turned + tt * turn + half + i);
+      s.load(sn);
+      o.load(sn + half);
+      Piece<T, V> y;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float y1, y2;
+        mi_rotate(x.f[e], z.f[e], s.f[e], o.f[e], y1, y2);
+        y.f[e] = k < half ? y1 : y2;
       }
+      put(tt, k, y);
+    }
+  }
+  if (tok0 == 0 && past && !(TAPS > 0 && ql <= STAGE_RUN)) {
+    auto moved = [&](int r, int k) {      // what row r of the state becomes: a later row, or one of the portion's last
+      const int src = ql - (taps - 1) + r;
+      return src >= 0 ? mi_to_float(packed[(size_t)(qs + src) * stride + base + k]) : past[(size_t)(r + ql) * C + base + k];
+    };
+    for (int k = tid; k < width; k += STAGE_THREADS) {
+      if constexpr (TAPS > 0) {               // all rows are asked for before the first is written
+        float v[NH];
+#pragma unroll
+        for (int r = 0; r < TAPS - 1; ++r) v[r] = moved(r, k);
+#pragma unroll
+        for (int r = 0; r < TAPS - 1; ++r) past[(size_t)r * C + base + k] = v[r];
+      } else {
+        for (int r = 0; r < taps - 1; ++r)    // ascending: a row that moves up is read before it is written over
+          past[(size_t)r * C + base + k] = moved(r, k);
+      }
+    }
   }
 }
 
@@ -253,12 +284,14 @@ extern "C" int mi_conv_rope_store(const void* packed, int stride, const float* w
   const int n_heads = nq + 2 * nkv;
   if (n_heads > 65535) MI_REFUSE("conv_rope_store: too many heads for one launch");
   const size_t piece = dtype == MI_DTYPE_F32 ? 16 : 8;
-  const bool four = d % 8 == 0 && dv % 8 == 0 && rot % 8 == 0 && stride % 4 == 0 && mi_aligned(packed, piece) &&
+  const bool four = d % 4 == 0 && dv % 4 == 0 && rot % 8 == 0 && stride % 4 == 0 && mi_aligned(packed, piece) &&
                     mi_aligned(q_out, piece) && mi_aligned(kcache, 16) && mi_aligned(vcache, 16) && mi_aligned(weight, 16) &&
                     mi_aligned(angles, 16);
+  const size_t smem = (size_t)STAGE_TILE * rot * sizeof(float);
+  if (smem > 47 * 1024) MI_REFUSE("conv_rope_store: %d rotated dimensions do not fit in shared memory", rot);
   const dim3 grid((unsigned)n_tiles, (unsigned)n_heads);
 #define MI_CONV(T, V, TAPS)                                                                                           \
-  MI_LAUNCH((conv_rope_store_kernel<T, V, TAPS>), grid, STAGE_THREADS, 0, stream, (const T*)packed, stride, weight,   \
+  MI_LAUNCH((conv_rope_store_kernel<T, V, TAPS>), grid, STAGE_THREADS, smem, stream, (const T*)packed, stride, weight,   \
             taps, taps > 1 ? state : (float*)nullptr, state_stride, state_slot, q_start, q_len, tile_req, tile_tok0,  \
             nq, nkv, d, dv, rot, angles, slots, (T*)q_out, (T*)kcache, (T*)vcache, page_size)
 #define MI_CONV_TAPS(T, V)                                                                                            \
