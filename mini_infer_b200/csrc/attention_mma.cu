@@ -1695,7 +1695,7 @@ extern "C" int mi_attention_prefill_tile_tokens(int g) {
   return PROWS / gb;
 }
 
-extern "C" int mi_attention_prefill_capped(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
+extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
                                     const void* vcache, const int* block_table, int bt_stride, const int* table_rows,
                                     int page_size, const int* q_start, const int* q_len, const int* kv_len,
                                     const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens,
@@ -1732,16 +1732,6 @@ extern "C" int mi_attention_prefill_capped(const void* q, int q_stride, void* ou
   else MI_PREFILL(256);
 #undef MI_PREFILL
   MI_RETURN_LAUNCH_STATUS();
-}
-
-extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int out_stride, const void* kcache,
-                                    const void* vcache, const int* block_table, int bt_stride, const int* table_rows,
-                                    int page_size, const int* q_start, const int* q_len, const int* kv_len,
-                                    const int* tile_req, const int* tile_tok0, int n_tiles, int tile_tokens,
-                                    int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
-  return mi_attention_prefill_capped(q, q_stride, out, out_stride, kcache, vcache, block_table, bt_stride, table_rows,
-                                     page_size, q_start, q_len, kv_len, tile_req, tile_tok0, n_tiles, tile_tokens, nq,
-                                     nkv, d, scale, window, 0, 0.f, stream);
 }
 
 // ------------------------------------------------------------------------------- no allocation

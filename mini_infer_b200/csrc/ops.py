@@ -190,10 +190,6 @@ def _sig_attention_mma(lib: ctypes.CDLL) -> None:
     lib.mi_attention_prefill.argtypes = [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-        c_float, c_int, c_void_p]
-    lib.mi_attention_prefill_capped.argtypes = [
-        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
         c_float, c_int, c_int, c_float, c_void_p]
     lib.mi_attention_prefill_tile_tokens.argtypes = [c_int]
     lib.mi_attention_prefill_tile_tokens.restype = c_int
@@ -884,7 +880,7 @@ def attention_prefill(q, q_stride, out, kcache, vcache, block_table, page_size, 
                            ("kv_len", kv_len), ("tile_req", tile_req), ("tile_tok0", tile_tok0),
                            ("table_rows", table_rows)))
     lib = _waiting_lib("attention_mma", q.device)
-    rc = lib.mi_attention_prefill_capped(
+    rc = lib.mi_attention_prefill(
         _ptr(q), int(q_stride), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(block_table),
         block_table.stride(0), _ptr(table_rows), int(page_size), _ptr(q_start), _ptr(q_len), _ptr(kv_len), _ptr(tile_req),
         _ptr(tile_tok0), int(n_tiles), int(tile_tokens), nq, nkv, head_dim, float(scale), int(window),
