@@ -92,7 +92,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
   for (int e = 0; e < DMAX / 8; ++e) acc[e] = 0.f;
   const int ne = (dv + 7) >> 3;
 
-  const MiKeyWalk walk(j_lo, keep, BK);
+  const MiKeyWalk<true> walk(j_lo, keep, BK);
   const int n_chunks = walk.count(j_end, BK);
   for (int ci = 0; ci < n_chunks; ++ci) {
     const int j0 = walk.chunk(ci) * BK;

@@ -220,15 +220,15 @@ __device__ __forceinline__ void consumer_barrier(int count) {
   asm volatile("bar.sync 1, %0;\n" ::"r"(count) : "memory");
 }
 
-template <int THREADS, bool NAMED = false>
+template <int THREADS, bool NAMED = false, bool KEEP = false>
 __device__ __forceinline__ void zero_masked_values(bf16* vtile, int chunk, int lo, int hi, int d, int keep = 0) {
   const int cb = chunk * KCHUNK;
-  if ((cb >= lo || cb + KCHUNK <= keep) && cb + KCHUNK <= hi) return;   // uniform over the calling threads
+  if ((cb >= lo || (KEEP && cb + KCHUNK <= keep)) && cb + KCHUNK <= hi) return;   // uniform over the calling threads
   const int units = d >> 3;
   for (int idx = threadIdx.x; idx < KCHUNK * units; idx += THREADS) {
     const int r = idx / units, u = idx - r * units;
     const int j = cb + r;
-    if ((j < lo && j >= keep) || j >= hi) *reinterpret_cast<uint4*>(vtile + r * d + u * 8) = make_uint4(0u, 0u, 0u, 0u);
+    if ((j < lo && !(KEEP && j < keep)) || j >= hi) *reinterpret_cast<uint4*>(vtile + r * d + u * 8) = make_uint4(0u, 0u, 0u, 0u);
   }
   fence_proxy_async();   // these writes come before the copy engine's next writes to the tile
   if (NAMED) consumer_barrier(THREADS);
@@ -753,7 +753,8 @@ __device__ __noinline__ void balanced_merge_unit(const float* __restrict__ part_
 }
 
 #define BAL_THREADS (NTHREADS + 64)   // four consumer warps, the copy warp, the store warp (ROPE only)
-template <int DMAX, bool ROPE>
+// EXT: an instance of its own for kept keys and capped scores, so that the others keep their code.
+template <int DMAX, bool ROPE, bool EXT>
 __global__ void __launch_bounds__(ROPE ? BAL_THREADS : DEC_THREADS, DMAX <= 128 ? 2 : 1)
 attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
                                  const bf16* __restrict__ kcache, const bf16* __restrict__ vcache,
@@ -763,7 +764,8 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
                                  int nkv, int d, float scale, int window, int min_chunks, int unit_cost,
                                  float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                                  int* __restrict__ status, const float* __restrict__ rope_cs, int store_kv,
-                                 const float* __restrict__ sinks, int keep, float cap_k, float cap_h) {
+                                 const float* __restrict__ sinks, int keep_any, float cap_k, float cap_h) {
+  const int keep = EXT ? keep_any : 0;
   // sinks [nq] (optional): per head a score that joins the softmax's denominator with neither key nor value.
   // ROPE (the head size is then DMAX exactly): rope_cs holds per query token [d / 2] sines then
   // [d / 2] cosines of its rotary angles; q arrives un-rotated and is rotated here, in registers; and with store_kv
@@ -793,7 +795,7 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
   for (int b = tid; b < B; b += (ROPE ? BAL_THREADS : DEC_THREADS)) {
     const int kl = kv_len[b];
     const int lo = first_visible(kl - 1, window);   // (a window skips the chunks below it)
-    cum[b + 1] = MiKeyWalk(lo, keep, KCHUNK).count(kl, KCHUNK);
+    cum[b + 1] = MiKeyWalk<EXT>(lo, keep, KCHUNK).count(kl, KCHUNK);
   }
   __syncthreads();
   if (warp == 0) {
@@ -858,11 +860,11 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
       const int kvh = u / hblocks;
       const int kl = kv_len[b];
       const int lo_w = first_visible(kl - 1, window);
-      const MiKeyWalk walk(lo_w, keep, KCHUNK);
+      const MiKeyWalk<EXT> walk(lo_w, keep, KCHUNK);
       const int* table = block_table + (size_t)(table_rows ? table_rows[b] : b) * bt_stride;
       for (int s = 0; s < seg && ok; ++s, ++it) {
         const int c = walk.chunk(c_rel + s), st = it % DEC_STAGES;
-        const int lo = c * KCHUNK < keep ? 0 : lo_w;     // a chunk with kept keys is copied from its beginning
+        const int lo = EXT && c * KCHUNK < keep ? 0 : lo_w;     // a chunk with kept keys is copied from its beginning
         if (it >= DEC_STAGES)
           ok = __all_sync(0xffffffffu, mbar_wait_bounded(&empty[st], ((it / DEC_STAGES) - 1) & 1, status));
         if (!ok) break;
@@ -962,7 +964,7 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
     const int head0 = kvh * g + hb * DEC_HEADS;
     const int kl = kv_len[b], tok = q_start[b];
     const int lo = first_visible(kl - 1, window);
-    const MiKeyWalk walk(lo, keep, KCHUNK);
+    const MiKeyWalk<EXT> walk(lo, keep, KCHUNK);
 
     // Q as the B operand: lane (qd, t4) holds head qd, dims ks*16 + 2*t4 + {0,1} and + 8
     uint32_t qb[DMAX / 16][2];
@@ -1002,14 +1004,14 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
         warp_dead = true;
         if (lane == 0) dead = 1;
       }
-      zero_masked_values<NTHREADS, true>(Vs + buf * KCHUNK * d, c, lo, kl, d, keep);
+      zero_masked_values<NTHREADS, true, EXT>(Vs + buf * KCHUNK * d, c, lo, kl, d, keep);
       const int key0 = c * KCHUNK + warp * 16;
       const int kr = lane & 15, vr = (lane & 7) + (lane >> 4) * 8;
       const int ksw = inpage_of(key0 + kr, page_size, page_shift) & swz_mask;
       const int vsw = inpage_of(key0 + vr, page_size, page_shift) & swz_mask;
       const bf16* Kb = Ks + buf * KCHUNK * d + (warp * 16 + kr) * d;
       const bf16* Vb = Vs + buf * KCHUNK * d + (warp * 16 + vr) * d;
-      if (arrived && key0 < kl && (key0 + 16 > lo || key0 < keep)) {   // (the arithmetic of attention_decode_kernel)
+      if (arrived && key0 < kl && (key0 + 16 > lo || (EXT && key0 < keep))) {   // (the arithmetic of attention_decode_kernel)
         constexpr int GROUP = (DMAX / 16) < 8 ? (DMAX / 16) : 8;
         float sa[4] = {0.f, 0.f, 0.f, 0.f}, s_odd[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -1032,18 +1034,12 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
         for (int k = 0; k < GROUP; ++k)
           if (k < ksteps) ldmatrix_x4_trans(vf[k], Vb + (((k * 2 + ((lane >> 3) & 1)) ^ vsw) << 3));
         const int j0 = key0 + qd, j1 = j0 + 8;
-        const bool ok0 = j0 < kl && (j0 >= lo || j0 < keep), ok1 = j1 < kl && (j1 >= lo || j1 < keep);
-        if (cap_k > 0.f) {   // (the same for the whole launch)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) sa[e] = mi_softcap(sa[e], cap_k, cap_h);
-        } else {
-#pragma unroll
-          for (int e = 0; e < 4; ++e) sa[e] *= sc;
-        }
-        sa[0] = ok0 ? sa[0] : -INFINITY;
-        sa[1] = ok0 ? sa[1] : -INFINITY;
-        sa[2] = ok1 ? sa[2] : -INFINITY;
-        sa[3] = ok1 ? sa[3] : -INFINITY;
+        const bool ok0 = j0 < kl && (j0 >= lo || (EXT && j0 < keep)), ok1 = j1 < kl && (j1 >= lo || (EXT && j1 < keep));
+        auto scored = [&](float s) { return EXT && cap_k > 0.f ? mi_softcap(s, cap_k, cap_h) : s * sc; };
+        sa[0] = ok0 ? scored(sa[0]) : -INFINITY;
+        sa[1] = ok0 ? scored(sa[1]) : -INFINITY;
+        sa[2] = ok1 ? scored(sa[2]) : -INFINITY;
+        sa[3] = ok1 ? scored(sa[3]) : -INFINITY;
         float alpha[2], p[4];
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
@@ -1201,7 +1197,8 @@ struct PrefillShape {
   static constexpr int BLOCKS_PER_SM = DMAX <= 128 ? 2 : 1;
 };
 
-template <int DMAX>
+// EXT: as in the balanced decode kernel
+template <int DMAX, bool EXT>
 __global__ void __launch_bounds__(PrefillShape<DMAX>::THREADS, PrefillShape<DMAX>::BLOCKS_PER_SM)
 attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
                          const bf16* __restrict__ kcache, const bf16* __restrict__ vcache,
@@ -1210,7 +1207,8 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                          const int* __restrict__ q_start, const int* __restrict__ q_len,
                          const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                          const int* __restrict__ tile_tok0, int nq, int nkv, int d, float scale, int window,
-                         int gb, int tt, int* __restrict__ status, int keep, float cap_k, float cap_h) {
+                         int gb, int tt, int* __restrict__ status, int keep_any, float cap_k, float cap_h) {
+  const int keep = EXT ? keep_any : 0;
   constexpr int MT = PrefillShape<DMAX>::MT;
   constexpr int THREADS = PrefillShape<DMAX>::THREADS;
   mi_pdl_enter();   // inputs come from the kernels before this one
@@ -1282,12 +1280,12 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
 #pragma unroll
     for (int i = 0; i < DMAX / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
   }
-  const float sc = cap_k > 0.f ? 1.f : scale * LOG2E;   // capped scores are exponents already
+  const float sc = EXT && cap_k > 0.f ? 1.f : scale * LOG2E;   // capped scores are exponents already
   const int ksteps = d >> 4;
-  const MiKeyWalk walk(lo, keep, KCHUNK);
+  const MiKeyWalk<EXT> walk(lo, keep, KCHUNK);
   const int n_chunks = walk.count(hi, KCHUNK);
   const int c0 = walk.chunk(0);
-  auto load_lo = [&](int c) { return c * KCHUNK < keep ? 0 : lo; };   // a chunk with kept keys is copied from its beginning
+  auto load_lo = [&](int c) { return EXT && c * KCHUNK < keep ? 0 : lo; };   // a chunk with kept keys is copied from its beginning
   const uint32_t q_addr = smem_u32(Qs) + (uint32_t)((row0 + (lane & 15)) * sd + (lane >> 4) * 8) * 2u;
 
   __shared__ __align__(8) uint64_t bars[2];
@@ -1315,7 +1313,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       if (it + 2 < n_chunks) loader.fetch(table, page_size, page_shift, walk.chunk(it + 2), load_lo(walk.chunk(it + 2)), hi);
     }
     const bool arrived = __all_sync(0xffffffffu, mbar_wait_bounded(&bars[buf], (it >> 1) & 1, status));
-    zero_masked_values<THREADS>(Vs + buf * KCHUNK * d, c, lo, hi, d, keep);
+    zero_masked_values<THREADS, false, EXT>(Vs + buf * KCHUNK * d, c, lo, hi, d, keep);
     const bf16* Kb = Ks + buf * KCHUNK * d;
     const bf16* Vb = Vs + buf * KCHUNK * d;
     const int key0 = c * KCHUNK;
@@ -1338,7 +1336,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         vxor[i] = (uint32_t)((vsw & ~1) << 4);
       }
     }
-    if (arrived && warp_active && key0 < warp_hi && (key0 + KCHUNK > warp_lo || key0 < keep)) {
+    if (arrived && warp_active && key0 < warp_hi && (key0 + KCHUNK > warp_lo || (EXT && key0 < keep))) {
       float s[MT][8][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
@@ -1368,10 +1366,10 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       // few on the diagonal and at a window's edge) needs no mask.  Scores stay unscaled; the
       // scale is folded into the exponent's multiply-add: p = 2^(s * sc - m), m = sc * max(s).
       const bool interior = key0 + KCHUNK - 1 <= p_first + wt0 &&
-                            (key0 >= first_visible(p_first + wt1, window) || key0 + KCHUNK <= keep);
+                            (key0 >= first_visible(p_first + wt1, window) || (EXT && key0 + KCHUNK <= keep));
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
-        if (cap_k > 0.f) {   // (the same for the whole launch)
+        if (EXT && cap_k > 0.f) {   // (the same for the whole launch)
 #pragma unroll
           for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
@@ -1384,7 +1382,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
             for (int e = 0; e < 4; ++e) {
               const int hr = e >> 1;
               const int j = key0 + nt * 8 + 2 * t4 + (e & 1);
-              if (!(rvalid[mt][hr] && j <= prow[mt][hr] && (j >= lorow[mt][hr] || j < keep))) s[mt][nt][e] = -INFINITY;
+              if (!(rvalid[mt][hr] && j <= prow[mt][hr] && (j >= lorow[mt][hr] || (EXT && j < keep)))) s[mt][nt][e] = -INFINITY;
             }
         }
         // both rows of the lane side by side and sums in four strands: short dependency chains
@@ -1665,9 +1663,9 @@ extern "C" int mi_attention_decode_balanced(const void* q, int q_stride, void* o
   if (B > 16384) MI_REFUSE("attention: %d requests in one decode step", B);
   const int page_shift = shift_of(page_size);
   const size_t smem = balanced_smem_bytes(B, d);
-#define MI_DECODE_BAL(DMAX, ROPE)                                                                         \
+#define MI_DECODE_BAL(DMAX, ROPE, EXT)                                                                         \
   do {                                                                                                    \
-    auto kern = attention_decode_balanced_kernel<DMAX, ROPE>;                                             \
+    auto kern = attention_decode_balanced_kernel<DMAX, ROPE, EXT>;                                             \
     if (smem > 40 * 1024) {                                                                               \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       if (e != cudaSuccess) return (int)e;                                                                \
@@ -1679,12 +1677,17 @@ extern "C" int mi_attention_decode_balanced(const void* q, int q_stride, void* o
               cap_k, cap_h);                                                                              \
   } while (0)
   if (rope_cs) {
-    if (d == 64) MI_DECODE_BAL(64, true);
-    else if (d == 128) MI_DECODE_BAL(128, true);
-    else MI_DECODE_BAL(256, true);
-  } else if (d <= 64) MI_DECODE_BAL(64, false);
-  else if (d <= 128) MI_DECODE_BAL(128, false);
-  else MI_DECODE_BAL(256, false);
+    if (keep || softcap > 0.f) MI_REFUSE("attention: the decode kernel that rotates takes neither kept keys nor a cap");
+    if (d == 64) MI_DECODE_BAL(64, true, false);
+    else if (d == 128) MI_DECODE_BAL(128, true, false);
+    else MI_DECODE_BAL(256, true, false);
+  } else if (keep || softcap > 0.f) {
+    if (d <= 64) MI_DECODE_BAL(64, false, true);
+    else if (d <= 128) MI_DECODE_BAL(128, false, true);
+    else MI_DECODE_BAL(256, false, true);
+  } else if (d <= 64) MI_DECODE_BAL(64, false, false);
+  else if (d <= 128) MI_DECODE_BAL(128, false, false);
+  else MI_DECODE_BAL(256, false, false);
 #undef MI_DECODE_BAL
   MI_RETURN_LAUNCH_STATUS();
 }
@@ -1714,9 +1717,9 @@ extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int 
   const size_t smem = smem_bytes(PROWS, d);
   const int page_shift = shift_of(page_size);
   dim3 grid((unsigned)(n_tiles * nkv * hblocks));
-#define MI_PREFILL(DMAX)                                                                                \
+#define MI_PREFILL(DMAX, EXT)                                                                                \
   do {                                                                                                  \
-    auto kern = attention_prefill_kernel<DMAX>;                                                         \
+    auto kern = attention_prefill_kernel<DMAX, EXT>;                                                         \
     if (smem > 40 * 1024) {                                                                             \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       if (e != cudaSuccess) return (int)e;                                                              \
@@ -1727,9 +1730,13 @@ extern "C" int mi_attention_prefill(const void* q, int q_stride, void* out, int 
                                            tile_req, tile_tok0, nq, nkv, d, scale, window, gb,          \
                                            PROWS / gb, wait_status_ptr(), keep, cap_k, cap_h);          \
   } while (0)
-  if (d <= 64) MI_PREFILL(64);
-  else if (d <= 128) MI_PREFILL(128);
-  else MI_PREFILL(256);
+  if (keep || softcap > 0.f) {
+    if (d <= 64) MI_PREFILL(64, true);
+    else if (d <= 128) MI_PREFILL(128, true);
+    else MI_PREFILL(256, true);
+  } else if (d <= 64) MI_PREFILL(64, false);
+  else if (d <= 128) MI_PREFILL(128, false);
+  else MI_PREFILL(256, false);
 #undef MI_PREFILL
   MI_RETURN_LAUNCH_STATUS();
 }

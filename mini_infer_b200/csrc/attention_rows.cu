@@ -119,7 +119,8 @@ struct RowMap {
 
 // DVW: value columns per warp that the accumulators have room for (dv <= 4 * DVW).  DB: two buffers for
 // the chunk's rows; the next chunk is copied (cp.async) while this one is multiplied.
-template <int DVW, int MT, bool DB>
+// EXT: an instance of its own for kept keys and capped scores, so that the others keep their code.
+template <int DVW, int MT, bool DB, bool EXT>
 __global__ void __launch_bounds__(QUARTERS * MT * 32)
 attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
                       const bf16* __restrict__ kcache, const bf16* __restrict__ vcache,
@@ -128,8 +129,9 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
                       const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                       const int* __restrict__ tile_tok0, int tile_tokens, int nq, int nkv, int d, int dv, float scale,
                       const float* __restrict__ sinks, const float* __restrict__ slopes, int v_prefix,
-                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep,
+                      int n_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep_any,
                       float softcap) {
+  const int keep = EXT ? keep_any : 0;
   mi_pdl_enter();
   constexpr int R = ROWS * MT, NW = QUARTERS * MT, NT = NW * 32;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -168,10 +170,10 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
   auto row_head = [&](int r) { return rows.head(r); };
   // this block's run of keys: whole chunks, the same cut for every row of the tile
   const int j_lo = window > 0 ? max(0, p0 - window + 1) : 0;    // the first key that any row sees
-  const MiKeyWalk walk(j_lo, keep, CHUNK);
+  const MiKeyWalk<EXT> walk(j_lo, keep, CHUNK);
   const int chunks_all = walk.count(j_end, CHUNK), chunks_mine = (chunks_all + n_splits - 1) / n_splits;
   const int i_begin = split * chunks_mine, i_stop = min(chunks_all, (split + 1) * chunks_mine);
-  const float cap_k = softcap > 0.f ? scale / softcap : 0.f;
+  const float cap_k = EXT && softcap > 0.f ? scale / softcap : 0.f;
 
   // ---- the queries: 16-byte pieces, zero for rows without a token
   const int pieces = d >> 3;
@@ -203,7 +205,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
     if (tid < CHUNK) {
       const int j = walk.chunk(i) * CHUNK + tid;
       int base = -1;
-      if (i < i_stop && j < j_end && (j >= j_lo || j < keep)) {
+      if (i < i_stop && j < j_end && (j >= j_lo || (EXT && j < keep))) {
         const int page = block_table[(size_t)trow * bt_stride + j / page_size];
         base = (page * nkv + kvh) * page_size + j % page_size;
       }
@@ -281,8 +283,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict
         const bool hi = e >= 2;
         const int pos = hi ? pos_hi : pos_lo;
         // not behind the query; not before its window, unless it is one of the kept first keys
-        const bool ok = (hi ? ok_hi : ok_lo) && ((unsigned)(pos - j) < span || (j < keep && j <= pos));
-        const float raw = softcap > 0.f ? mi_softcap(s[n][e], cap_k, softcap) : s[n][e] * scale;
+        const bool ok = (hi ? ok_hi : ok_lo) && ((unsigned)(pos - j) < span || (EXT && j < keep && j <= pos));
+        const float raw = EXT && softcap > 0.f ? mi_softcap(s[n][e], cap_k, softcap) : s[n][e] * scale;
         const float v = ok ? (raw - (hi ? slope_hi : slope_lo) * (float)(pos - j)) * LOG2E : -INFINITY;
         s[n][e] = v;
         if (hi) mx_hi = fmaxf(mx_hi, v); else mx_lo = fmaxf(mx_lo, v);
@@ -541,9 +543,10 @@ extern "C" int mi_attention_rows(const void* q, int q_stride, void* out, int out
                        (size_t)rows * (CHUNK + PAD)) * sizeof(bf16) +
                       2 * QUARTERS * rows * sizeof(float) + (size_t)stages * 2 * CHUNK * sizeof(int);
   if (smem > 227 * 1024) MI_REFUSE("attention_rows: keys of %d and values of %d do not fit in shared memory", d, dv);
+  const bool ext = keep > 0 || softcap > 0.f;
 #define MI_GO(DVW, MT, DB)                                                                                      \
   do {                                                                                                          \
-    auto kern = attention_rows_kernel<DVW, MT, DB>;                                                             \
+    auto kern = ext ? attention_rows_kernel<DVW, MT, DB, true> : attention_rows_kernel<DVW, MT, DB, false>;                                                            \
     if (smem > 48 * 1024) {                                                                                     \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
       if (e != cudaSuccess) return (int)e;                                                                      \

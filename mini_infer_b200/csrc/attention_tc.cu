@@ -228,6 +228,11 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // A row of 64 raw scores s to cap_h tanh(s cap_k).  Scores far below the cap (the whole warp's) take the
 // polynomial in the two-wide instructions, six per pair; others the exponential form.
 __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
@@ -252,8 +257,16 @@ __device__ __forceinline__ void cap_scores(float (&s)[64], float cap_k, float ca
       unpair(mul2(x, fma2(fma2(fma2(fma2(p4, z, p3), z, p2), z, p1), z, p0)), s[j], s[j + 1]);
     }
   } else {
+    // cap_h tanh(t) = cap_h - 2 cap_h / (e^(2t) + 1), for either sign and any size of t
+    const float k = 2.f * LOG2E * cap_k;
+    const uint64_t k2 = pair_of(k, k), one = pair_of(1.f, 1.f), top = pair_of(cap_h, cap_h), minus = pair_of(-2.f * cap_h, -2.f * cap_h);
 #pragma unroll
-    for (int j = 0; j < 64; ++j) s[j] = mi_softcap(s[j], cap_k, cap_h);
+    for (int j = 0; j < 64; j += 2) {
+      float a, b;
+      unpair(mul2(pair_of(s[j], s[j + 1]), k2), a, b);
+      unpair(add2(pair_of(fast_exp2(a), fast_exp2(b)), one), a, b);
+      unpair(fma2(pair_of(fast_rcp(a), fast_rcp(b)), minus, top), s[j], s[j + 1]);
+    }
   }
 }
 
@@ -282,9 +295,9 @@ enum {
   B_COUNT = 4 * NSTAGE + 12
 };
 
-// CAPPED (with cap_k > 0): a raw score s counts as cap_h tanh(s cap_k), in the exponents' units, before the mask.
-// keep > 0: beside its window a row also sees the first `keep` keys of the sequence.
-template <bool CAPPED>
+// Instances of their own, so that the plain one keeps its code: KEEP, beside its window a row also sees the first
+// `keep` keys of the sequence; CAPPED, a raw score s counts as cap_h tanh(s cap_k), in the exponents' units.
+template <bool KEEP, bool CAPPED>
 __global__ void __launch_bounds__(TC_THREADS, 2 / NTILE)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out, int out_stride,
@@ -294,7 +307,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             const int* __restrict__ kv_len, const int* __restrict__ tile_req,
                             const int* __restrict__ tile_tok0, int nq, int nkv, int d, float scale, int window,
                             int chunk, int gb, int tt, const float* __restrict__ sinks, const float* __restrict__ slopes,
-                            int keep, float cap_k, float cap_h) {
+                            int keep_any, float cap_k, float cap_h) {
+  const int keep = KEEP ? keep_any : 0;
   mi_pdl_enter();   // inputs come from the kernels before this one
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -326,7 +340,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   int lo = window > 0 ? max(0, p_first - window + 1) : 0;
   if (chunk > 0) lo = max(lo, (p_first / chunk) * chunk);
   const int heads_here = min(gb, g - hb * gb);
-  const MiKeyWalk walk(lo, keep, KC);
+  const MiKeyWalk<KEEP> walk(lo, keep, KC);
   const int n_chunks = walk.count(hi, KC);
   volatile int* gu = &give_up;
 
@@ -521,11 +535,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       }
       const bool interior = key0 + KC - 1 <= t_first &&
                             ((key0 >= (window > 0 ? max(0, t_last - window + 1) : 0) &&
-                              key0 >= (chunk > 0 ? (t_last / chunk) * chunk : 0) && key0 >= lo) || key0 + KC <= keep);
+                              key0 >= (chunk > 0 ? (t_last / chunk) * chunk : 0) && key0 >= lo) || (KEEP && key0 + KC <= keep));
       if (!interior || !rvalid) {
 #pragma unroll
         for (int j = 0; j < 64; ++j)
-          if (!(rvalid && key0 + j <= prow && (key0 + j >= lorow || key0 + j < keep))) s[j] = -INFINITY;
+          if (!(rvalid && key0 + j <= prow && (key0 + j >= lorow || (KEEP && key0 + j < keep)))) s[j] = -INFINITY;
       }
       // The exponents are taken relative to m_run, which follows the true running maximum
       // lazily: it moves (and O and l are rescaled) only when some row of the warp found a
@@ -609,12 +623,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       // clear them, 0 * NaN is NaN.  Only a request's first and last chunks have such rows.  Each
       // tile does it before it publishes its probabilities (the tiles' second products are
       // issued independently; both write the same zeros).
-      if ((key0 < lo && key0 + KC > keep) || key0 + KC > hi) {
+      if ((key0 < lo && !(KEEP && key0 + KC <= keep)) || key0 + KC > hi) {
         if (!warp_wait(&bars[B_VFULL + st], round & 1, gu)) { ok = false; break; }
         unsigned char* vt = Vs + st * tile_bytes;
         for (int idx = r; idx < KC * halves * 8; idx += ROWS) {
           const int j = idx / (halves * 8), rest = idx - j * (halves * 8);
-          if ((key0 + j < lo && key0 + j >= keep) || key0 + j >= hi)
+          if ((key0 + j < lo && !(KEEP && key0 + j < keep)) || key0 + j >= hi)
             *reinterpret_cast<uint4*>(vt + (rest >> 3) * (KC * 128) + j * 128 + ((rest & 7) << 4)) = make_uint4(0u, 0u, 0u, 0u);
         }
         fence_async_smem();   // plain stores that the tensor core reads
@@ -1058,7 +1072,8 @@ extern "C" int mi_attention_prefill_tc_capped(const void* q, int q_stride, void*
     MI_REFUSE("attention_tc: the driver refused a tensor map");
   const int halves = d / 64;
   const size_t smem = (size_t)NTILE * ROWS * 128 * halves + 2 * NSTAGE * (size_t)KC * 128 * halves + 1024;
-  auto kern = softcap > 0.f ? attention_prefill_tc_kernel<true> : attention_prefill_tc_kernel<false>;
+  auto kern = keep ? (softcap > 0.f ? attention_prefill_tc_kernel<true, true> : attention_prefill_tc_kernel<true, false>)
+                   : (softcap > 0.f ? attention_prefill_tc_kernel<false, true> : attention_prefill_tc_kernel<false, false>);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const long long n_blocks = (long long)n_tiles * nkv * hblocks;

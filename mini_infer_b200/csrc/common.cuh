@@ -196,15 +196,16 @@ __device__ __forceinline__ void mi_rotate(float x1, float x2, float s, float c, 
 
 // The walk over a row of keys cut into chunks of `size`, for queries that see the keys from `lo` on and, with
 // keep > 0, the first `keep` keys of the sequence as well: the chunks that hold kept keys below lo's chunk, then
-// the chunks from lo's on.
+// the chunks from lo's on.  Without KEEP no key is kept, and nothing of it is left in the code.
+template <bool KEEP>
 struct MiKeyWalk {
   int pre, c0;
   __host__ __device__ __forceinline__ MiKeyWalk(int lo, int keep, int size) {
     c0 = lo / size;
-    pre = keep > 0 ? (keep + size - 1) / size : 0;
-    if (pre > c0) pre = c0;
+    pre = KEEP && keep > 0 ? (keep + size - 1) / size : 0;
+    if (KEEP && pre > c0) pre = c0;
   }
-  __host__ __device__ __forceinline__ int chunk(int i) const { return i < pre ? i : c0 + i - pre; }
+  __host__ __device__ __forceinline__ int chunk(int i) const { return KEEP && i < pre ? i : c0 + i - pre; }
   // chunks of the walk when the keys end at `hi` (exclusive)
   __host__ __device__ __forceinline__ int count(int hi, int size) const { return pre + (hi + size - 1) / size - c0; }
 };
