@@ -1035,11 +1035,17 @@ attention_decode_balanced_kernel(const bf16* __restrict__ q, int q_stride, bf16*
           if (k < ksteps) ldmatrix_x4_trans(vf[k], Vb + (((k * 2 + ((lane >> 3) & 1)) ^ vsw) << 3));
         const int j0 = key0 + qd, j1 = j0 + 8;
         const bool ok0 = j0 < kl && (j0 >= lo || (EXT && j0 < keep)), ok1 = j1 < kl && (j1 >= lo || (EXT && j1 < keep));
-        auto scored = [&](float s) { return EXT && cap_k > 0.f ? mi_softcap(s, cap_k, cap_h) : s * sc; };
-        sa[0] = ok0 ? scored(sa[0]) : -INFINITY;
-        sa[1] = ok0 ? scored(sa[1]) : -INFINITY;
-        sa[2] = ok1 ? scored(sa[2]) : -INFINITY;
-        sa[3] = ok1 ? scored(sa[3]) : -INFINITY;
+        if (EXT && cap_k > 0.f) {   // (the same for the whole launch)
+          sa[0] = ok0 ? mi_softcap(sa[0], cap_k, cap_h) : -INFINITY;
+          sa[1] = ok0 ? mi_softcap(sa[1], cap_k, cap_h) : -INFINITY;
+          sa[2] = ok1 ? mi_softcap(sa[2], cap_k, cap_h) : -INFINITY;
+          sa[3] = ok1 ? mi_softcap(sa[3], cap_k, cap_h) : -INFINITY;
+        } else {
+          sa[0] = ok0 ? sa[0] * sc : -INFINITY;
+          sa[1] = ok0 ? sa[1] * sc : -INFINITY;
+          sa[2] = ok1 ? sa[2] * sc : -INFINITY;
+          sa[3] = ok1 ? sa[3] * sc : -INFINITY;
+        }
         float alpha[2], p[4];
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {

@@ -228,11 +228,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-__device__ __forceinline__ float fast_rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+// tanh(t) for |t| <= TANH_POLY as t P(t^2): the coefficients are a minimax fit (iteratively reweighted least squares
+// on a dense grid) with an error of 2e-8.
+#define TANH_POLY 0.6f
+#define TANH_C0 0.999999627f
+#define TANH_C1 -0.333312086f
+#define TANH_C2 0.132992106f
+#define TANH_C3 -0.0516967532f
+#define TANH_C4 0.0149769696f
 // A row of 64 raw scores s to cap_h tanh(s cap_k).  Scores far below the cap (the whole warp's) take the
 // polynomial in the two-wide instructions, six per pair; others the exponential form.
 __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
@@ -245,11 +248,11 @@ __device__ __forceinline__ void cap_scores(float (&s)[64], float cap_k, float ca
 #pragma unroll
   for (int j = 0; j < 64; j += 2) m4[j >> 4] = (j & 15) ? max3(m4[j >> 4], fabsf(s[j]), fabsf(s[j + 1])) : fmaxf(fabsf(s[j]), fabsf(s[j + 1]));
   const float largest = fmaxf(max3(m4[0], m4[1], m4[2]), m4[3]) * cap_k;
-  if (__all_sync(0xffffffffu, largest <= MI_TANH_POLY)) {
+  if (__all_sync(0xffffffffu, largest <= TANH_POLY)) {
     // the factors ride in the coefficients: y = s (c0 + z (c1 + z (c2 + z (c3 + z c4)))), z = s^2
     const float k1 = cap_h * cap_k, k2 = cap_k * cap_k;
-    const float c0 = MI_TANH_C0 * k1, c1 = MI_TANH_C1 * k1 * k2, c2 = MI_TANH_C2 * k1 * k2 * k2,
-                c3 = MI_TANH_C3 * k1 * k2 * k2 * k2, c4 = MI_TANH_C4 * k1 * k2 * k2 * k2 * k2;
+    const float c0 = TANH_C0 * k1, c1 = TANH_C1 * k1 * k2, c2 = TANH_C2 * k1 * k2 * k2,
+                c3 = TANH_C3 * k1 * k2 * k2 * k2, c4 = TANH_C4 * k1 * k2 * k2 * k2 * k2;
     const uint64_t p0 = pair_of(c0, c0), p1 = pair_of(c1, c1), p2 = pair_of(c2, c2), p3 = pair_of(c3, c3), p4 = pair_of(c4, c4);
 #pragma unroll
     for (int j = 0; j < 64; j += 2) {
@@ -257,7 +260,7 @@ __device__ __forceinline__ void cap_scores(float (&s)[64], float cap_k, float ca
       unpair(mul2(x, fma2(fma2(fma2(fma2(p4, z, p3), z, p2), z, p1), z, p0)), s[j], s[j + 1]);
     }
   } else {
-    // cap_h tanh(t) = cap_h - 2 cap_h / (e^(2t) + 1), for either sign and any size of t
+    // mi_softcap, two at a time
     const float k = 2.f * LOG2E * cap_k;
     const uint64_t k2 = pair_of(k, k), one = pair_of(1.f, 1.f), top = pair_of(cap_h, cap_h), minus = pair_of(-2.f * cap_h, -2.f * cap_h);
 #pragma unroll
@@ -265,7 +268,7 @@ __device__ __forceinline__ void cap_scores(float (&s)[64], float cap_k, float ca
       float a, b;
       unpair(mul2(pair_of(s[j], s[j + 1]), k2), a, b);
       unpair(add2(pair_of(fast_exp2(a), fast_exp2(b)), one), a, b);
-      unpair(fma2(pair_of(fast_rcp(a), fast_rcp(b)), minus, top), s[j], s[j + 1]);
+      unpair(fma2(pair_of(mi_fast_rcp(a), mi_fast_rcp(b)), minus, top), s[j], s[j + 1]);
     }
   }
 }

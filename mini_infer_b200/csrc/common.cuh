@@ -210,24 +210,22 @@ struct MiKeyWalk {
   __host__ __device__ __forceinline__ int count(int hi, int size) const { return pre + (hi + size - 1) / size - c0; }
 };
 
-// tanh(t) for |t| <= MI_TANH_POLY as t P(t^2): the coefficients are a minimax fit (iteratively reweighted least
-// squares on a dense grid) with an error of 2e-8.
-#define MI_TANH_POLY 0.6f
-#define MI_TANH_C0 0.999999627f
-#define MI_TANH_C1 -0.333312086f
-#define MI_TANH_C2 0.132992106f
-#define MI_TANH_C3 -0.0516967532f
-#define MI_TANH_C4 0.0149769696f
-__device__ __forceinline__ float mi_tanh_wide(float t) {      // 1 - 2 / (e^(2t) + 1), an absolute error near 1e-7
-  return 1.f - __fdividef(2.f, __expf(2.f * t) + 1.f);
+__device__ __forceinline__ float mi_fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
-// A capped score for scores whose weights are rounded to bfloat16: height * tanh(s * k), with k = scale / cap and
-// height = cap (or cap log2 e, for exponents to base two).
+__device__ __forceinline__ float mi_fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// A capped score for scores whose weights are rounded to bfloat16: height * tanh(s * k), k = scale / cap and height = cap
+// (or cap log2 e, for exponents to base two), as height - 2 height / (e^(2 s k) + 1): for either sign and any size of s,
+// with an absolute error near 1e-7 of the height.
 __device__ __forceinline__ float mi_softcap(float s, float k, float height) {
-  const float t = s * k, z = t * t;
-  const float p = fmaf(fmaf(fmaf(fmaf(MI_TANH_C4, z, MI_TANH_C3), z, MI_TANH_C2), z, MI_TANH_C1), z, MI_TANH_C0);
-  const float a = fminf(fabsf(t), 40.f);
-  return height * (a <= MI_TANH_POLY ? t * p : copysignf(mi_tanh_wide(a), t));
+  constexpr float TWO_LOG2E = 2.8853900817779268f;
+  return fmaf(-2.f * height, mi_fast_rcp(mi_fast_exp2(s * (TWO_LOG2E * k)) + 1.f), height);
 }
 
 // An activation of one value: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0.
